@@ -31,6 +31,19 @@ def add_rmsnorm(h, delta, gain, eps, out, rows=None):
     out.copy_(((x * scale) * gain).to(out.dtype))
 
 
+def add_layernorm(h, delta, gain, bias, eps, out, rows=None):
+    if rows is None:
+        if delta is not None:
+            h += delta.float()
+        x = h
+    else:
+        x = h[rows.long()]
+        if delta is not None:
+            x = x + delta[rows.long()].float()
+    x = x - x.mean(-1, keepdim=True)
+    out.copy_((x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * gain + bias).to(out.dtype))
+
+
 def residual_add(h, delta):
     h += delta.float()
 
@@ -382,9 +395,10 @@ def qkv_bias_rope_cache(q, k, v, num_heads, num_kv_heads, key_dim, value_dim, q_
                     v_cache[s // page_size, :, s % page_size, :] = vv[t].to(v_cache.dtype)
 
 
-def causal_conv_act(x, w, bias, y, num_seqs, seq_ids, q_start, state_slots, state, conv_offset):
+def causal_conv_act(x, w, bias, y, num_seqs, seq_ids, q_start, state_slots, state, conv_offset,
+                    keep=True):
     C, taps = w.shape
-    keep = taps - 1
+    moves_on, keep = keep, taps - 1
     for b in range(num_seqs):
         t0, t1 = int(q_start[b]), int(q_start[b + 1])
         row = state[int(state_slots[b])]
@@ -392,8 +406,32 @@ def causal_conv_act(x, w, bias, y, num_seqs, seq_ids, q_start, state_slots, stat
         full = torch.cat([kept, x[t0:t1].float()], dim=0)
         for t in range(t1 - t0):
             a = (full[t:t + taps] * w.t()).sum(0) + (bias if bias is not None else 0.0)
-            y[t0 + t] = a * torch.sigmoid(a)
-        if keep:
+            y[t0 + t] = (a * torch.sigmoid(a)).to(y.dtype)
+        if keep and moves_on:
+            kept.copy_(full[full.shape[0] - keep:])
+
+
+def channel_scan(x, z, dt_raw, dt_bias, a2, bm, cm, d_skip, y, num_seqs, q_start, state_slots, state,
+                 ssm_offset, conv_in=None, taps=1, conv_offset=0):
+    T, C = x.shape
+    N = a2.shape[1]
+    for b in range(num_seqs):
+        t0, t1 = int(q_start[b]), int(q_start[b + 1])
+        row = state[int(state_slots[b])]
+        S = row[ssm_offset:ssm_offset + C * N].view(C, N)
+        for t in range(t0, t1):
+            dt = torch.nn.functional.softplus(dt_raw[t] + (dt_bias if dt_bias is not None else 0.0),
+                                              threshold=1e9)
+            xt = x[t].float()
+            S.mul_(torch.exp2(dt[:, None] * a2)).add_((dt * xt)[:, None] * bm[t].float()[None, :])
+            out = S @ cm[t].float()
+            if d_skip is not None:
+                out = out + d_skip * xt
+            y[t] = (out * torch.nn.functional.silu(z[t].float())).to(y.dtype)
+        keep = taps - 1
+        if conv_in is not None and keep:
+            kept = row[conv_offset:conv_offset + keep * C].view(keep, C)
+            full = torch.cat([kept.clone(), conv_in[t0:t1].float()])
             kept.copy_(full[full.shape[0] - keep:])
 
 
@@ -428,7 +466,8 @@ def _plain_act(z, activation):
 
 
 def moe_feed_forward(x, w_router, b_router, w_gate, w_up, w_down, top, activation, extra=None,
-                     scores="chosen", correction=None, identity=0, extra_gated=False):
+                     scores="chosen", correction=None, identity=0, extra_gated=False, groups=1, keep=1,
+                     renormalize=True, route_scale=1.0, beside=None, residual=None):
     T, d = x.shape
     E = w_up.shape[0]
     outputs = E + identity
@@ -437,15 +476,23 @@ def moe_feed_forward(x, w_router, b_router, w_gate, w_up, w_down, top, activatio
     z = z[:, :outputs] + (b_router if b_router is not None else 0.0)
     out = torch.zeros((T, d), dtype=torch.float32)
     for t in range(T):
-        if scores == "all":
-            sc = torch.softmax(z[t], dim=0)
+        if scores != "chosen":
+            sc = torch.softmax(z[t], dim=0) if scores == "all" else torch.sigmoid(z[t])
             choice = sc + (correction if correction is not None else 0.0)
+            if groups > 1:
+                runs = choice.reshape(groups, -1)
+                strength = runs.topk(min(2, runs.shape[1]), dim=1).values.sum(1)
+                best = sorted(range(groups), key=lambda g: (-float(strength[g]), g))[:keep]
+                closed = [g for g in range(groups) if g not in best]
+                runs = runs.clone()
+                runs[closed] = -math.inf
+                choice = runs.reshape(-1)
             order = sorted(range(outputs), key=lambda e: (-float(choice[e]), e))[:top]
-            w = sc[order] / (sc[order].sum() + 1e-20)
+            w = sc[order] / (sc[order].sum() + 1e-20) if renormalize else sc[order]
         else:
             order = sorted(range(outputs), key=lambda e: (-float(z[t, e]), e))[:top]
             w = torch.softmax(z[t, order], dim=0)
-        for e, we in zip(order, w):
+        for e, we in zip(order, w * route_scale):
             if e >= E:
                 out[t] += we * x[t].float()
                 continue
@@ -457,6 +504,11 @@ def moe_feed_forward(x, w_router, b_router, w_gate, w_up, w_down, top, activatio
             out[t] += we * (hid.to(x.dtype).float() @ w_down[e].float().t())
     if extra is not None:
         out += extra * gate[:, None] if gate is not None else extra
+    if beside is not None:
+        out += beside.float()
+    if residual is not None:
+        residual += out
+        return None
     return out
 
 
@@ -615,11 +667,13 @@ def rope_slice(src, src_head, src_off, dst, dst_head, dst_off, num_heads, width,
         dst[:, h * dst_head + dst_off:h * dst_head + dst_off + width] = y[:, h].to(dst.dtype)
 
 
-def head_linear(x, x_head, w, y, y_head):
+def head_linear(x, x_head, w, y, y_head, gate=None):
     H, N, K = w.shape
     for h in range(H):
-        y[:, h * y_head:h * y_head + N] = \
-            (x[:, h * x_head:h * x_head + K].float() @ w[h].float().t()).to(y.dtype)
+        v = x[:, h * x_head:h * x_head + K].float() @ w[h].float().t()
+        if gate is not None:
+            v = v * torch.sigmoid(gate[:, h * N:(h + 1) * N].float())
+        y[:, h * y_head:h * y_head + N] = v.to(y.dtype)
 
 
 def mlstm(q, k, v, gate_i, gate_f, bias_i, bias_f, cap, q_scale, out, num_seqs, num_heads, key_dim,
@@ -690,7 +744,7 @@ def attention_sink_wide_supports(num_heads, num_kv_heads, key_dim, value_dim):
     return False
 
 
-NAMES = ["act_rows", "stream_spread", "stream_read_norm", "stream_write", "qkv_conv_rope_norm_cache",
+NAMES = ["add_layernorm", "channel_scan", "act_rows", "stream_spread", "stream_read_norm", "stream_write", "qkv_conv_rope_norm_cache",
          "scaled_add_norm", "add_bias", "qk_rownorm_rope_cache", "latent_row_cache", "rope_slice",
          "head_linear", "mlstm", "mlstm_chunked", "mlstm_chunk_tokens", "mlstm_chunked_supports",
          "gated_group_norm", "qkv_bias_rope_cache", "causal_conv_act", "selective_scan",

@@ -37,6 +37,7 @@ class NormSpec:
     eps: float
     groups: int = 1                      # grouped kinds: equal consecutive parts, each normed alone
     unit_offset: bool = False            # a zero-centred weight: the gain is 1 + w
+    bias_suffix: str = ""                # kinds with a bias: its checkpoint name is the gain's + this
 
 
 @dataclass(frozen=True)
@@ -107,6 +108,14 @@ class MixerSpec:
     latent_rank: int = 0
     query_rank: int = 0
     rope_dim: int = 0
+    # latent attention kinds: the layer makes no latent of its own; it reads the rows that the
+    # call whose cache it borrows has written, `cache_row` wide (0: as wide as its own would be)
+    borrows_latent: bool = False
+    cache_row: int = 0
+    # state-space kinds with a decay per channel: channels inside the mixer, and the width that
+    # the step sizes are projected up from (head_dim is the state size)
+    inner_dim: int = 0
+    dt_rank: int = 0
     # gated recurrences: the bound c of a gate's pre-activation, c tanh(x / c)
     gate_cap: float = 0.0
     # attention kinds with a window: the first `keep_first` tokens of a request stay visible to
@@ -144,8 +153,12 @@ class FeedForwardSpec:
     # routed kinds: experts without a gate matrix (down act(up x)) when False
     gated: bool = True
     # routed kinds: "chosen": softmax over the chosen logits; "all": softmax over every logit,
-    # the chosen scores divided by their sum
+    # the chosen scores divided by their sum; "sigmoid": the logistic function of each logit
     router_scores: str = "chosen"
+    router_renormalize: bool = True      # "all", "sigmoid": the chosen scores divided by their sum
+    router_scale: float = 1.0            # the weights are multiplied by this
+    router_groups: Optional[tuple] = None    # (count, keep): the router outputs in `count` equal
+                                         # runs, of which only the best `keep` can be chosen from
     router_correction: bool = False      # a per-expert term added to the scores for the choice only
     identity_experts: int = 0            # router outputs past `experts` whose expert is the input itself
     shared_gate: bool = False            # the shared feed-forward times a logistic gate per token
@@ -198,6 +211,7 @@ class ModelSpec:
     tied_head_alias: Optional[str] = None   # name a tied checkpoint may ship anyway
     max_positions: int = 0           # advisory, as in the reference
     logit_softcap: Optional[float] = None   # c: logits <- c tanh(logits / c)
+    logit_scale: float = 1.0         # the logits are multiplied by this
     embedding_scale: float = 1.0     # the embedding rows are multiplied by this
     source: dict = field(default_factory=dict)   # the config.json it came from
 

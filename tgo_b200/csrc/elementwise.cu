@@ -211,6 +211,134 @@ TGO_API int tgo_add_rmsnorm(float* h, const void* delta, int delta_dtype, const 
     return TGO_E_BAD_ARG;
 }
 
+// ------------------------------------------------------ residual add + layer norm
+// As add_rmsnorm with the mean taken off first and a bias: x = h[r] (+ delta[r]), written back
+// to h when rows is null; m = mean x; out[i] = (x - m) * rsqrt(mean (x - m)^2 + eps) * gain +
+// bias. The squared deviations are summed from the row itself (a second pass over registers,
+// or over memory), not as mean x^2 - m^2. One block per row.
+template <typename TD, typename TO>
+__global__ void add_layernorm_kernel(float* __restrict__ h, const TD* __restrict__ delta,
+                                     const float* __restrict__ gain, const float* __restrict__ bias,
+                                     float eps, TO* __restrict__ out, const int* __restrict__ rows, int d) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    pdl_launch();
+    const int i = blockIdx.x;
+    const int r = rows ? rows[i] : i;
+    float* hr = h + (size_t)r * d;
+    const TD* dr = delta ? delta + (size_t)r * d : nullptr;
+    TO* o = out + (size_t)i * d;
+    float sum = 0.f;
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        float v = hr[j];
+        if (dr) v += to_f32(dr[j]);
+        if (dr && !rows) hr[j] = v;                      // later passes read what this thread wrote
+        sum += v;
+    }
+    const bool again = dr && rows;                       // the sum is in no memory: add once more
+    const float mean = block_sum(sum, scratch) / (float)d;
+    float ss = 0.f;
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        const float v = hr[j] + (again ? to_f32(dr[j]) : 0.f) - mean;
+        ss += v * v;
+    }
+    const float scale = rsqrtf(block_sum(ss, scratch) / (float)d + eps);
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        const float v = hr[j] + (again ? to_f32(dr[j]) : 0.f) - mean;
+        o[j] = from_f32<TO>(fmaf(v * scale, gain[j], bias[j]));
+    }
+}
+
+// Four consecutive elements per thread, the row in registers: d % 4 == 0.
+template <typename TD, typename TO, int CH4>
+__global__ void add_layernorm_vec_kernel(float* __restrict__ h, const TD* __restrict__ delta,
+                                         const float* __restrict__ gain, const float* __restrict__ bias,
+                                         float eps, TO* __restrict__ out, const int* __restrict__ rows,
+                                         int d) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    pdl_launch();
+    const int i = blockIdx.x;
+    const int r = rows ? rows[i] : i;
+    float* hr = h + (size_t)r * d;
+    const TD* dr = delta ? delta + (size_t)r * d : nullptr;
+    TO* o = out + (size_t)i * d;
+    float4 x[CH4];
+    float sum = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH4; ++c) {
+        const int j = 4 * (threadIdx.x + c * blockDim.x);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < d) {
+            v = *(const float4*)(hr + j);
+            if (dr) {
+                const float4 dl = Delta4<TD>::load(dr + j);
+                v.x += dl.x; v.y += dl.y; v.z += dl.z; v.w += dl.w;
+                if (!rows) *(float4*)(hr + j) = v;
+            }
+        }
+        x[c] = v;
+        sum += (v.x + v.y) + (v.z + v.w);
+    }
+    const float mean = block_sum(sum, scratch) / (float)d;
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH4; ++c) {
+        if (4 * (threadIdx.x + c * blockDim.x) < d) {
+            x[c].x -= mean; x[c].y -= mean; x[c].z -= mean; x[c].w -= mean;
+            ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
+        }
+    }
+    const float scale = rsqrtf(block_sum(ss, scratch) / (float)d + eps);
+#pragma unroll
+    for (int c = 0; c < CH4; ++c) {
+        const int j = 4 * (threadIdx.x + c * blockDim.x);
+        if (j < d) {
+            const float4 g = *(const float4*)(gain + j), b = *(const float4*)(bias + j);
+            Out4<TO>::store(o + j, make_float4(fmaf(x[c].x * scale, g.x, b.x), fmaf(x[c].y * scale, g.y, b.y),
+                                               fmaf(x[c].z * scale, g.z, b.z), fmaf(x[c].w * scale, g.w, b.w)));
+        }
+    }
+}
+
+template <typename TD, typename TO>
+static int add_layernorm_launch(float* h, const void* delta, const float* gain, const float* bias, float eps,
+                                void* out, const int* rows, int n, int d, cudaStream_t s) {
+    const TD* dl = (const TD*)delta;
+    TO* o = (TO*)out;
+    if (d % 4 == 0 && d <= 16384 && ((uintptr_t)h % 16 == 0) && ((uintptr_t)out % 16 == 0) &&
+        ((uintptr_t)gain % 16 == 0) && ((uintptr_t)bias % 16 == 0) && (!delta || (uintptr_t)delta % 16 == 0)) {
+        const int quads = d / 4;
+        const int vt = quads <= 256 ? 128 : quads <= 1024 ? 256 : 512;
+        const int ch = (quads + vt - 1) / vt;
+#define LN_GO(CH) tgo_launch_pdl(add_layernorm_vec_kernel<TD, TO, CH>, dim3(n), dim3(vt), 0, s, h, dl, gain, \
+                                 bias, eps, o, rows, d)
+        if (ch <= 1) return LN_GO(1);
+        if (ch <= 2) return LN_GO(2);
+        if (ch <= 4) return LN_GO(4);
+        return LN_GO(8);
+#undef LN_GO
+    }
+    return tgo_launch_pdl(add_layernorm_kernel<TD, TO>, dim3(n), dim3(d > 2048 ? 512 : 256), 0, s, h, dl, gain,
+                          bias, eps, o, rows, d);
+}
+
+TGO_API int tgo_add_layernorm(float* h, const void* delta, int delta_dtype, const float* gain,
+                              const float* bias, float eps, void* out, int out_dtype, const int* rows,
+                              int n, int d, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (d <= 0 || !gain || !bias) return TGO_E_BAD_ARG;
+    if (out_dtype == TGO_BF16 && delta && delta_dtype == TGO_BF16)
+        return add_layernorm_launch<bf16, bf16>(h, delta, gain, bias, eps, out, rows, n, d, stream);
+    if (out_dtype == TGO_BF16 && (delta_dtype == TGO_F32 || !delta))
+        return add_layernorm_launch<float, bf16>(h, delta, gain, bias, eps, out, rows, n, d, stream);
+    if (out_dtype == TGO_F32 && (delta_dtype == TGO_F32 || !delta))
+        return add_layernorm_launch<float, float>(h, delta, gain, bias, eps, out, rows, n, d, stream);
+    if (out_dtype == TGO_F32 && delta_dtype == TGO_BF16)
+        return add_layernorm_launch<bf16, float>(h, delta, gain, bias, eps, out, rows, n, d, stream);
+    return TGO_E_BAD_ARG;
+}
+
 // h[r] += delta[r] for every row, nothing else (the add a block leaves pending when
 // no norm follows it).
 template <typename TD>

@@ -125,14 +125,18 @@ TGO_API int tgo_rope_slice(const void* src, long long src_stride, int src_head, 
 // one head; a thread sums one output's k in ascending order for one or several tokens, so an
 // output's bits do not depend on what else is in the step. HL_N is 64, or 16 when that gives
 // too few blocks to fill the device (few tokens, few outputs a head). x, y: rows with unit
-// column stride.
+// column stride. With `gate` ([T, H N] in the storage type, rows gate_stride apart) every output is
+// multiplied by the logistic function of its place in it (an output gate on the heads).
+__device__ __forceinline__ float hl_gated(float v, float g) { return v / (1.f + expf(-g)); }
+
 #define HL_TOK 16
 #define HL_K 32
 
 template <typename T, int HL_N>
 __global__ void __launch_bounds__(256)
 head_linear_kernel(const T* __restrict__ x, long long x_stride, int x_head, const T* __restrict__ w,
-                   T* __restrict__ y, long long y_stride, int y_head, int Tn, int N, int K) {
+                   T* __restrict__ y, long long y_stride, int y_head, int Tn, int N, int K,
+                   const T* __restrict__ gate, long long gate_stride) {
     __shared__ float xs[HL_TOK][HL_K + 1];
     __shared__ float ws[HL_N][HL_K + 1];
     pdl_wait();
@@ -167,7 +171,10 @@ head_linear_kernel(const T* __restrict__ x, long long x_stride, int x_head, cons
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         const int t = t0 + tg + TG * i;
-        if (t < Tn) y[(size_t)t * y_stride + (size_t)h * y_head + n0 + nl] = from_f32<T>(acc[i]);
+        if (t < Tn) {
+            if (gate) acc[i] = hl_gated(acc[i], to_f32(gate[(size_t)t * gate_stride + (size_t)h * N + n0 + nl]));
+            y[(size_t)t * y_stride + (size_t)h * y_head + n0 + nl] = from_f32<T>(acc[i]);
+        }
     }
 }
 
@@ -180,7 +187,8 @@ head_linear_kernel(const T* __restrict__ x, long long x_stride, int x_head, cons
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_linear_few_kernel(const T* __restrict__ x, long long x_stride, int x_head, const T* __restrict__ w,
-                       T* __restrict__ y, long long y_stride, int y_head, int Tn, int N, int K) {
+                       T* __restrict__ y, long long y_stride, int y_head, int Tn, int N, int K,
+                       const T* __restrict__ gate, long long gate_stride) {
     pdl_wait();
     const int lane = threadIdx.x & 31;
     const int n = blockIdx.x * 8 + (threadIdx.x >> 5), h = blockIdx.y;
@@ -202,7 +210,9 @@ head_linear_few_kernel(const T* __restrict__ x, long long x_stride, int x_head, 
         }
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-            const float a = warp_sum(acc[u]);
+            float a = warp_sum(acc[u]);
+            if (lane == 0 && t0 + u < Tn && gate)
+                a = hl_gated(a, to_f32(gate[(size_t)(t0 + u) * gate_stride + (size_t)h * N + n]));
             if (lane == 0 && t0 + u < Tn) y[(size_t)(t0 + u) * y_stride + (size_t)h * y_head + n] = from_f32<T>(a);
         }
     }
@@ -210,17 +220,19 @@ head_linear_few_kernel(const T* __restrict__ x, long long x_stride, int x_head, 
 
 TGO_API int tgo_head_linear(const void* x, long long x_stride, int x_head, const void* w, void* y,
                             long long y_stride, int y_head, int dtype, int T, int H, int N, int K,
-                            cudaStream_t stream) {
+                            const void* gate, long long gate_stride, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || N <= 0 || K <= 0 || H > 65535) return TGO_E_BAD_ARG;
     if (T <= 16 && K <= 32 * HLF_PER && (N + 7) / 8 <= 0x7fffffff) {
         const dim3 fgrid((N + 7) / 8, H), fblock(256);
         if (dtype == TGO_BF16)
             return tgo_launch_pdl(head_linear_few_kernel<bf16>, fgrid, fblock, 0, stream, (const bf16*)x, x_stride,
-                                  x_head, (const bf16*)w, (bf16*)y, y_stride, y_head, T, N, K);
+                                  x_head, (const bf16*)w, (bf16*)y, y_stride, y_head, T, N, K,
+                                  (const bf16*)gate, gate_stride);
         if (dtype == TGO_F32)
             return tgo_launch_pdl(head_linear_few_kernel<float>, fgrid, fblock, 0, stream, (const float*)x,
-                                  x_stride, x_head, (const float*)w, (float*)y, y_stride, y_head, T, N, K);
+                                  x_stride, x_head, (const float*)w, (float*)y, y_stride, y_head, T, N, K,
+                                  (const float*)gate, gate_stride);
         return TGO_E_BAD_ARG;
     }
     const long long blocks64 = (long long)((T + HL_TOK - 1) / HL_TOK) * H * ((N + 63) / 64);
@@ -229,7 +241,7 @@ TGO_API int tgo_head_linear(const void* x, long long x_stride, int x_head, const
     if (grid.z > 65535) return TGO_E_BAD_ARG;
 #define HL_GO(TT, NN)                                                                                       \
     return tgo_launch_pdl(head_linear_kernel<TT, NN>, grid, block, 0, stream, (const TT*)x, x_stride, x_head, \
-                          (const TT*)w, (TT*)y, y_stride, y_head, T, N, K)
+                          (const TT*)w, (TT*)y, y_stride, y_head, T, N, K, (const TT*)gate, gate_stride)
     if (dtype == TGO_BF16) {
         if (hn == 16) HL_GO(bf16, 16);
         HL_GO(bf16, 64);
@@ -239,5 +251,67 @@ TGO_API int tgo_head_linear(const void* x, long long x_stride, int x_head, const
         HL_GO(float, 64);
     }
 #undef HL_GO
+    return TGO_E_BAD_ARG;
+}
+
+// ------------------------------------------------- a product's head-major rows, into token rows
+// y[t, h * y_head + n] = src[h][t][n] * logistic(gate[t, h * N + n]): what a batched product per
+// head leaves ([H][T][N] contiguous) put into rows, with an output gate.
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_rows_gate_kernel(const T* __restrict__ src, T* __restrict__ y, long long y_stride, int y_head, int Tn, int H,
+                      int N, const T* __restrict__ gate, long long gate_stride) {
+    pdl_wait();
+    const int t = blockIdx.x;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * N; i += gridDim.y * blockDim.x) {
+        const int h = i / N, n = i - h * N;
+        const float v = to_f32(src[((size_t)h * Tn + t) * N + n]);
+        y[(size_t)t * y_stride + (size_t)h * y_head + n] =
+            from_f32<T>(hl_gated(v, to_f32(gate[(size_t)t * gate_stride + i])));
+    }
+}
+
+// bfloat16, eight columns a thread: N, y_head and the row strides multiples of 8, 16-byte aligned.
+__global__ void __launch_bounds__(256)
+head_rows_gate_x8_kernel(const bf16* __restrict__ src, bf16* __restrict__ y, long long y_stride, int y_head, int Tn,
+                         int H, int N, const bf16* __restrict__ gate, long long gate_stride) {
+    pdl_wait();
+    const int t = blockIdx.x, n8 = N / 8;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * n8; i += gridDim.y * blockDim.x) {
+        const int h = i / n8, n = (i - h * n8) * 8;
+        const uint4 a = *(const uint4*)(src + ((size_t)h * Tn + t) * N + n);
+        const uint4 g = *(const uint4*)(gate + (size_t)t * gate_stride + (size_t)h * N + n);
+        uint4 o;
+        const uint32_t* ap = (const uint32_t*)&a;
+        const uint32_t* gp = (const uint32_t*)&g;
+        uint32_t* op = (uint32_t*)&o;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float2 av = __bfloat1622float2(*(const __nv_bfloat162*)(ap + k));
+            const float2 gv = __bfloat1622float2(*(const __nv_bfloat162*)(gp + k));
+            const __nv_bfloat162 r = __floats2bfloat162_rn(hl_gated(av.x, gv.x), hl_gated(av.y, gv.y));
+            op[k] = *(const uint32_t*)&r;
+        }
+        *(uint4*)(y + (size_t)t * y_stride + (size_t)h * y_head + n) = o;
+    }
+}
+
+TGO_API int tgo_head_rows_gate(const void* src, void* y, long long y_stride, int y_head, int dtype, int T, int H,
+                               int N, const void* gate, long long gate_stride, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || N <= 0 || !gate) return TGO_E_BAD_ARG;
+    if (dtype == TGO_BF16 && N % 8 == 0 && y_head % 8 == 0 && y_stride % 8 == 0 && gate_stride % 8 == 0 &&
+        (uintptr_t)src % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)gate % 16 == 0) {
+        const int blocks = (H * (N / 8) + 255) / 256;
+        return tgo_launch_pdl(head_rows_gate_x8_kernel, dim3(T, blocks), dim3(256), 0, stream, (const bf16*)src,
+                              (bf16*)y, y_stride, y_head, T, H, N, (const bf16*)gate, gate_stride);
+    }
+    const int cy = (H * N + 255) / 256 > 64 ? 64 : (H * N + 255) / 256;
+    if (dtype == TGO_BF16)
+        return tgo_launch_pdl(head_rows_gate_kernel<bf16>, dim3(T, cy), dim3(256), 0, stream, (const bf16*)src,
+                              (bf16*)y, y_stride, y_head, T, H, N, (const bf16*)gate, gate_stride);
+    if (dtype == TGO_F32)
+        return tgo_launch_pdl(head_rows_gate_kernel<float>, dim3(T, cy), dim3(256), 0, stream, (const float*)src,
+                              (float*)y, y_stride, y_head, T, H, N, (const float*)gate, gate_stride);
     return TGO_E_BAD_ARG;
 }

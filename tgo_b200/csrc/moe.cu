@@ -21,7 +21,11 @@
 // is by that score plus a per-expert `correction`, the weights are the chosen experts' scores
 // (without the correction) divided by their sum (+ 1e-20). The last router outputs past the
 // `E_real` experts that have matrices are identity experts: their output is the token's input
-// row itself; they get no place and no tile, the combine adds weight * x for them. One more
+// row itself; they get no place and no tile, the combine adds weight * x for them.
+// `score_mode` 2 takes the logistic function of each logit as its score; with `groups` > 1 the
+// experts are that many equal runs of neighbours, a run's strength is the sum of its two largest
+// choice scores, and only experts of the `keep` strongest runs can be chosen; without `renorm`
+// the weights are the chosen scores themselves; `route_scale` multiplies the weights. One more
 // router row after all experts (`gate_out`) gives a logistic gate per token that multiplies
 // `extra` in the combine. Experts without a gate matrix (wg null) are W_down act(W_up x);
 // activation 3 is the square of relu.
@@ -41,8 +45,10 @@ __global__ void __launch_bounds__(128)
 moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ wr,
                  const float* __restrict__ br, int Tn, int d, int E, int top, int* __restrict__ ids,
                  float* __restrict__ wts, int* __restrict__ counts, int score_mode,
-                 const float* __restrict__ correction, int E_real, float* __restrict__ gate_out) {
-    extern __shared__ float smem[];                      // [MOE_RT][E + 1] logits, [MOE_RT][E] scores
+                 const float* __restrict__ correction, int E_real, float* __restrict__ gate_out,
+                 int groups, int keep, int renorm, float route_scale) {
+    // [MOE_RT][E + 1] logits, [MOE_RT][E] scores, [MOE_RT][groups] strengths of the groups
+    extern __shared__ float smem[];
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * MOE_RT;
@@ -72,57 +78,14 @@ moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __res
     if (gate_out && lane == 0) gate_out[t] = 1.f / (1.f + expf(-lg[E]));
     float first = 0.f, sum = 0.f, mine = 0.f;
     int mine_e = 0;
-    if (score_mode == 1) {
-        // scores: the softmax over every logit; the choice adds the correction
-        float* sc = smem + (size_t)MOE_RT * ld + (size_t)warp * E;
-        float mx = -INFINITY;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
-        mx = warp_max(mx);
-        float den = 0.f;
-        for (int e = lane; e < E; e += 32) {
-            const float w = expf(lg[e] - mx);
-            sc[e] = w;
-            den += w;
-        }
-        den = warp_sum(den);
-        for (int e = lane; e < E; e += 32) {
-            const float sv = sc[e] / den;
-            sc[e] = sv;
-            lg[e] = sv + (correction ? correction[e] : 0.f);
-        }
-        __syncwarp();
-        for (int j = 0; j < top; ++j) {
-            float best = -INFINITY;
-            int be = 0x7fffffff;
-            for (int e = lane; e < E; e += 32) {
-                const float v = lg[e];
-                if (v > best || (v == best && e < be)) { best = v; be = e; }
-            }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-                if (ov > best || (ov == best && oe < be)) { best = ov; be = oe; }
-            }
-            const float w = sc[be];
-            sum += w;
-            if (lane == j) { mine = w; mine_e = be; }
-            if (lane == 0) lg[be] = -INFINITY;
-            __syncwarp();
-        }
-        if (lane < top) {
-            ids[(size_t)t * top + lane] = mine_e;
-            wts[(size_t)t * top + lane] = mine / (sum + 1e-20f);
-            if (mine_e < E_real) atomicAdd(&counts[mine_e], 1);
-        }
-        return;
-    }
-    for (int j = 0; j < top; ++j) {
-        float best = -INFINITY;
+    // the largest of n values in shared memory and its index (ties: the lower index), the same
+    // in every lane; with nothing above -inf the index is `fallback`
+    auto largest = [&](const float* v, int n, int fallback, float& best) {
+        best = -INFINITY;
         int be = 0x7fffffff;
-        for (int e = lane; e < E; e += 32) {
-            const float v = lg[e];
-            if (v > best || (v == best && e < be)) { best = v; be = e; }
+        for (int e = lane; e < n; e += 32) {
+            const float x = v[e];
+            if (x > best) { best = x; be = e; }
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -130,16 +93,94 @@ moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __res
             const int oe = __shfl_xor_sync(0xffffffffu, be, o);
             if (ov > best || (ov == best && oe < be)) { best = ov; be = oe; }
         }
+        return be < n ? be : fallback;
+    };
+    if (score_mode != 0) {
+        // scores: the softmax over every logit, or each logit's logistic; the choice adds the correction
+        float* sc = smem + (size_t)MOE_RT * ld + (size_t)warp * E;
+        float mx = 0.f, den = 1.f;
+        if (score_mode == 1) {
+            mx = -INFINITY;
+            for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
+            mx = warp_max(mx);
+            den = 0.f;
+            for (int e = lane; e < E; e += 32) {
+                const float w = expf(lg[e] - mx);
+                sc[e] = w;
+                den += w;
+            }
+            den = warp_sum(den);
+        }
+        for (int e = lane; e < E; e += 32) {
+            const float sv = score_mode == 1 ? sc[e] / den : 1.f / (1.f + expf(-lg[e]));
+            sc[e] = sv;
+            lg[e] = sv + (correction ? correction[e] : 0.f);
+        }
+        __syncwarp();
+        if (groups > 1) {
+            float* gs = smem + (size_t)MOE_RT * (ld + E) + (size_t)warp * groups;
+            const int size = E / groups;
+            for (int g = lane; g < groups; g += 32) {
+                float a = -INFINITY, c = -INFINITY;      // the two largest of the run
+                for (int e = g * size; e < (g + 1) * size; ++e) {
+                    const float v = lg[e];
+                    if (v > a) { c = a; a = v; } else if (v > c) { c = v; }
+                }
+                gs[g] = size > 1 ? a + c : a;
+            }
+            __syncwarp();
+            // the weakest groups - keep runs go: mark the strongest with +inf, then close the others
+            for (int j = 0; j < keep; ++j) {
+                float best = -INFINITY;
+                int bg = 0x7fffffff;
+                for (int g = lane; g < groups; g += 32) {
+                    const float v = gs[g];
+                    if (v < INFINITY && v > best) { best = v; bg = g; }
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+                    const int og = __shfl_xor_sync(0xffffffffu, bg, o);
+                    if (ov > best || (ov == best && og < bg)) { best = ov; bg = og; }
+                }
+                if (lane == 0 && bg < groups) gs[bg] = INFINITY;
+                __syncwarp();
+            }
+            for (int e = lane; e < E; e += 32)
+                if (gs[e / size] != INFINITY) lg[e] = -INFINITY;
+            __syncwarp();
+        }
+        for (int j = 0; j < top; ++j) {
+            float best;
+            const int be = largest(lg, E, j, best);
+            const float w = sc[be];
+            sum += w;
+            if (lane == j) { mine = w; mine_e = be; }
+            __syncwarp();                                // every lane has read lg
+            if (lane == 0) lg[be] = -INFINITY;
+            __syncwarp();
+        }
+        if (lane < top) {
+            ids[(size_t)t * top + lane] = mine_e;
+            wts[(size_t)t * top + lane] = (renorm ? mine / (sum + 1e-20f) : mine) * route_scale;
+            if (mine_e < E_real) atomicAdd(&counts[mine_e], 1);
+        }
+        return;
+    }
+    for (int j = 0; j < top; ++j) {
+        float best;
+        const int be = largest(lg, E, j, best);
         if (j == 0) first = best;
         const float w = expf(best - first);
         sum += w;
         if (lane == j) { mine = w; mine_e = be; }
+        __syncwarp();
         if (lane == 0) lg[be] = -INFINITY;
         __syncwarp();
     }
     if (lane < top) {
         ids[(size_t)t * top + lane] = mine_e;
-        wts[(size_t)t * top + lane] = mine / sum;
+        wts[(size_t)t * top + lane] = mine / sum * route_scale;
         if (mine_e < E_real) atomicAdd(&counts[mine_e], 1);
     }
 }
@@ -423,13 +464,16 @@ moe_tc_kernel(const bf16* __restrict__ a, long long a_stride, const bf16* __rest
 
 // out[t][c] = sum_j wts[t][j] y[t top + j][c] + extra_gate[t] * extra[t][c]; a pair whose
 // expert is an identity expert (ids >= E_real; `ids` null: there are none) contributes
-// wts * x[t][c] instead.
-template <typename T>
+// wts * x[t][c] instead. `beside` [T, d] (TB: float32 or bfloat16; null: none) is added too, and
+// with `accumulate` the whole is added to out: a block whose mixer and feed-forward read the
+// same rows has both results put into the stream by this one pass.
+template <typename T, typename TB>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ wts,
                                    const float* __restrict__ extra, float* __restrict__ out, int d,
                                    int top, const int* __restrict__ ids, int E_real,
                                    const T* __restrict__ x, long long x_stride,
-                                   const float* __restrict__ extra_gate) {
+                                   const float* __restrict__ extra_gate,
+                                   const TB* __restrict__ beside, int accumulate) {
     pdl_wait();
     const int t = blockIdx.x;
     const float eg = extra_gate ? extra_gate[t] : 1.f;
@@ -441,6 +485,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
             a = fmaf(wts[pair], v, a);
         }
         if (extra) a = fmaf(eg, extra[(size_t)t * d + c], a);
+        if (beside) a += to_f32(beside[(size_t)t * d + c]);
+        if (accumulate) a += out[(size_t)t * d + c];
         out[(size_t)t * d + c] = a;
     }
 }
@@ -453,24 +499,28 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
                           const float* br, int T, int d, int E, int top, int* ids, float* wts,
                           int* counts, int* fill, int* offsets, int* perm, int* place,
                           int* tile_info, int* tiles, int max_tiles, int score_mode,
-                          const float* correction, int E_real, float* gate_out, cudaStream_t stream) {
+                          const float* correction, int E_real, float* gate_out, int groups, int keep,
+                          int renorm, float route_scale, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0 || E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || max_tiles <= 0 ||
-        E_real < 0 || E_real > E || score_mode < 0 || score_mode > 1)
+        E_real < 0 || E_real > E || score_mode < 0 || score_mode > 2 || groups < 1 || E % groups ||
+        keep < 1 || keep > groups || (long long)keep * (E / groups) < top || (groups > 1 && score_mode == 0))
         return TGO_E_BAD_ARG;
     int rc = E_real ? (int)cudaMemsetAsync(counts, 0, sizeof(int) * E_real, stream) : 0;
     if (rc) return rc;
-    const size_t smem = (size_t)MOE_RT * (2 * E + 1) * sizeof(float);
-    if (smem > 48 * 1024) {                              // more than about 1500 router outputs
+    const size_t smem = (size_t)MOE_RT * (2 * E + 1 + groups) * sizeof(float);
+    if (smem > 48 * 1024) {                              // more than about 1000 router outputs
         cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     }
     if (dtype == TGO_BF16)
         moe_route_kernel<bf16><<<(T + MOE_RT - 1) / MOE_RT, 128, smem, stream>>>((const bf16*)x, x_stride, wr, br, T, d, E,
-                                                                  top, ids, wts, counts, score_mode, correction, E_real, gate_out);
+                                                                  top, ids, wts, counts, score_mode, correction, E_real, gate_out,
+                                                                  groups, keep, renorm, route_scale);
     else if (dtype == TGO_F32)
         moe_route_kernel<float><<<(T + MOE_RT - 1) / MOE_RT, 128, smem, stream>>>((const float*)x, x_stride, wr, br, T, d,
-                                                                   E, top, ids, wts, counts, score_mode, correction, E_real, gate_out);
+                                                                   E, top, ids, wts, counts, score_mode, correction, E_real, gate_out,
+                                                                  groups, keep, renorm, route_scale);
     else
         return TGO_E_BAD_ARG;
     if ((rc = launch_status())) return rc;
@@ -489,13 +539,16 @@ TGO_API int tgo_moe_experts(const void* x, long long x_stride, int dtype, const 
                             const float* wts, const float* extra, float* out, int T, int d, int ff,
                             int top, int act, const int* perm, const int* tile_info,
                             const int* tiles, int max_tiles, const int* ids, int E_real,
-                            const float* extra_gate, cudaStream_t stream) {
+                            const float* extra_gate, const void* beside, int beside_dtype,
+                            int accumulate, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0 || ff <= 0 || top <= 0 || max_tiles <= 0 || max_tiles > 65535 || act < 0 || act > 3)
         return TGO_E_BAD_ARG;
-#define MOE_COMBINE(TT)                                                                            \
-    tgo_launch_pdl(moe_combine_kernel<TT>, dim3(T), dim3(256), 0, stream, (const float*)y, wts, extra, out, \
-                   d, top, ids, E_real, (const TT*)x, x_stride, extra_gate)
+    if (beside && beside_dtype != TGO_F32 && beside_dtype != TGO_BF16) return TGO_E_BAD_ARG;
+#define MOE_COMBINE_OF(TT, TB)                                                                             \
+    tgo_launch_pdl(moe_combine_kernel<TT, TB>, dim3(T), dim3(256), 0, stream, (const float*)y, wts, extra, out, \
+                   d, top, ids, E_real, (const TT*)x, x_stride, extra_gate, (const TB*)beside, accumulate)
+#define MOE_COMBINE(TT) (beside && beside_dtype == TGO_BF16 ? MOE_COMBINE_OF(TT, bf16) : MOE_COMBINE_OF(TT, float))
     const dim3 g1((ff + MOE_TN - 1) / MOE_TN, max_tiles), g2((d + MOE_TN - 1) / MOE_TN, max_tiles);
     int rc;
     const bool chunks = d % 8 == 0 && ff % 8 == 0 && x_stride % 8 == 0 && (uintptr_t)x % 16 == 0 &&
@@ -545,4 +598,5 @@ TGO_API int tgo_moe_experts(const void* x, long long x_stride, int dtype, const 
     if (rc) return rc;
     return MOE_COMBINE(float);
 #undef MOE_COMBINE
+#undef MOE_COMBINE_OF
 }

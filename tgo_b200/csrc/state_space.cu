@@ -9,19 +9,27 @@
 // reads B and C of group floor(h / (H / G)). Everything after the convolution's input is
 // float32 whatever the storage type of the projections.
 //
+// A second scan (the form known as Mamba-1) has a decay of its own for every channel and state,
+// and B and C shared by all channels:
+//
+//   dt_t    = softplus(raw_t + dt_bias)                     per channel c
+//   S[c, n] = exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n       S is [channels, N], float32
+//   y_c     = (sum_n S[c, n] C_n + D_c x_c) * silu(z_c)
+//
 // A request's state row (float32, `state_stride` floats apart) holds the scan's state
-// [H][N][P] at `ssm_offset` and the convolution's last taps - 1 inputs [taps - 1][C] (oldest
+// [H][N][P] (or [channels][N]) at `ssm_offset` and the convolution's last taps - 1 inputs [taps - 1][C] (oldest
 // first) at `conv_offset`.
 #include "common.cuh"
 
 // ------------------------------------------------------------------------- convolution
 // y[t][c] = silu(bias[c] + sum_j w[c][j] x[t - (taps - 1 - j)][c]); inputs before the step's
 // first token come from the request's kept inputs, zeros before the request's start (a fresh
-// state row is zero). x is a column view [T, C] in the storage type; y float32 [T, C].
-template <typename T>
+// state row is zero). x is a column view [T, C] in the storage type; y [T, C] float32 or in the
+// storage type (TY).
+template <typename T, typename TY>
 __global__ void __launch_bounds__(256)
 causal_conv_act_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ w,
-                       const float* __restrict__ bias, float* __restrict__ y, int C, int taps,
+                       const float* __restrict__ bias, TY* __restrict__ y, int C, int taps,
                        const int* __restrict__ seq_ids, const int* __restrict__ q_start,
                        const int* __restrict__ state_slots, const float* __restrict__ state,
                        long long state_stride, long long conv_offset) {
@@ -39,7 +47,7 @@ causal_conv_act_kernel(const T* __restrict__ x, long long x_stride, const float*
             else v = kept[(size_t)(taps - 1 - (back - r)) * C + c];
             a = fmaf(w[(size_t)c * taps + j], v, a);
         }
-        y[(size_t)t * C + c] = a / (1.f + expf(-a));
+        y[(size_t)t * C + c] = from_f32<TY>(a / (1.f + expf(-a)));
     }
 }
 
@@ -66,27 +74,28 @@ causal_conv_keep_kernel(const T* __restrict__ x, long long x_stride, int C, int 
     }
 }
 
+// y_dtype: float32, or the storage type. `keep` 0 leaves the kept inputs where they are (the
+// channel scan below moves them on itself).
 TGO_API int tgo_causal_conv_act(const void* x, long long x_stride, int dtype, const float* w,
-                                const float* bias, float* y, int T, int B, int C, int taps,
+                                const float* bias, void* y, int y_dtype, int T, int B, int C, int taps,
                                 const int* seq_ids, const int* q_start, const int* state_slots,
-                                float* state, long long state_stride, long long conv_offset,
+                                float* state, long long state_stride, long long conv_offset, int keep,
                                 cudaStream_t stream) {
     if (T <= 0 || B <= 0) return 0;
     if (C <= 0 || taps <= 0 || taps > 64 || state_stride < conv_offset + (long long)(taps - 1) * C)
         return TGO_E_BAD_ARG;
     const int cy = (C + 255) / 256 > 64 ? 64 : (C + 255) / 256;
     int rc;
-    if (dtype == TGO_BF16)
-        rc = tgo_launch_pdl(causal_conv_act_kernel<bf16>, dim3(T, cy), dim3(256), 0, stream, (const bf16*)x,
-                            x_stride, w, bias, y, C, taps, seq_ids, q_start, state_slots,
-                            (const float*)state, state_stride, conv_offset);
-    else if (dtype == TGO_F32)
-        rc = tgo_launch_pdl(causal_conv_act_kernel<float>, dim3(T, cy), dim3(256), 0, stream, (const float*)x,
-                            x_stride, w, bias, y, C, taps, seq_ids, q_start, state_slots,
-                            (const float*)state, state_stride, conv_offset);
-    else
-        return TGO_E_BAD_ARG;
-    if (rc || taps == 1) return rc;
+#define CONV_GO(TT, TY)                                                                                    \
+    tgo_launch_pdl(causal_conv_act_kernel<TT, TY>, dim3(T, cy), dim3(256), 0, stream, (const TT*)x, x_stride, w, \
+                   bias, (TY*)y, C, taps, seq_ids, q_start, state_slots, (const float*)state, state_stride, \
+                   conv_offset)
+    if (dtype == TGO_BF16 && y_dtype == TGO_F32) rc = CONV_GO(bf16, float);
+    else if (dtype == TGO_BF16 && y_dtype == TGO_BF16) rc = CONV_GO(bf16, bf16);
+    else if (dtype == TGO_F32 && y_dtype == TGO_F32) rc = CONV_GO(float, float);
+    else return TGO_E_BAD_ARG;
+#undef CONV_GO
+    if (rc || taps == 1 || !keep) return rc;
     if (dtype == TGO_BF16)
         return tgo_launch_pdl(causal_conv_keep_kernel<bf16>, dim3(B, cy), dim3(256), 0, stream, (const bf16*)x,
                               x_stride, C, taps, q_start, state_slots, state, state_stride, conv_offset);
@@ -277,4 +286,209 @@ TGO_API int tgo_selective_scan(const float* xbc, int C, const void* dt_raw, long
         return scan_by_size<float>(xbc, C, (const float*)dt_raw, dt_stride, dt_bias, A_log, D, y, B, H, G, N,
                                    P, q_start, state_slots, state, state_stride, ssm_offset, stream);
     return TGO_E_BAD_ARG;
+}
+
+// ---------------------------------------------------------------------- scan per channel
+// A block per (request, CS_CH channels): L lanes share a channel and lane l keeps states
+// l * NS .. l * NS + NS - 1 of it in registers for the whole walk over the request's tokens,
+// CS_TOK at a time. A tile's inputs (x, raw dt, z, B, C) are loaded into registers while the
+// tile before it is walked, dt goes through softplus once per (token, channel) and lies in
+// shared memory beside dt * x, B and C as float32 rows. Four tokens are taken together: their
+// decays do not depend on the state, so only one FMA per state and token is a chain, and the
+// four sums over n are joined by a transposing exchange in the quad (three shuffles for four
+// tokens) and, for L > 4, by shuffles over the quads, the same order for every token. Tokens
+// past the end of a tile have dt = 0 and leave the state as it is. The thread that loaded a
+// (token, channel) pair adds D x, multiplies by silu(z) and stores. `a2` is A log2(e).
+//
+// The walk ends with the convolution's kept inputs: the last taps - 1 of (kept, then the
+// step's raw inputs `conv_in`), which the convolution has read before this kernel starts.
+#define CS_TOK 32
+#define CS_THREADS 128
+
+template <typename T, int L, int NS>
+__global__ void __launch_bounds__(CS_THREADS)
+channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ z, long long z_stride,
+                    const float* __restrict__ dt_raw, long long dt_stride, const float* __restrict__ dt_bias,
+                    const float* __restrict__ a2, const T* __restrict__ bm, const T* __restrict__ cm,
+                    long long bc_stride, const float* __restrict__ D, T* __restrict__ y, int C, int N,
+                    const int* __restrict__ q_start, const int* __restrict__ state_slots,
+                    float* __restrict__ state, long long state_stride, long long ssm_offset,
+                    const T* __restrict__ conv_in, long long conv_in_stride, int taps, long long conv_offset) {
+    constexpr int CH = CS_THREADS / L;                   // channels of this block
+    constexpr int NP = L * NS;                           // N rounded up
+    constexpr int PER = CS_TOK * CH / CS_THREADS;        // (token, channel) pairs a thread loads
+    constexpr int RSTEP = CS_THREADS / CH;               // tokens between a thread's pairs (= L)
+    constexpr int PBC = (CS_TOK * NP + CS_THREADS - 1) / CS_THREADS;
+    extern __shared__ __align__(16) float cs_smem[];
+    float* s_b = cs_smem;                                // [CS_TOK][NP]
+    float* s_c = s_b + CS_TOK * NP;                      // [CS_TOK][NP]
+    float2* s_dt = (float2*)(s_c + CS_TOK * NP);         // [CS_TOK][CH + 1]: dt, dt x
+    float* s_y = (float*)(s_dt + CS_TOK * (CH + 1));     // [CS_TOK][CH + 1]
+    pdl_wait();
+    const int b = blockIdx.x, c0 = blockIdx.y * CH;
+    const int t0 = q_start[b], n_tok = q_start[b + 1] - t0;
+    const int tid = threadIdx.x;
+    float* row = state + (size_t)state_slots[b] * state_stride;
+    // the walking role: channel wc, states from n0
+    const int lane_l = tid % L, wc = c0 + tid / L, n0 = lane_l * NS;
+    const bool live = wc < C;
+    float S[NS], A[NS];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+        const bool ok = live && n0 + i < N;
+        S[i] = ok ? row[ssm_offset + (size_t)wc * N + n0 + i] : 0.f;
+        A[i] = ok ? a2[(size_t)wc * N + n0 + i] : 0.f;
+    }
+    // the loading role: channel lc, tokens lt + RSTEP k
+    const int lcl = tid % CH, lc = c0 + lcl, lt = tid / CH;
+    const bool lok = lc < C;
+    const float bias = (lok && dt_bias) ? dt_bias[lc] : 0.f;
+    const float skip = (lok && D) ? D[lc] : 0.f;
+    float xn[PER], zn[PER], dn[PER];
+    float bn[PBC], cn[PBC];
+    auto fetch = [&](int base) {
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int r = base + lt + RSTEP * k;
+            const bool ok = lok && r < n_tok;
+            const size_t t = (size_t)(t0 + r);
+            xn[k] = ok ? to_f32(x[t * x_stride + lc]) : 0.f;
+            zn[k] = ok ? to_f32(z[t * z_stride + lc]) : 0.f;
+            dn[k] = ok ? dt_raw[t * dt_stride + lc] : 0.f;
+        }
+#pragma unroll
+        for (int k = 0; k < PBC; ++k) {
+            const int i = tid + CS_THREADS * k;
+            const int r = base + i / NP, n = i % NP;
+            const bool ok = i < CS_TOK * NP && n < N && r < n_tok;
+            bn[k] = ok ? to_f32(bm[(size_t)(t0 + r) * bc_stride + n]) : 0.f;
+            cn[k] = ok ? to_f32(cm[(size_t)(t0 + r) * bc_stride + n]) : 0.f;
+        }
+    };
+    fetch(0);
+    for (int base = 0; base < n_tok; base += CS_TOK) {
+        const int nt = n_tok - base < CS_TOK ? n_tok - base : CS_TOK;
+        float xc[PER], zc[PER];
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int r = lt + RSTEP * k;
+            const float v = dn[k] + bias;
+            const float dt = r < nt ? (v > 20.f ? v : log1pf(expf(v))) : 0.f;
+            s_dt[r * (CH + 1) + lcl] = make_float2(dt, dt * xn[k]);
+            xc[k] = xn[k];
+            zc[k] = zn[k];
+        }
+#pragma unroll
+        for (int k = 0; k < PBC; ++k) {
+            const int i = tid + CS_THREADS * k;
+            if (i < CS_TOK * NP) { s_b[i] = bn[k]; s_c[i] = cn[k]; }
+        }
+        __syncthreads();
+        if (base + CS_TOK < n_tok) fetch(base + CS_TOK);
+        for (int r = 0; r < nt; r += 4) {
+            float part[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const float2 dd = s_dt[(r + u) * (CH + 1) + tid / L];
+                const float* br = s_b + (r + u) * NP + n0;
+                const float* cr = s_c + (r + u) * NP + n0;
+                float p = 0.f;
+#pragma unroll
+                for (int i = 0; i < NS; i += 4) {
+                    const float4 bq = *(const float4*)(br + i), cq = *(const float4*)(cr + i);
+                    S[i] = fmaf(exp2f(dd.x * A[i]), S[i], dd.y * bq.x);
+                    S[i + 1] = fmaf(exp2f(dd.x * A[i + 1]), S[i + 1], dd.y * bq.y);
+                    S[i + 2] = fmaf(exp2f(dd.x * A[i + 2]), S[i + 2], dd.y * bq.z);
+                    S[i + 3] = fmaf(exp2f(dd.x * A[i + 3]), S[i + 3], dd.y * bq.w);
+                    p = fmaf(S[i], cq.x, p);
+                    p = fmaf(S[i + 1], cq.y, p);
+                    p = fmaf(S[i + 2], cq.z, p);
+                    p = fmaf(S[i + 3], cq.w, p);
+                }
+                part[u] = p;
+            }
+            // four sums over the quad, transposed: lane q of a quad ends with token r + q
+            const bool odd = tid & 1, high = tid & 2;
+            const float s0 = odd ? part[0] : part[1], s1 = odd ? part[2] : part[3];
+            float k0 = odd ? part[1] : part[0], k1 = odd ? part[3] : part[2];
+            k0 += __shfl_xor_sync(0xffffffffu, s0, 1);
+            k1 += __shfl_xor_sync(0xffffffffu, s1, 1);
+            const float s2 = high ? k0 : k1;
+            float sum = high ? k1 : k0;
+            sum += __shfl_xor_sync(0xffffffffu, s2, 2);
+#pragma unroll
+            for (int o = 4; o < L; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            if (lane_l < 4) s_y[(r + (tid & 3)) * (CH + 1) + tid / L] = sum;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int r = lt + RSTEP * k;
+            if (lok && r < nt) {
+                const float v = fmaf(skip, xc[k], s_y[r * (CH + 1) + lcl]);
+                y[(size_t)(t0 + base + r) * C + lc] = from_f32<T>(v * (zc[k] / (1.f + expf(-zc[k]))));
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NS; ++i)
+        if (live && n0 + i < N) row[ssm_offset + (size_t)wc * N + n0 + i] = S[i];
+    if (conv_in && tid < CH && c0 + tid < C) {
+        const int c = c0 + tid, keep = taps - 1;
+        float* kept = row + conv_offset;
+        // ascending i reads kept[n_tok + i] before any later write could reach it
+        for (int i = 0; i < keep; ++i) {
+            const int at = n_tok + i;                    // place in (kept, then new)
+            kept[(size_t)i * C + c] = at < keep ? kept[(size_t)at * C + c]
+                                                : to_f32(conv_in[(size_t)(t0 + at - keep) * conv_in_stride + c]);
+        }
+    }
+}
+
+template <typename T, int L, int NS>
+static int launch_channel_scan(const void* x, long long x_stride, const void* z, long long z_stride,
+                               const float* dt_raw, long long dt_stride, const float* dt_bias, const float* a2,
+                               const void* bm, const void* cm, long long bc_stride, const float* D, void* y, int B,
+                               int C, int N, const int* q_start, const int* state_slots, float* state,
+                               long long state_stride, long long ssm_offset, const void* conv_in,
+                               long long conv_in_stride, int taps, long long conv_offset, cudaStream_t stream) {
+    constexpr int CH = CS_THREADS / L, NP = L * NS;
+    const size_t smem = (size_t)CS_TOK * (2 * NP + 3 * (CH + 1)) * sizeof(float);
+    auto kernel = channel_scan_kernel<T, L, NS>;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return tgo_launch_pdl(kernel, dim3(B, (C + CH - 1) / CH), dim3(CS_THREADS), smem, stream, (const T*)x, x_stride,
+                          (const T*)z, z_stride, dt_raw, dt_stride, dt_bias, a2, (const T*)bm, (const T*)cm,
+                          bc_stride, D, (T*)y, C, N, q_start, state_slots, state, state_stride, ssm_offset,
+                          (const T*)conv_in, conv_in_stride, taps, conv_offset);
+}
+
+// x, z column views [T, C], bm, cm column views [T, N] (row stride bc_stride) and conv_in a
+// column view [T, C] (null: no kept inputs to move on), all in the storage type; dt_raw float32
+// [T, C] (strided); a2 float32 [C, N]; y [T, C] in the storage type. A request's state [C][N] lies
+// at `ssm_offset` of its state row, its kept inputs [taps - 1][C] at `conv_offset`.
+TGO_API int tgo_channel_scan(const void* x, long long x_stride, const void* z, long long z_stride, int dtype,
+                             const float* dt_raw, long long dt_stride, const float* dt_bias, const float* a2,
+                             const void* bm, const void* cm, long long bc_stride, const float* D, void* y, int B,
+                             int C, int N, const int* q_start, const int* state_slots, float* state,
+                             long long state_stride, long long ssm_offset, const void* conv_in,
+                             long long conv_in_stride, int taps, long long conv_offset, cudaStream_t stream) {
+    if (B <= 0) return 0;
+    if (C <= 0 || N <= 0 || N > 256 || (dtype != TGO_BF16 && dtype != TGO_F32) ||
+        state_stride < ssm_offset + (long long)C * N || (C + 3) / 4 > 65535 ||
+        (conv_in && (taps < 1 || state_stride < conv_offset + (long long)(taps - 1) * C)))
+        return TGO_E_BAD_ARG;
+#define CS_GO(L, NS)                                                                                          \
+    (dtype == TGO_BF16                                                                                        \
+         ? launch_channel_scan<bf16, L, NS>(x, x_stride, z, z_stride, dt_raw, dt_stride, dt_bias, a2, bm, cm,  \
+                                            bc_stride, D, y, B, C, N, q_start, state_slots, state, state_stride, \
+                                            ssm_offset, conv_in, conv_in_stride, taps, conv_offset, stream)   \
+         : launch_channel_scan<float, L, NS>(x, x_stride, z, z_stride, dt_raw, dt_stride, dt_bias, a2, bm, cm, \
+                                             bc_stride, D, y, B, C, N, q_start, state_slots, state, state_stride, \
+                                             ssm_offset, conv_in, conv_in_stride, taps, conv_offset, stream))
+    if (N <= 16) return CS_GO(4, 4);
+    if (N <= 32) return CS_GO(4, 8);
+    if (N <= 64) return CS_GO(8, 8);
+    if (N <= 128) return CS_GO(16, 8);
+    return CS_GO(32, 8);
+#undef CS_GO
 }

@@ -32,6 +32,9 @@ class Model:
                        for ls in spec.layers]
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm, spec.hidden_size,
                                                           spec.final_norm_name)
+        if spec.logit_scale != 1.0 and not hasattr(self.final_norm, "fold_scale"):
+            raise ValueError(f"model: the final norm {spec.final_norm.kind!r} takes no factor for the "
+                             "logits (no fold_scale)")
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
         self._layout()
@@ -42,7 +45,7 @@ class Model:
         out = [WeightSpec(s.embedding_name, (s.vocab_size, s.hidden_size), "table")]
         for b in self.blocks:
             out += b.weight_specs()
-        out.append(WeightSpec(s.final_norm_name, (s.hidden_size,), "gain"))
+        out += self.final_norm.weight_specs()
         if s.head_name is not None:
             out.append(WeightSpec(s.head_name, (s.vocab_size, s.hidden_size), "matrix"))
         return out
@@ -60,6 +63,8 @@ class Model:
         for b in self.blocks:
             b.bind(weights)
         self.final_norm.bind(weights)
+        if s.logit_scale != 1.0:
+            self.final_norm.fold_scale(float(s.logit_scale))
 
     def weight_bytes(self) -> int:
         """Bytes of every matrix a decode step reads once (the embedding table is read by
@@ -81,11 +86,19 @@ class Model:
 
     # --------------------------------------------------------------------- cache
     def _layout(self) -> None:
-        """Group the cache-owning calls by what they need."""
+        """Group the cache-owning calls by what they need: a call whose cache later calls borrow
+        keeps what the farthest-reading of them needs."""
         self.groups: List[GroupLayout] = []
         self.call_group: Dict[int, int] = {}
         self.state_shapes: Dict[int, tuple] = {}
         by_key = {}
+        readers: Dict[int, list] = {}            # owning call -> the needs of the calls that borrow it
+        for call in self.spec.run_order:
+            mixer = self.blocks[call.layer].mixer
+            if call.cache_from is not None and hasattr(mixer, "cache_need"):
+                need = mixer.cache_need()
+                if need is not None:
+                    readers.setdefault(call.cache_from, []).append(need)
         for ci, call in enumerate(self.spec.run_order):
             if call.cache_from is not None:
                 continue
@@ -94,11 +107,18 @@ class Model:
             if need is not None:
                 shapes = getattr(need, "plane_shapes", None)
                 keep = int(getattr(need, "keep_first", 0) or 0)
-                key = (need.kind, need.window, need.planes, tuple(need.row_shape), shapes, keep)
+                kind, window = need.kind, need.window
+                for other in readers.get(ci, []):
+                    keep = max(keep, int(getattr(other, "keep_first", 0) or 0))
+                    if kind == "full" or other.kind == "full":
+                        kind, window, keep = "full", None, 0
+                    else:
+                        window = max(window, other.window)
+                key = (kind, window, need.planes, tuple(need.row_shape), shapes, keep)
                 if key not in by_key:
                     by_key[key] = len(self.groups)
-                    self.groups.append(GroupLayout(need.kind, need.window, need.planes,
-                                                   need.row_shape, [], shapes, keep))
+                    self.groups.append(GroupLayout(kind, window, need.planes, need.row_shape, [], shapes,
+                                                   keep))
                 self.groups[by_key[key]].calls.append(ci)
                 self.call_group[ci] = by_key[key]
             st = mixer.state_need() if hasattr(mixer, "state_need") else None

@@ -89,6 +89,30 @@ def add_rmsnorm(h: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tens
                                _ptr(rows), c_int(n), c_int(d), _stream()), "add_rmsnorm")
 
 
+def add_layernorm(h: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tensor,
+                  bias: torch.Tensor, eps: float, out: torch.Tensor,
+                  rows: Optional[torch.Tensor] = None) -> None:
+    """`add_rmsnorm` with the mean taken off each row first and a bias added last: out =
+    (x - mean x) / sqrt(mean (x - mean x)^2 + eps) * gain + bias, x = h (+ delta)."""
+    _need_cuda(h, delta, gain, bias, out, rows)
+    n, d = out.shape
+    assert h.dtype == gain.dtype == bias.dtype == torch.float32 and h.is_contiguous()
+    assert gain.numel() == d and bias.numel() == d and out.is_contiguous() and h.shape[1] == d
+    assert gain.is_contiguous() and bias.is_contiguous()
+    if delta is not None:
+        assert delta.shape == h.shape and delta.is_contiguous()
+    if rows is not None:
+        assert rows.dtype == torch.int32 and rows.numel() == n
+    else:
+        assert h.shape[0] == n
+    lib = load_library("elementwise")
+    _check(lib.tgo_add_layernorm(_ptr(h), _ptr(delta),
+                                 c_int(dtype_code(delta.dtype) if delta is not None else 0),
+                                 _ptr(gain), _ptr(bias), c_float(eps), _ptr(out),
+                                 c_int(dtype_code(out.dtype)), _ptr(rows), c_int(n), c_int(d),
+                                 _stream()), "add_layernorm")
+
+
 def residual_add(h: torch.Tensor, delta: torch.Tensor) -> None:
     """h += delta, h float32."""
     _need_cuda(h, delta)
@@ -835,54 +859,67 @@ HEAD_LINEAR_LIBRARY_ROWS = 65     # bfloat16 steps of this many rows or more: th
                                   # batched product
 
 
-def head_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, y: torch.Tensor, y_head: int) -> None:
+def head_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, y: torch.Tensor, y_head: int,
+                gate: Optional[torch.Tensor] = None) -> None:
     """A product per head: y[t, h * y_head + n] = sum_k x[t, h * x_head + k] w[h, n, k], with
-    w [H, N, K]; x and y 2-D views with unit column stride. float32, and bfloat16 with few
+    w [H, N, K]; x and y 2-D views with unit column stride. With `gate` (a 2-D view [T, H N] in
+    x's type) every output is multiplied by the logistic function of gate[t, h * N + n].
+    float32, and bfloat16 with few
     rows: this package's kernels (up to 16 rows and K up to 512: a warp an output, the lanes'
     partial sums joined in a fixed order; else tiles, k summed in order); bfloat16 with many
     rows: the library's batched product, where the dense products of as many rows take the
     library too."""
-    _need_cuda(x, w, y)
+    _need_cuda(x, w, y, gate)
     T = x.shape[0]
     H, N, K = w.shape
+    assert gate is None or (gate.shape == (T, H * N) and gate.stride(1) == 1 and gate.dtype == x.dtype)
     assert w.is_contiguous() and x.stride(1) == 1 and y.stride(1) == 1
     assert x.dtype == w.dtype == y.dtype and y.shape[0] == T
     if x.dtype == torch.bfloat16 and T >= HEAD_LINEAR_LIBRARY_ROWS:
         xv = torch.as_strided(x, (H, T, K), (x_head, x.stride(0), 1))
+        if gate is not None:
+            lib = load_library("latent")
+            by_head = torch.bmm(xv, w.transpose(1, 2))
+            _check(lib.tgo_head_rows_gate(_ptr(by_head), _ptr(y), c_ll(y.stride(0)), c_int(y_head),
+                                          c_int(dtype_code(y.dtype)), c_int(T), c_int(H), c_int(N),
+                                          _ptr(gate), c_ll(gate.stride(0)), _stream()), "head_rows_gate")
+            return
         yv = torch.as_strided(y, (H, T, N), (y_head, y.stride(0), 1))
         yv.copy_(torch.bmm(xv, w.transpose(1, 2)))
         return
     lib = load_library("latent")
     _check(lib.tgo_head_linear(_ptr(x), c_ll(x.stride(0)), c_int(x_head), _ptr(w), _ptr(y),
                                c_ll(y.stride(0)), c_int(y_head), c_int(dtype_code(x.dtype)), c_int(T),
-                               c_int(H), c_int(N), c_int(K), _stream()), "head_linear",
+                               c_int(H), c_int(N), c_int(K), _ptr(gate),
+                               c_ll(gate.stride(0) if gate is not None else 0), _stream()), "head_linear",
            f"(H={H}, N={N}, K={K})")
 
 
 def causal_conv_act(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], y: torch.Tensor,
                     num_seqs: int, seq_ids: torch.Tensor, q_start: torch.Tensor,
-                    state_slots: torch.Tensor, state: torch.Tensor, conv_offset: int) -> None:
+                    state_slots: torch.Tensor, state: torch.Tensor, conv_offset: int,
+                    keep: bool = True) -> None:
     """y = silu(bias + causal convolution of x per channel): x a 2-D view [T, C] in the
-    activation type, w float32 [C, taps] (the last column meets the current token), y float32
-    [T, C]. The inputs before a request's portion come from its state row (float32
+    activation type, w float32 [C, taps] (the last column meets the current token), y [T, C]
+    float32 or in the activation type. The inputs before a request's portion come from its state row (float32
     [slots, n]; the last taps - 1 inputs [taps - 1, C] at `conv_offset`), which is then moved
-    on by the step's inputs."""
+    on by the step's inputs, unless `keep` is False (`channel_scan` moves them on)."""
     _need_cuda(x, w, bias, y, seq_ids, q_start, state_slots, state)
     T, C = x.shape
     taps = w.shape[1]
     assert x.stride(1) == 1 and w.dtype == torch.float32 and w.is_contiguous() and w.shape[0] == C
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == C)
-    assert y.dtype == torch.float32 and y.is_contiguous() and y.shape == (T, C)
+    assert y.dtype in (torch.float32, x.dtype) and y.is_contiguous() and y.shape == (T, C)
     assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
     assert seq_ids.dtype == q_start.dtype == state_slots.dtype == torch.int32
     assert q_start.numel() == num_seqs + 1 and state_slots.numel() == num_seqs
     lib = load_library("state_space")
     _check(lib.tgo_causal_conv_act(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w), _ptr(bias), _ptr(y),
-        c_int(T), c_int(num_seqs), c_int(C), c_int(taps), _ptr(seq_ids), _ptr(q_start),
-        _ptr(state_slots), _ptr(state), c_ll(state.stride(0)), c_ll(conv_offset), _stream()),
-        "causal_conv_act", f"(C={C}, taps={taps})")
-    if taps > 1:
+        c_int(dtype_code(y.dtype)), c_int(T), c_int(num_seqs), c_int(C), c_int(taps), _ptr(seq_ids), _ptr(q_start),
+        _ptr(state_slots), _ptr(state), c_ll(state.stride(0)), c_ll(conv_offset),
+        c_int(1 if keep else 0), _stream()), "causal_conv_act", f"(C={C}, taps={taps})")
+    if taps > 1 and keep:
         LAUNCHES[0] += 1
 
 
@@ -915,6 +952,46 @@ def selective_scan(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: Optional[to
         f"(heads={heads}, groups={groups}, state={state_dim}, vdim={value_dim})")
 
 
+def channel_scan(x: torch.Tensor, z: torch.Tensor, dt_raw: torch.Tensor, dt_bias: Optional[torch.Tensor],
+                 a2: torch.Tensor, bm: torch.Tensor, cm: torch.Tensor, d_skip: Optional[torch.Tensor],
+                 y: torch.Tensor, num_seqs: int, q_start: torch.Tensor, state_slots: torch.Tensor,
+                 state: torch.Tensor, ssm_offset: int, conv_in: Optional[torch.Tensor] = None,
+                 taps: int = 1, conv_offset: int = 0) -> None:
+    """The scan of a selective state-space mixer with a decay per channel and state, over each
+    request's tokens, from and into its state row (float32 [slots, n]; S [C, N] at `ssm_offset`):
+    dt = softplus(dt_raw + dt_bias), S <- exp(dt A) S + dt x B^T, y = (S C + D x) silu(z). x and z
+    [T, C], bm and cm [T, N] are 2-D views in the activation type, dt_raw float32 [T, C], a2
+    float32 [C, N] = A log2(e), y [T, C] in the activation type. With `conv_in` (the raw inputs
+    [T, C] of the convolution before the scan) the kept inputs [taps - 1, C] at `conv_offset` of
+    the state row are moved on as `causal_conv_act` would have."""
+    _need_cuda(x, z, dt_raw, dt_bias, a2, bm, cm, d_skip, y, q_start, state_slots, state, conv_in)
+    T, C = x.shape
+    N = a2.shape[1]
+    assert x.dtype == z.dtype == bm.dtype == cm.dtype == y.dtype and z.shape == y.shape == (T, C)
+    assert bm.shape == cm.shape == (T, N) and bm.stride(0) == cm.stride(0)
+    assert dt_raw.dtype == torch.float32 and dt_raw.shape == (T, C) and y.is_contiguous()
+    assert all(t.stride(1) == 1 for t in (x, z, dt_raw) + ((bm, cm) if N > 1 else ()))
+    assert a2.dtype == torch.float32 and a2.is_contiguous() and a2.shape[0] == C
+    for t in (dt_bias, d_skip):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == C and t.is_contiguous())
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+    assert q_start.dtype == state_slots.dtype == torch.int32
+    assert q_start.numel() == num_seqs + 1 and state_slots.numel() == num_seqs
+    assert conv_in is None or (conv_in.shape == (T, C) and conv_in.stride(1) == 1 and conv_in.dtype == x.dtype)
+    lib = load_library("state_space")
+    _check(lib.tgo_channel_scan(
+        _ptr(x), c_ll(x.stride(0)), _ptr(z), c_ll(z.stride(0)), c_int(dtype_code(x.dtype)), _ptr(dt_raw),
+        c_ll(dt_raw.stride(0)), _ptr(dt_bias), _ptr(a2), _ptr(bm), _ptr(cm), c_ll(bm.stride(0)),
+        _ptr(d_skip), _ptr(y), c_int(num_seqs), c_int(C), c_int(N), _ptr(q_start), _ptr(state_slots),
+        _ptr(state), c_ll(state.stride(0)), c_ll(ssm_offset), _ptr(conv_in),
+        c_ll(conv_in.stride(0) if conv_in is not None else 0), c_int(taps), c_ll(conv_offset), _stream()),
+        "channel_scan", f"(channels={C}, state={N})")
+
+
+# how a router's logits become scores
+ROUTER_SCORES = {"chosen": 0, "all": 1, "sigmoid": 2}
+
+
 def moe_tile_rows() -> int:
     """Rows of one expert a tile of the routed products holds at most."""
     return int(load_library("moe").tgo_moe_tile_rows())
@@ -924,7 +1001,10 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
                      w_gate: Optional[torch.Tensor], w_up: torch.Tensor, w_down: torch.Tensor, top: int,
                      activation: str, extra: Optional[torch.Tensor] = None,
                      scores: str = "chosen", correction: Optional[torch.Tensor] = None,
-                     identity: int = 0, extra_gated: bool = False) -> torch.Tensor:
+                     identity: int = 0, extra_gated: bool = False, groups: int = 1, keep: int = 1,
+                     renormalize: bool = True, route_scale: float = 1.0,
+                     beside: Optional[torch.Tensor] = None,
+                     residual: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """A routed feed-forward: each row of x [T, d] goes to the `top` experts with the largest
     router scores (w_router float32 [E, d], b_router float32 [E]; float32 sums); expert e is
     w_down[e] (act(w_gate[e] x) * (w_up[e] x)), or, with w_gate None, w_down[e] act(w_up[e] x).
@@ -936,8 +1016,16 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
     `correction` (float32, one per router output), the weights are the chosen scores divided by
     their sum. `identity`: the router has that many outputs after the E experts that stand for
     experts whose output is the row of x itself. `extra_gated`: w_router carries one more row,
-    after all of those, whose logit through a logistic function multiplies `extra`."""
-    _need_cuda(x, w_router, b_router, w_gate, w_up, w_down, extra, correction)
+    after all of those, whose logit through a logistic function multiplies `extra`.
+
+    `scores` "sigmoid": as "all" with each logit's logistic function as its score. With either,
+    `groups` > 1 cuts the router outputs into equal runs of neighbours and only those of the
+    `keep` runs whose two largest choice scores sum highest can be chosen; without `renormalize`
+    the weights are the chosen scores as they are. `route_scale` multiplies the weights.
+
+    `beside` ([T, d], float32 or bfloat16) is added to the result; with `residual` (float32
+    [T, d]) the result is added there and None is returned."""
+    _need_cuda(x, w_router, b_router, w_gate, w_up, w_down, extra, correction, beside, residual)
     T, d = x.shape
     E, ff = w_up.shape[0], w_up.shape[1]
     outputs = E + identity
@@ -952,7 +1040,12 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
     assert extra is None or (extra.shape == (T, d) and extra.is_contiguous() and
                              extra.dtype == torch.float32)
     assert not extra_gated or extra is not None
-    assert 0 < top <= outputs and E > 0 and scores in ("chosen", "all")
+    assert 0 < top <= outputs and E > 0 and scores in ROUTER_SCORES
+    assert groups >= 1 and outputs % groups == 0 and 0 < keep <= groups and \
+        keep * (outputs // groups) >= top and (groups == 1 or scores != "chosen")
+    for t in (beside, residual):
+        assert t is None or (t.shape == (T, d) and t.is_contiguous())
+    assert residual is None or residual.dtype == torch.float32
     dev, pairs = x.device, T * top
     max_tiles = min(pairs, pairs // moe_tile_rows() + E)
     ints = torch.empty(3 * pairs + 3 * E + 2 + 3 * max_tiles, dtype=torch.int32, device=dev)
@@ -965,22 +1058,23 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
     gate = torch.empty(T, dtype=torch.float32, device=dev) if extra_gated else None
     hidden = torch.empty((pairs, ff), dtype=x.dtype, device=dev)
     y = torch.empty((pairs, d), dtype=torch.float32, device=dev)
-    out = torch.empty((T, d), dtype=torch.float32, device=dev)
+    out = residual if residual is not None else torch.empty((T, d), dtype=torch.float32, device=dev)
     lib = load_library("moe")
     _check(lib.tgo_moe_route(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w_router), _ptr(b_router),
         c_int(T), c_int(d), c_int(outputs), c_int(top), _ptr(ids), _ptr(wts), _ptr(counts), _ptr(fill),
         _ptr(offsets), _ptr(perm), _ptr(place), _ptr(tile_info), _ptr(tiles), c_int(max_tiles),
-        c_int(1 if scores == "all" else 0), _ptr(correction), c_int(E), _ptr(gate),
-        _stream()), "moe_route", f"(E={E}+{identity}, top={top})")
+        c_int(ROUTER_SCORES[scores]), _ptr(correction), c_int(E), _ptr(gate), c_int(groups), c_int(keep),
+        c_int(1 if renormalize else 0), c_float(route_scale), _stream()), "moe_route", f"(E={E}+{identity}, top={top})")
     _check(lib.tgo_moe_experts(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w_gate), _ptr(w_up),
         _ptr(w_down), _ptr(hidden), _ptr(y), _ptr(wts), _ptr(extra), _ptr(out), c_int(T), c_int(d),
         c_int(ff), c_int(top), c_int(PLAIN_ACTIVATIONS[activation]), _ptr(perm), _ptr(tile_info),
         _ptr(tiles), c_int(max_tiles), _ptr(ids if identity else None), c_int(E), _ptr(gate),
-        _stream()), "moe_experts", f"(d={d}, ff={ff})")
+        _ptr(beside), c_int(dtype_code(beside.dtype) if beside is not None else 0),
+        c_int(1 if residual is not None else 0), _stream()), "moe_experts", f"(d={d}, ff={ff})")
     LAUNCHES[0] += 4
-    return out
+    return None if residual is not None else out
 
 
 def attention_mixed(q: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv_heads: int,

@@ -7,7 +7,8 @@ pending and handed to the next norm, which does it in its own kernel. The two no
 checkpoint names come from the layer spec's `tensors` table (roles mixer_norm, ffn_norm).
 The second, `PostNormScaledResidual` below, norms and scales each sublayer's output instead;
 the third norms a sublayer's input and its output; the fourth, `PostNormResidual`, norms the
-sum, so that the stream itself is what the norm leaves.
+sum, so that the stream itself is what the norm leaves; `HyperConnections` keeps several copies
+of the stream; `ParallelResidual` gives both sublayers the same normed rows.
 """
 from __future__ import annotations
 
@@ -485,3 +486,52 @@ class HyperConnections(Part):
 
 
 BLOCKS.register("hyper_connections", HyperConnections)
+
+
+class ParallelResidual(Part):
+    """Arrangement in which both sublayers read one norm's rows and are added together:
+
+        n = norm(h);  h = h + (mixer(n) + feed_forward(n))
+
+    The stream, the norm and the adds are float32, and so are the rows of the sublayers' last
+    products. A feed-forward whose forward takes `beside` and `residual` adds the mixer's result
+    and its own to the stream in one pass; another's result is left pending after the mixer's
+    has been added. A layer may have no feed-forward. Tensor roles of the layer spec: mixer_norm."""
+
+    def __init__(self, spec: LayerSpec, hidden: int, device=None):
+        p = spec.prefix
+        names = tensor_names(spec.tensors, p, ["mixer_norm"], "parallel block")
+        self.norm1 = NORMS.get(spec.norm.kind)(spec.norm, hidden, names["mixer_norm"])
+        self.mixer = MIXERS.get(spec.mixer.kind)(spec.mixer, hidden, p, device)
+        self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward = FEED_FORWARDS.get(spec.feed_forward.kind)(spec.feed_forward, hidden, p, device)
+        for part in (self.mixer, self.feed_forward):
+            if part is not None and hasattr(part, "out_dtype"):
+                part.out_dtype = torch.float32
+        self._joins = self.feed_forward is not None and \
+            {"beside", "residual"} <= set(inspect.signature(self.feed_forward.forward).parameters)
+
+    def parts(self):
+        return [p for p in (self.norm1, self.mixer, self.feed_forward) if p is not None]
+
+    weight_specs = PreNormResidual.weight_specs
+    bind = PreNormResidual.bind
+    libraries = PreNormResidual.libraries
+    prepare_capture = PreNormResidual.prepare_capture
+    flops = PreNormResidual.flops
+    cache_bytes_read = PreNormResidual.cache_bytes_read
+
+    def forward(self, h, pending, ctx, cache):
+        n = self.norm1.forward(h, pending, ctx.act_dtype)
+        a = self.mixer.forward(n, ctx, cache)
+        if self.feed_forward is None:
+            return h, a
+        if self._joins:
+            self.feed_forward.forward(n, ctx, residual=h, beside=a)
+            return h, None
+        ops.residual_add(h, a)
+        return h, self.feed_forward.forward(n, ctx)
+
+
+BLOCKS.register("parallel_residual", ParallelResidual)

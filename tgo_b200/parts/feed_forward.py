@@ -173,7 +173,15 @@ class RoutedExperts(Part):
     weights are not; `identity_experts` n, the router has n more outputs after the experts,
     whose expert gives back its input; `shared_gate` (role shared_gate, [1, hidden]), the shared
     feed-forward's output is multiplied by a logistic gate per token (the gate's row rides as
-    the router matrix's last row, so its logit is a float32 sum too)."""
+    the router matrix's last row, so its logit is a float32 sum too); `router_scores` "sigmoid",
+    as "all" with the logistic function of each logit as its score; `router_groups` (count, keep),
+    the router outputs fall into `count` equal runs of neighbours, a run counts as the sum of its
+    two largest choice scores, and only the outputs of the best `keep` runs can be chosen;
+    `router_renormalize` False, the weights are the chosen scores as they are; `router_scale`, a
+    factor on the weights.
+
+    `beside` (what another sublayer made of the same rows) is added in the pass that sums the
+    experts; with `residual` that pass adds everything to the stream and None comes back."""
     out_dtype = None        # the result is float32 rows when a block asks, else the activations'
 
     def __init__(self, spec: FeedForwardSpec, hidden: int, prefix: str, device=None):
@@ -182,14 +190,28 @@ class RoutedExperts(Part):
         self.E, self.top = int(spec.experts), int(spec.top)
         self.gated = bool(getattr(spec, "gated", True))
         self.identity = int(getattr(spec, "identity_experts", 0) or 0)
-        self.scores = "all" if getattr(spec, "router_scores", "chosen") == "all" else "chosen"
+        self.scores = getattr(spec, "router_scores", "chosen") or "chosen"
+        if self.scores not in ops.ROUTER_SCORES:
+            raise ValueError(f"routed feed-forward: router scores {self.scores!r}; known: "
+                             f"{sorted(ops.ROUTER_SCORES)}")
+        self.renormalize = bool(getattr(spec, "router_renormalize", True))
+        self.route_scale = float(getattr(spec, "router_scale", 1.0))
+        self.groups, self.keep = getattr(spec, "router_groups", None) or (1, 1)
+        outputs = self.E + self.identity
+        if self.groups < 1 or outputs % self.groups or not 0 < self.keep <= self.groups or \
+                self.keep * (outputs // self.groups) < self.top:
+            raise ValueError(f"routed feed-forward: {self.keep} of {self.groups} groups of "
+                             f"{outputs} experts for a top {self.top}")
+        if self.scores == "chosen" and (self.groups > 1 or not self.renormalize):
+            raise ValueError("routed feed-forward: groups and weights that are not renormalized "
+                             "belong to scores over all experts")
         self.correction = bool(getattr(spec, "router_correction", False))
         self.shared_gate = bool(getattr(spec, "shared_gate", False))
         if not 0 < self.top <= self.E + self.identity:
             raise ValueError(f"routed feed-forward: top {self.top} of {self.E + self.identity} experts")
         if self.shared_gate and spec.shared is None:
             raise ValueError("routed feed-forward: a gate on the shared feed-forward needs one")
-        if self.correction and self.scores != "all":
+        if self.correction and self.scores == "chosen":
             raise ValueError("routed feed-forward: the correction belongs to scores over all experts")
         self.activation = spec.activation or "silu"
         known = ops.ACTIVATIONS if self.gated else ops.PLAIN_ACTIVATIONS
@@ -266,12 +288,16 @@ class RoutedExperts(Part):
             total += self.shared.flops(extents, first_positions, writes_cache)
         return total
 
-    def forward(self, x, ctx):
+    def forward(self, x, ctx, residual=None, beside=None):
         x = ops.rows_of(x)
         extra = self.shared.forward(x, ctx) if self.shared is not None else None
         y = ops.moe_feed_forward(x, self.w_router, self.b_router, self.w_gate, self.w_up,
                                  self.w_down, self.top, self.activation, extra, self.scores,
-                                 self.router_correction, self.identity, self.shared_gate)
+                                 self.router_correction, self.identity, self.shared_gate,
+                                 self.groups, self.keep, self.renormalize, self.route_scale,
+                                 beside, residual)
+        if residual is not None:
+            return None
         want = self.out_dtype or ctx.act_dtype
         if want == torch.float32:
             return y

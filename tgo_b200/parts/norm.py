@@ -23,6 +23,11 @@ def stored_gain(w: torch.Tensor, unit_offset: bool) -> torch.Tensor:
 
 
 class RMSNorm(Part):
+    def fold_scale(self, scale: float) -> None:
+        """From here on the normed rows come multiplied by `scale` (a factor on what the next
+        product makes of them, taken at no cost)."""
+        self.gain = (self.gain * scale).contiguous()
+
     def __init__(self, spec: NormSpec, width: int, name: str):
         self.eps = float(spec.eps)
         self.width = width
@@ -74,6 +79,8 @@ class GroupRMSNorm(Part):
         self.unit_offset = bool(getattr(spec, "unit_offset", False))
         self.gain: Optional[torch.Tensor] = None
 
+    fold_scale = RMSNorm.fold_scale
+
     def weight_specs(self):
         return [WeightSpec(self.name, (self.width,), "gain")]
 
@@ -106,5 +113,44 @@ class GroupRMSNorm(Part):
         ops.scaled_add_norm(h, y, bias, alpha, self.gain, self.eps, act)
 
 
+class LayerNorm(Part):
+    """Layer norm with a gain and a bias (named by the spec's `bias_suffix`): y = (x - mean x) / sqrt(mean
+    (x - mean x)^2 + eps) * gain + bias, float32, the residual add and the row selection fused
+    as in RMSNorm."""
+
+    def __init__(self, spec: NormSpec, width: int, name: str):
+        self.eps = float(spec.eps)
+        self.width = width
+        if not spec.bias_suffix:
+            raise ValueError("layer norm: the spec names no bias (bias_suffix)")
+        self.name, self.bias_name = name, name + spec.bias_suffix
+        self.unit_offset = bool(getattr(spec, "unit_offset", False))
+        self.gain: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def weight_specs(self):
+        return [WeightSpec(self.name, (self.width,), "gain"),
+                WeightSpec(self.bias_name, (self.width,), "constant")]
+
+    def bind(self, weights):
+        self.gain = stored_gain(weights[self.name], self.unit_offset)
+        self.bias = weights[self.bias_name].to(torch.float32).contiguous()
+
+    def fold_scale(self, scale: float) -> None:
+        self.gain = (self.gain * scale).contiguous()
+        self.bias = (self.bias * scale).contiguous()
+
+    def libraries(self, dtype, page_size):
+        return ["elementwise"]
+
+    def forward(self, h: torch.Tensor, delta: Optional[torch.Tensor], out_dtype: torch.dtype,
+                rows: Optional[torch.Tensor] = None):
+        n = h.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.width), dtype=out_dtype, device=h.device)
+        ops.add_layernorm(h, delta, self.gain, self.bias, self.eps, out, rows)
+        return out
+
+
 NORMS.register("rmsnorm", RMSNorm)
+NORMS.register("layernorm", LayerNorm)
 NORMS.register("group_rmsnorm", GroupRMSNorm)

@@ -76,6 +76,9 @@ def _register_builtin() -> None:
     from .config import vimelorn
     if vimelorn.ARCHITECTURE not in ARCHITECTURES:
         ARCHITECTURES.register(vimelorn.ARCHITECTURE, vimelorn.vimelorn_model_spec)
+    from .config import bekunex
+    if bekunex.ARCHITECTURE not in ARCHITECTURES:
+        ARCHITECTURES.register(bekunex.ARCHITECTURE, bekunex.bekunex_model_spec)
 
 
 _register_builtin()
