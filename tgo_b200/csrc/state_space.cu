@@ -305,6 +305,19 @@ TGO_API int tgo_selective_scan(const float* xbc, int C, const void* dt_raw, long
 #define CS_TOK 32
 #define CS_THREADS 128
 
+// One step of one state: 2^e S + add. A state that decays slowly is multiplied by nearly 1
+// thousands of times, and an exponential that is off by the same fraction of a unit in the last
+// place each time adds up; the float32 engine therefore takes the change S (2^e - 1), whose
+// rounding is relative to the change, while the decay is slow.
+template <typename T> __device__ __forceinline__ float cs_step(float S, float e, float add);
+template <> __device__ __forceinline__ float cs_step<bf16>(float S, float e, float add) {
+    return fmaf(exp2f(e), S, add);
+}
+template <> __device__ __forceinline__ float cs_step<float>(float S, float e, float add) {
+    if (e < -0.5f) return fmaf(exp2f(e), S, add);
+    return S + fmaf(expm1f(e * 0.69314718055994531f), S, add);
+}
+
 template <typename T, int L, int NS>
 __global__ void __launch_bounds__(CS_THREADS)
 channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ z, long long z_stride,
@@ -396,10 +409,10 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
 #pragma unroll
                 for (int i = 0; i < NS; i += 4) {
                     const float4 bq = *(const float4*)(br + i), cq = *(const float4*)(cr + i);
-                    S[i] = fmaf(exp2f(dd.x * A[i]), S[i], dd.y * bq.x);
-                    S[i + 1] = fmaf(exp2f(dd.x * A[i + 1]), S[i + 1], dd.y * bq.y);
-                    S[i + 2] = fmaf(exp2f(dd.x * A[i + 2]), S[i + 2], dd.y * bq.z);
-                    S[i + 3] = fmaf(exp2f(dd.x * A[i + 3]), S[i + 3], dd.y * bq.w);
+                    S[i] = cs_step<T>(S[i], dd.x * A[i], dd.y * bq.x);
+                    S[i + 1] = cs_step<T>(S[i + 1], dd.x * A[i + 1], dd.y * bq.y);
+                    S[i + 2] = cs_step<T>(S[i + 2], dd.x * A[i + 2], dd.y * bq.z);
+                    S[i + 3] = cs_step<T>(S[i + 3], dd.x * A[i + 3], dd.y * bq.w);
                     p = fmaf(S[i], cq.x, p);
                     p = fmaf(S[i + 1], cq.y, p);
                     p = fmaf(S[i + 2], cq.z, p);
