@@ -507,6 +507,66 @@ def vimelorn_beside_totatar(args):
     return 0
 
 
+def bekunex_config(width, heads, kv, dim, ff, layers, vocab=32768):
+    """(windowed latent attention, scan, rotated latent attention) repeated, every layer with
+    routed experts beside its mixer: latents of 512 with as many heads as the other designs' (the
+    rotated ones with a shared key part of 64; a window of 1024 with sinks and a gate, whose
+    latent the later windowed layers borrow), twice the width's channels of 16 states each in the
+    scans, 32 experts in 4 groups of which 2 stay open, top 4, with a shared expert (as much
+    active width as Totatar's)."""
+    moe = {"kind": "moe", "router": {"experts": 32, "top": 4, "scale": 1.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": ff // 8}, "shared": {"ff": ff // 2}}
+    win = {"heads": heads, "dim": dim, "vdim": dim, "kv_rank": 512, "mask": {"size": 1024}, "scale": dim ** -0.5}
+    scan = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
+    rot = {"heads": heads, "dim": dim, "rot_dim": 64, "vdim": dim, "kv_rank": 512,
+           "rot": {"dims": 64, "base": 1e4}, "scale": (dim + 64) ** -0.5}
+    out = []
+    for i in range(layers):
+        kind, mixer = (("latent_attention_2", win), ("mamba1", scan), ("latent_attention", rot))[i % 3]
+        if i % 3 == 0 and i:
+            mixer = dict(mixer, kv_from=0)
+        out.append({"type": kind, "mixer": mixer, "mlp": moe})
+    return {"architecture": "Bekunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "logit_scale": 0.5, "layers": out}
+
+
+def bekunex_beside_totatar(args):
+    """One JSON line per measurement: prefill of 2,048 tokens and decode at batch 8 and 64 for
+    Bekunex, for Totatar (the closest model the engine has by its layers: scans and routed experts
+    with a shared one) and for Derosun (the closest by its attention: latent rows), at each size;
+    then Bekunex's kernels one by one beside their like kernels."""
+    import torch
+
+    import tgo_b200
+    from tgo_b200.engine.measure import load_peaks, measure_decode, measure_prefill
+    from tgo_b200.engine.measure_kernels import measure_bekunex_kernels
+    peaks = load_peaks()
+    layers = args.layers or 6
+    steps = min(args.steps, 64)
+    for name, (width, heads, kv, dim, ff) in DESIGN_SIZES.items():
+        for arch, make in (("bekunex", bekunex_config), ("totatar", totatar_config), ("derosun", derosun_config)):
+            model = tgo_b200.open_random(make(width, heads, kv, dim, ff, layers), seed=SEED,
+                                         dtype="bfloat16", sigma=0.02, gain_sigma=0.05)
+            pre = measure_prefill(model, PREFILL_TOKENS, warmup=2, steps=3, seed=SEED, page_size=PAGE)
+            rec = {"size": name, "model": arch, "layers": layers,
+                   "prefill_ms": round(pre["ms"], 3), "prefill_tokens_per_s": round(pre["tokens_per_s"]),
+                   "prefill_frac_of_library_peak": round(pre["tflops"] / peaks["bf16_tflops"], 3)}
+            for b in (8, 64):
+                r = measure_decode(model, b, PROMPT, steps, warmup=max(args.warmup, 3), seed=SEED,
+                                   page_size=PAGE)
+                rec[f"decode_b{b}_ms"] = round(r["ms_per_step"], 4)
+                rec[f"decode_b{b}_tokens_per_s"] = round(r["tokens_per_s"])
+                rec[f"decode_b{b}_hbm_frac"] = round(r["gbs"] / peaks["hbm_gbs"], 3)
+            print(json.dumps(rec), flush=True)
+            del model
+            torch.cuda.empty_cache()
+        for rec in measure_bekunex_kernels(width, heads, dim, 512, 64, 1024, 2 * width, 16, width // 16, 4, 32, 4,
+                                           4, 2, ff // 8):
+            rec["size"] = name
+            print(json.dumps(rec), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -521,7 +581,8 @@ def main():
     ap.add_argument("--prompt", type=int, default=PROMPT, help="with --only decode: prompt length")
     ap.add_argument("--rows", default="256,512,1024,2048", help="with --only products: row counts")
     ap.add_argument("--only", default="", choices=["", "prefill", "decode", "serve", "check", "products",
-                                                   "gafonex", "totatar", "derosun", "vimelorn"],
+                                                   "gafonex", "totatar", "derosun", "vimelorn",
+                                                   "bekunex"],
                     help="run just the 2,048-token prefill, just the decode steps, the "
                          "continuous-batching workload, or the exactness check at real layer "
                          "sizes (float32 against bfloat16, alone against cut and mixed; 4 layers "
@@ -536,7 +597,9 @@ def main():
                          "in the same way; vimelorn: the Vimelorn design (several residual "
                          "streams, windowed attention that keeps the first keys, attention with "
                          "a bias by distance, routed small experts) beside Totatar and Qwen3 in "
-                         "the same way")
+                         "the same way; bekunex: the Bekunex design (latent attention with a "
+                         "window and lent latents, scans with a decay per channel, experts in "
+                         "groups beside the mixer) beside Totatar and Derosun in the same way")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -561,6 +624,8 @@ def main():
         return derosun_beside_gafonex(args)
     if args.only == "vimelorn":
         return vimelorn_beside_totatar(args)
+    if args.only == "bekunex":
+        return bekunex_beside_totatar(args)
     config, seed = dict(SHAPES[args.shape][0]), SHAPES[args.shape][1]
     if args.layers:
         config["num_hidden_layers"] = args.layers

@@ -721,15 +721,161 @@ def measure_vimelorn_kernels(width: int, heads: int, kv_heads: int, key_dim: int
     return out
 
 
+def measure_bekunex_kernels(width: int, heads: int, head_dim: int, latent_rank: int, rope_dim: int,
+                            window: int, inner: int, state: int, dt_rank: int, taps: int, experts: int,
+                            top: int, groups: int, keep: int, expert_ff: int, prompt: int = 2048,
+                            batch: int = 64, context: int = 2048, page: int = 16,
+                            device="cuda:0") -> List[Dict[str, object]]:
+    """The kernels of the layers that give one norm's rows to a latent attention (with a window, a
+    sink and a gate, or rotated) or a scan with a decay per channel, and to experts chosen inside
+    groups by logistic scores, each timed alone beside the like kernel of the framework's closest
+    layers at equal sizes (same timing and denominators as `measure_kernels`)."""
+    from types import SimpleNamespace
+
+    from ..parts.attention_sink import sink_attention
+    dev = torch.device(device)
+    peaks = load_peaks()
+    hbm, tc, fma = peaks["hbm_gbs"], peaks["bf16_tflops"], _fma_tflops(dev)
+    flush = L2Flusher(dev)
+    out: List[Dict[str, object]] = []
+    bf = torch.bfloat16
+
+    def row(name, ms, like, like_ms, bound, work, like_work=None):
+        peak = {"hbm": hbm * 1e9, "tensor": tc * 1e12, "fma": fma * 1e12}[bound]
+        rec = {"kernel": name, "us": round(ms * 1e3, 1), "bound": bound,
+               "frac": round(work / (ms * 1e-3) / peak, 4)}
+        if like:
+            rec.update(like=like, like_us=round(like_ms * 1e3, 1),
+                       like_frac=round((like_work or work) / (like_ms * 1e-3) / peak, 4))
+        out.append(rec)
+
+    def context_of(n_req, extent, first):
+        T = n_req * extent
+        pos = (torch.arange(extent, dtype=torch.int32, device=dev) + first).repeat(n_req)
+        seq = torch.arange(n_req, dtype=torch.int32, device=dev).repeat_interleave(extent)
+        qs = torch.arange(n_req + 1, dtype=torch.int32, device=dev) * extent
+        z = torch.zeros(n_req, dtype=torch.int32, device=dev)
+        return StepContext(T, n_req, pos, pos, seq, qs, z, torch.arange(n_req, dtype=torch.int32, device=dev),
+                           z, bf, extents=[extent] * n_req, first_positions=[first] * n_req,
+                           max_extent=extent, max_context=first + extent, decode_only=extent == 1)
+
+    H, dk, rank, dr = heads, head_dim, latent_rank, rope_dim
+    cases = ((1, prompt, 0, f"{prompt} tokens"), (batch, 1, context - 1, f"batch {batch} x {context} keys"))
+    # ---- attention over latent rows: the window with a sink, beside the rotated rows without
+    # either (the form that Derosun's latent layers run)
+    sinks = torch.randn(H, device=dev)
+    for n_req, extent, first, what in cases:
+        T = n_req * extent
+        ctx = context_of(n_req, extent, first)
+        plane, table = _paged(n_req, first + extent, 1, rank, page, dev)
+        wide, wtable = _paged(n_req, first + extent, 1, rank + dr, page, dev)
+        q = torch.randn((T, H * rank), device=dev).to(bf)
+        qr = torch.randn((T, H * (rank + dr)), device=dev).to(bf)
+        o = torch.empty((T, H * rank), dtype=bf, device=dev)
+        cache = SimpleNamespace(k=plane, v=None, page_size=page, block_tables=table)
+        wcache = SimpleNamespace(k=wide, v=None, page_size=page, block_tables=wtable)
+        ms = _timed(lambda: sink_attention(q, o, H, 1, rank, rank, cache, ctx, 0.05, window, sinks,
+                                           value_row=rank), flush)
+        like_ms = _timed(lambda: sink_attention(qr, o, H, 1, rank + dr, rank, wcache, ctx, 0.05, 0, None,
+                                                value_row=rank + dr), flush)
+        like = f"latent attention, rows of {rank + dr}, every earlier key"
+        if extent > 1:
+            keys = sum(min(t + 1, window) for t in range(prompt))
+            row(f"latent attention, window {window} and sink, {what}", ms, like, like_ms, "tensor",
+                4.0 * H * rank * keys, 2.0 * H * (2 * rank + dr) * (prompt * (prompt + 1) / 2))
+        else:
+            row(f"latent attention, window {window} and sink, {what}", ms, like, like_ms, "hbm",
+                2.0 * n_req * min(window, context) * rank, 2.0 * n_req * context * (rank + dr))
+        # ---- the values expanded per head, with the gate in the same pass, beside without
+        w_uv = (torch.randn((H, dk, rank), device=dev) * 0.05).to(bf)
+        wide_rows = torch.randn((T, 2 * H * dk), device=dev).to(bf)
+        y = torch.empty((T, H * dk), dtype=bf, device=dev)
+        ms = _timed(lambda: ops.head_linear(o, rank, w_uv, y, dk, wide_rows[:, H * dk:]), flush)
+        like_ms = _timed(lambda: ops.head_linear(o, rank, w_uv, y, dk), flush)
+        bound = ("tensor", 2.0 * T * H * rank * dk) if extent > 1 else \
+            ("hbm", 2.0 * (H * rank * dk + T * H * (rank + 2 * dk)))
+        row(f"value expansion per head with the output gate, {what}", ms, "the same without a gate", like_ms, *bound)
+    # ---- the scan: convolution, scan with its gate and kept inputs, beside the scan with a decay
+    # per head and a state of equal size (heads of 64 channels)
+    c, N = inner, state
+    floats = c * N + (taps - 1) * c
+    w, cb = torch.randn((c, taps), device=dev) * 0.3, torch.zeros(c, device=dev)
+    a2 = -torch.rand((c, N), device=dev) * 8.0
+    dtb, dsk = torch.zeros(c, device=dev), torch.ones(c, device=dev)
+    P, N2 = 64, 128
+    H2 = max(1, c * N // (P * N2))
+    C2 = H2 * P + 2 * N2
+    for n_req, extent, first, what in ((1, prompt, 0, f"{prompt} tokens"), (batch, 1, context - 1, f"batch {batch}")):
+        T = n_req * extent
+        ctx = context_of(n_req, extent, first)
+        xz = (torch.randn((T, 2 * c), device=dev) * 0.5).to(bf)
+        st = torch.zeros((n_req + 1, floats), dtype=torch.float32, device=dev)
+        u = torch.empty((T, c), dtype=bf, device=dev)
+        uf = torch.empty((T, c), dtype=torch.float32, device=dev)
+        conv = lambda y, keep: ops.causal_conv_act(xz[:, :c], w, cb, y, n_req, ctx.seq_ids, ctx.q_start,  # noqa: E731
+                                                   ctx.state_slots, st, c * N, keep=keep)
+        ms = _timed(lambda: conv(u, False), flush)
+        like_ms = _timed(lambda: conv(uf, True), flush)
+        row(f"causal_conv_act, bfloat16 rows out, {what}", ms, "float32 rows out + kept inputs", like_ms, "hbm",
+            4.0 * T * c, 6.0 * T * c)
+        conv(u, False)
+        rbc = (torch.randn((T, dt_rank + 2 * N), device=dev) * 0.5).to(bf)
+        dt = torch.randn((T, c), device=dev)
+        y = torch.empty((T, c), dtype=bf, device=dev)
+        ms = _timed(lambda: ops.channel_scan(u, xz[:, c:], dt, dtb, a2, rbc[:, dt_rank:dt_rank + N],
+                                             rbc[:, dt_rank + N:], dsk, y, n_req, ctx.q_start, ctx.state_slots,
+                                             st, 0, xz[:, :c], taps, c * N), flush)
+        xbc = torch.randn((T, C2), device=dev)
+        st2 = torch.zeros((n_req + 1, H2 * N2 * P), device=dev)
+        dtr, dtb2 = torch.randn((T, H2), device=dev).to(bf), torch.zeros(H2, device=dev)
+        y2 = torch.empty((T, H2 * P), dtype=torch.float32, device=dev)
+        like_ms = _timed(lambda: ops.selective_scan(xbc, dtr, dtb2, dtb2, dtb2, y2, n_req, H2, 1, N2, P,
+                                                    ctx.q_start, ctx.state_slots, st2, 0), flush)
+        like = f"selective_scan, {H2} heads of {P} x {N2}"
+        if extent > 1:
+            row(f"channel_scan, {c} channels x {N}, {what}", ms, like, like_ms, "fma", 6.0 * T * c * N,
+                6.0 * T * H2 * N2 * P)
+        else:
+            row(f"channel_scan, {c} channels x {N}, {what}", ms, like, like_ms, "hbm",
+                8.0 * n_req * c * N + T * c * (4 + 2 * 3), 8.0 * n_req * H2 * N2 * P)
+    # ---- the norm
+    for T, what in ((prompt, f"{prompt} rows"), (batch, f"{batch} rows")):
+        h = torch.randn((T, width), device=dev)
+        n = torch.empty((T, width), dtype=bf, device=dev)
+        gain, bias = torch.ones(width, device=dev), torch.zeros(width, device=dev)
+        ms = _timed(lambda: ops.add_layernorm(h, None, gain, bias, 1e-6, n), flush)
+        like_ms = _timed(lambda: ops.add_rmsnorm(h, None, gain, 1e-6, n), flush)
+        row(f"add_layernorm, {what}", ms, "add_rmsnorm", like_ms, "hbm", T * width * 6.0)
+    # ---- routed experts: logistic scores inside groups, both sublayers' sums into the stream,
+    # beside the softmax over the chosen
+    E, ff = experts, expert_ff
+    wr, corr = torch.randn((E, width), device=dev) * 0.05, torch.randn(E, device=dev) * 0.1
+    wg, wu = ((torch.randn((E, ff, width), device=dev) * 0.02).to(bf) for _ in range(2))
+    wd = (torch.randn((E, width, ff), device=dev) * 0.02).to(bf)
+    for T, what in ((prompt, f"{prompt} tokens"), (batch, f"batch {batch}"), (8, "batch 8")):
+        x = torch.randn((T, width), device=dev).to(bf)
+        extra, beside, h = (torch.randn((T, width), device=dev) for _ in range(3))
+        ms = _timed(lambda: ops.moe_feed_forward(x, wr, None, wg, wu, wd, top, "silu", extra, "sigmoid", corr,
+                                                 0, False, groups, keep, False, 1.5, beside, h), flush)
+        like_ms = _timed(lambda: ops.moe_feed_forward(x, wr, None, wg, wu, wd, top, "silu", extra), flush)
+        bound = ("tensor", 6.0 * T * top * width * ff) if T >= 1024 else \
+            ("hbm", 6.0 * min(E, T * top) * width * ff)
+        row(f"routed experts ({E}, top {top}, best {keep} of {groups} groups, ff {ff}) into the stream, {what}", ms,
+            "routed experts (scores over the chosen)", like_ms, *bound)
+    return out
+
+
 if __name__ == "__main__":
-    # python -m tgo_b200.engine.measure_kernels vimelorn|derosun|totatar|gafonex [width]: the kernels of one design
+    # python -m tgo_b200.engine.measure_kernels bekunex|vimelorn|derosun|totatar|gafonex [width]: the kernels of one design
     # at one size, a JSON line each (small enough to run under a profiler)
     import json
     import sys
     design = sys.argv[1] if len(sys.argv) > 1 else "totatar"
     w = int(sys.argv[2]) if len(sys.argv) > 2 else 2048
     ff = 3 * w
-    if design == "vimelorn":
+    if design == "bekunex":
+        recs = measure_bekunex_kernels(w, 16, 128, 512, 64, 1024, 2 * w, 16, w // 16, 4, 32, 4, 4, 2, ff // 8)
+    elif design == "vimelorn":
         recs = measure_vimelorn_kernels(w, 16, 4, 128, 128, 1024, 4, 4, 4, 32, 2, 4, ff // 8)
     elif design == "derosun":
         recs = measure_derosun_kernels(w, 16, 4, 128, 128, 30.0, 512, 64, 3 * w // 4, w // 256, 128, 256, ff)
