@@ -1,10 +1,11 @@
 // A routed feed-forward (mixture of experts): every token goes to the `top` experts with the
 // largest router logits, weighted by the softmax over those logits alone.
 //
-//   route      logits = Wr x + br in float32 (Wr, br float32; x in the storage type), the top
-//              experts (ties: the lower index), their weights, and a count per expert
+//   logits     Wr x + br in float32 (Wr, br float32; x in the storage type)
+//   pick       the top experts (ties: the lower index), their weights, and a count per expert
 //   plan       expert e's (token, choice) pairs get places offsets[e] .. offsets[e+1]-1; the
 //              places are cut into row tiles of one expert each
+//              (steps of few tokens: pick, plan and scatter are one block's work)
 //   scatter    pair -> place (within an expert the order is whatever the atomics give; a
 //              pair's result does not depend on its place)
 //   up         hidden[place] = act(x Wg_e^T) * (x Wu_e^T) for the token of the pair at `place`
@@ -35,46 +36,84 @@
 #define MOE_TN 64
 #define MOE_TK 16
 
-// ------------------------------------------------------------------------------- route
-// A block of four warps per MOE_RT tokens: warp w takes experts w, w + 4, ... and makes their
-// logits for all the block's tokens at once (a row of Wr is read once per block), lanes over
-// the width; then warp t picks token t's experts.
-#define MOE_RT 4
-template <typename T>
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ wr,
-                 const float* __restrict__ br, int Tn, int d, int E, int top, int* __restrict__ ids,
-                 float* __restrict__ wts, int* __restrict__ counts, int score_mode,
-                 const float* __restrict__ correction, int E_real, float* __restrict__ gate_out,
-                 int groups, int keep, int renorm, float route_scale) {
-    // [MOE_RT][E + 1] logits, [MOE_RT][E] scores, [MOE_RT][groups] strengths of the groups
-    extern __shared__ float smem[];
+// ------------------------------------------------------------------------------ logits
+// A warp takes one router row (an expert) and up to ML_TOK tokens, lanes over the width four
+// channels at a time; a block's eight warps share the tokens, so x comes from the first-level
+// cache after the first. The order of a sum depends on the width alone. out [T, rows]; the last
+// row may have no bias (the gate of a shared expert). Block 0 also zeroes the experts' counts.
+#define ML_TOK 8
+template <typename T> struct Load4;
+template <> struct Load4<bf16> {
+    static __device__ __forceinline__ float4 get(const bf16* p) {
+        const uint2 v = *(const uint2*)p;
+        const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&v.x);
+        const float2 b = __bfloat1622float2(*(const __nv_bfloat162*)&v.y);
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+};
+template <> struct Load4<float> {
+    static __device__ __forceinline__ float4 get(const float* p) { return *(const float4*)p; }
+};
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+moe_logits_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ wr,
+                  const float* __restrict__ br, int Tn, int d, int rows, int E, float* __restrict__ out,
+                  int* __restrict__ counts, int E_real) {
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t0 = blockIdx.x * MOE_RT;
-    const int nt = Tn - t0 < MOE_RT ? Tn - t0 : MOE_RT;
-    const int rows = E + (gate_out ? 1 : 0), ld = E + 1;
-    for (int e = warp; e < rows; e += 4) {
-        const float* w = wr + (size_t)e * d;
-        float a[MOE_RT];
+    if (blockIdx.x == 0 && blockIdx.y == 0)
+        for (int i = threadIdx.x; i < E_real; i += 256) counts[i] = 0;
+    const int e = blockIdx.y * 8 + warp, t0 = blockIdx.x * ML_TOK;
+    if (e >= rows) return;
+    const int nt = Tn - t0 < ML_TOK ? Tn - t0 : ML_TOK;
+    const float* w = wr + (size_t)e * d;
+    const T* xt = x + (size_t)t0 * x_stride;
+    float a[ML_TOK];
 #pragma unroll
-        for (int j = 0; j < MOE_RT; ++j) a[j] = 0.f;
+    for (int j = 0; j < ML_TOK; ++j) a[j] = 0.f;
+    if (VEC) {
+#pragma unroll 4
+        for (int i = 4 * lane; i < d; i += 128) {
+            const float4 wv = *(const float4*)(w + i);
+#pragma unroll
+            for (int j = 0; j < ML_TOK; ++j)
+                if (j < nt) {
+                    const float4 xv = Load4<T>::get(xt + (size_t)j * x_stride + i);
+                    a[j] = fmaf(wv.x, xv.x, a[j]);
+                    a[j] = fmaf(wv.y, xv.y, a[j]);
+                    a[j] = fmaf(wv.z, xv.z, a[j]);
+                    a[j] = fmaf(wv.w, xv.w, a[j]);
+                }
+        }
+    } else {
         for (int i = lane; i < d; i += 32) {
             const float wv = w[i];
 #pragma unroll
-            for (int j = 0; j < MOE_RT; ++j)
-                if (j < nt) a[j] = fmaf(wv, to_f32(x[(size_t)(t0 + j) * x_stride + i]), a[j]);
-        }
-#pragma unroll
-        for (int j = 0; j < MOE_RT; ++j) {
-            const float v = warp_sum(a[j]);
-            if (lane == 0) smem[j * ld + e] = v + ((br && e < E) ? br[e] : 0.f);
+            for (int j = 0; j < ML_TOK; ++j)
+                if (j < nt) a[j] = fmaf(wv, to_f32(xt[(size_t)j * x_stride + i]), a[j]);
         }
     }
-    __syncthreads();
-    if (warp >= nt) return;
-    const int t = t0 + warp;
-    float* lg = smem + (size_t)warp * ld;
+    const float bias = (br && e < E) ? br[e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < ML_TOK; ++j) {
+        const float v = warp_sum(a[j]);
+        if (lane == 0 && j < nt) out[(size_t)(t0 + j) * rows + e] = v + bias;
+    }
+}
+
+// -------------------------------------------------------------------------------- pick
+// One warp picks one token's experts. lg [E + 1], sc [E] and gs [groups] are the warp's own
+// shared memory; `z` the token's logits.
+__device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg, float* sc, float* gs,
+                                         int t, int E, int top, int* __restrict__ ids,
+                                         float* __restrict__ wts, int* counts, int score_mode,
+                                         const float* __restrict__ correction, int E_real,
+                                         float* __restrict__ gate_out, int groups, int keep, int renorm,
+                                         float route_scale) {
+    const int lane = threadIdx.x & 31;
+    for (int e = lane; e < E + (gate_out ? 1 : 0); e += 32) lg[e] = z[e];
+    __syncwarp();
     if (gate_out && lane == 0) gate_out[t] = 1.f / (1.f + expf(-lg[E]));
     float first = 0.f, sum = 0.f, mine = 0.f;
     int mine_e = 0;
@@ -97,7 +136,6 @@ moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __res
     };
     if (score_mode != 0) {
         // scores: the softmax over every logit, or each logit's logistic; the choice adds the correction
-        float* sc = smem + (size_t)MOE_RT * ld + (size_t)warp * E;
         float mx = 0.f, den = 1.f;
         if (score_mode == 1) {
             mx = -INFINITY;
@@ -118,7 +156,6 @@ moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __res
         }
         __syncwarp();
         if (groups > 1) {
-            float* gs = smem + (size_t)MOE_RT * (ld + E) + (size_t)warp * groups;
             const int size = E / groups;
             for (int g = lane; g < groups; g += 32) {
                 float a = -INFINITY, c = -INFINITY;      // the two largest of the run
@@ -185,29 +222,108 @@ moe_route_kernel(const T* __restrict__ x, long long x_stride, const float* __res
     }
 }
 
-// -------------------------------------------------------------------------------- plan
-// One thread: offsets [E + 1], tiles (expert, first place, rows) and their count in
-// tile_info[0]; the fill counters go back to zero.
-__global__ void moe_plan_kernel(const int* __restrict__ counts, int E, int* __restrict__ offsets,
-                                int* __restrict__ fill, int* __restrict__ tile_info,
-                                int* __restrict__ tiles, int max_tiles) {
+#define MOE_PW 4
+__global__ void __launch_bounds__(32 * MOE_PW)
+moe_pick_kernel(const float* __restrict__ logits, int rows, int Tn, int E, int top, int* __restrict__ ids,
+                float* __restrict__ wts, int* __restrict__ counts, int score_mode,
+                const float* __restrict__ correction, int E_real, float* __restrict__ gate_out, int groups,
+                int keep, int renorm, float route_scale) {
+    extern __shared__ float smem[];                      // [MOE_PW][2 E + 1 + groups]
     pdl_wait();
-    if (threadIdx.x || blockIdx.x) return;
-    int at = 0, nt = 0;
-    for (int e = 0; e < E; ++e) {
-        offsets[e] = at;
-        fill[e] = 0;
-        const int c = counts[e];
-        for (int r = 0; r < c && nt < max_tiles; r += MOE_TM) {
-            tiles[3 * nt] = e;
-            tiles[3 * nt + 1] = at + r;
-            tiles[3 * nt + 2] = c - r < MOE_TM ? c - r : MOE_TM;
-            ++nt;
+    const int warp = threadIdx.x >> 5, t = blockIdx.x * MOE_PW + warp;
+    if (t >= Tn) return;
+    float* lg = smem + (size_t)warp * (2 * E + 1 + groups);
+    moe_pick(logits + (size_t)t * rows, lg, lg + E + 1, lg + 2 * E + 1, t, E, top, ids, wts, counts, score_mode,
+             correction, E_real, gate_out, groups, keep, renorm, route_scale);
+}
+
+// -------------------------------------------------------------------------------- plan
+// One block: offsets [E + 1], tiles (expert, first place, rows) and their count in tile_info[0];
+// the fill counters go back to zero. Experts are taken blockDim at a time, the places and tiles
+// before each by a running sum over the block. `scan` is 2 x blockDim ints of shared memory.
+__device__ __forceinline__ void moe_plan(const int* counts, int E, int* __restrict__ offsets, int* fill,
+                                         int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles,
+                                         int* scan) {
+    const int n = blockDim.x, i = threadIdx.x;
+    int at = 0, nt = 0;                                  // places and tiles of the experts before
+    for (int e0 = 0; e0 < E; e0 += n) {
+        const int e = e0 + i;
+        const int c = e < E ? counts[e] : 0, mine = (c + MOE_TM - 1) / MOE_TM;
+        int pc = c, pt = mine;                           // inclusive sums
+        for (int o = 1; o < n; o <<= 1) {
+            scan[i] = pc;
+            scan[n + i] = pt;
+            __syncthreads();
+            if (i >= o) { pc += scan[i - o]; pt += scan[n + i - o]; }
+            __syncthreads();
         }
-        at += c;
+        if (e < E) {
+            offsets[e] = at + pc - c;
+            fill[e] = 0;
+            for (int k = 0; k < mine; ++k) {
+                const int q = nt + pt - mine + k;
+                if (q < max_tiles) {
+                    tiles[3 * q] = e;
+                    tiles[3 * q + 1] = at + pc - c + k * MOE_TM;
+                    tiles[3 * q + 2] = c - k * MOE_TM < MOE_TM ? c - k * MOE_TM : MOE_TM;
+                }
+            }
+        }
+        scan[i] = pc;
+        scan[n + i] = pt;
+        __syncthreads();
+        at += scan[n - 1];
+        nt += scan[2 * n - 1];
+        __syncthreads();
     }
-    offsets[E] = at;
-    tile_info[0] = nt;
+    if (i == 0) {
+        offsets[E] = at;
+        tile_info[0] = nt < max_tiles ? nt : max_tiles;
+    }
+}
+
+__global__ void __launch_bounds__(256)
+moe_plan_kernel(const int* __restrict__ counts, int E, int* __restrict__ offsets, int* __restrict__ fill,
+                int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles) {
+    __shared__ int scan[512];
+    pdl_wait();
+    moe_plan(counts, E, offsets, fill, tile_info, tiles, max_tiles, scan);
+}
+
+// A step of few tokens: pick, plan and scatter by one block, the counts and fill counters in
+// shared memory.
+#define MOE_FEW_WARPS 16
+__global__ void __launch_bounds__(32 * MOE_FEW_WARPS)
+moe_route_few_kernel(const float* __restrict__ logits, int rows, int Tn, int E, int top, int* __restrict__ ids,
+                     float* __restrict__ wts, int score_mode, const float* __restrict__ correction, int E_real,
+                     float* __restrict__ gate_out, int groups, int keep, int renorm, float route_scale,
+                     int* __restrict__ offsets, int* __restrict__ perm, int* __restrict__ place,
+                     int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles) {
+    extern __shared__ float smem[];                      // [warps][2 E + 1 + groups], counts, fill, scan
+    const int per = 2 * E + 1 + groups;
+    int* counts = (int*)(smem + (size_t)MOE_FEW_WARPS * per);
+    int* fill = counts + E_real;
+    int* scan = fill + E_real;
+    const int warp = threadIdx.x >> 5, n = 32 * MOE_FEW_WARPS;
+    for (int i = threadIdx.x; i < E_real; i += n) counts[i] = 0;
+    pdl_wait();
+    __syncthreads();
+    float* lg = smem + (size_t)warp * per;
+    for (int t = warp; t < Tn; t += MOE_FEW_WARPS) {
+        moe_pick(logits + (size_t)t * rows, lg, lg + E + 1, lg + 2 * E + 1, t, E, top, ids, wts, counts, score_mode,
+                 correction, E_real, gate_out, groups, keep, renorm, route_scale);
+        __syncwarp();
+    }
+    __syncthreads();                                     // ids are in memory for the whole block
+    moe_plan(counts, E_real, offsets, fill, tile_info, tiles, max_tiles, scan);
+    __syncthreads();
+    for (int p = threadIdx.x; p < Tn * top; p += n) {
+        const int e = ids[p];
+        if (e >= E_real) { place[p] = -1; continue; }
+        const int at = offsets[e] + atomicAdd(&fill[e], 1);
+        perm[at] = p;
+        place[p] = at;
+    }
 }
 
 __global__ void moe_scatter_kernel(const int* __restrict__ ids, int pairs,
@@ -473,11 +589,36 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
                                    int top, const int* __restrict__ ids, int E_real,
                                    const T* __restrict__ x, long long x_stride,
                                    const float* __restrict__ extra_gate,
-                                   const TB* __restrict__ beside, int accumulate) {
+                                   const TB* __restrict__ beside, int accumulate, int vec) {
     pdl_wait();
     const int t = blockIdx.x;
     const float eg = extra_gate ? extra_gate[t] : 1.f;
-    for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    if (vec) {                                           // four columns a thread
+        for (int c = 4 * (blockIdx.y * blockDim.x + threadIdx.x); c < d; c += 4 * blockDim.x * gridDim.y) {
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 ex = extra ? *(const float4*)(extra + (size_t)t * d + c) : a;
+            const float4 bs = beside ? Load4<TB>::get(beside + (size_t)t * d + c) : a;
+            const float4 o = accumulate ? *(const float4*)(out + (size_t)t * d + c) : a;
+#pragma unroll 4
+            for (int j = 0; j < top; ++j) {
+                const size_t pair = (size_t)t * top + j;
+                const float w = wts[pair];
+                const float4 v = (ids && ids[pair] >= E_real) ? Load4<T>::get(x + (size_t)t * x_stride + c)
+                                                              : *(const float4*)(y + pair * d + c);
+                a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y);
+                a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+            }
+            if (extra) {
+                a.x = fmaf(eg, ex.x, a.x); a.y = fmaf(eg, ex.y, a.y);
+                a.z = fmaf(eg, ex.z, a.z); a.w = fmaf(eg, ex.w, a.w);
+            }
+            if (beside) { a.x += bs.x; a.y += bs.y; a.z += bs.z; a.w += bs.w; }
+            if (accumulate) { a.x += o.x; a.y += o.y; a.z += o.z; a.w += o.w; }
+            *(float4*)(out + (size_t)t * d + c) = a;
+        }
+        return;
+    }
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < d; c += blockDim.x * gridDim.y) {
         float a = 0.f;
         for (int j = 0; j < top; ++j) {
             const size_t pair = (size_t)t * top + j;
@@ -493,38 +634,52 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
 
 TGO_API int tgo_moe_tile_rows() { return MOE_TM; }
 
-// ids, place int32 [T top]; wts float32 [T top]; counts, fill int32 [E]; offsets int32 [E + 1];
-// perm int32 [T top]; tile_info int32 [1]; tiles int32 [3 max_tiles].
+// ids, place int32 [T top]; wts float32 [T top]; logits float32 [T, router rows]; counts, fill
+// int32 [E]; offsets int32 [E + 1]; perm int32 [T top]; tile_info int32 [1]; tiles int32
+// [3 max_tiles].
+#define MOE_FEW_TOKENS 128
 TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const float* wr,
-                          const float* br, int T, int d, int E, int top, int* ids, float* wts,
+                          const float* br, int T, int d, int E, int top, float* logits, int* ids, float* wts,
                           int* counts, int* fill, int* offsets, int* perm, int* place,
                           int* tile_info, int* tiles, int max_tiles, int score_mode,
                           const float* correction, int E_real, float* gate_out, int groups, int keep,
-                          int renorm, float route_scale, cudaStream_t stream) {
+                          int renorm, float route_scale, int* launches, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0 || E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || max_tiles <= 0 ||
         E_real < 0 || E_real > E || score_mode < 0 || score_mode > 2 || groups < 1 || E % groups ||
-        keep < 1 || keep > groups || (long long)keep * (E / groups) < top || (groups > 1 && score_mode == 0))
+        keep < 1 || keep > groups || (long long)keep * (E / groups) < top || (groups > 1 && score_mode == 0) ||
+        (dtype != TGO_BF16 && dtype != TGO_F32))
         return TGO_E_BAD_ARG;
-    int rc = E_real ? (int)cudaMemsetAsync(counts, 0, sizeof(int) * E_real, stream) : 0;
+    const int rows = E + (gate_out ? 1 : 0);
+    const dim3 lgrid((T + ML_TOK - 1) / ML_TOK, (rows + 7) / 8);
+    const bool vec = d % 4 == 0 && x_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)wr % 16 == 0;
+#define LOGITS_GO(TT, V)                                                                                    \
+    tgo_launch_pdl(moe_logits_kernel<TT, V>, lgrid, dim3(256), 0, stream, (const TT*)x, x_stride, wr, br, T, d, \
+                   rows, E, logits, counts, E_real)
+    int rc = dtype == TGO_BF16 ? (vec ? LOGITS_GO(bf16, true) : LOGITS_GO(bf16, false))
+                               : (vec ? LOGITS_GO(float, true) : LOGITS_GO(float, false));
+#undef LOGITS_GO
     if (rc) return rc;
-    const size_t smem = (size_t)MOE_RT * (2 * E + 1 + groups) * sizeof(float);
-    if (smem > 48 * 1024) {                              // more than about 1000 router outputs
-        cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t per = (size_t)(2 * E + 1 + groups) * sizeof(float);
+    const size_t few = MOE_FEW_WARPS * per + (size_t)(2 * E_real + 64 * MOE_FEW_WARPS) * sizeof(int);
+    if (T <= MOE_FEW_TOKENS && few <= 200 * 1024) {
+        if (few > 48 * 1024)
+            cudaFuncSetAttribute(moe_route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)few);
+        *launches = 2;
+        return tgo_launch_pdl(moe_route_few_kernel, dim3(1), dim3(32 * MOE_FEW_WARPS), few, stream,
+                              (const float*)logits, rows, T, E, top, ids, wts, score_mode, correction, E_real,
+                              gate_out, groups, keep, renorm, route_scale, offsets, perm, place, tile_info, tiles,
+                              max_tiles);
     }
-    if (dtype == TGO_BF16)
-        moe_route_kernel<bf16><<<(T + MOE_RT - 1) / MOE_RT, 128, smem, stream>>>((const bf16*)x, x_stride, wr, br, T, d, E,
-                                                                  top, ids, wts, counts, score_mode, correction, E_real, gate_out,
-                                                                  groups, keep, renorm, route_scale);
-    else if (dtype == TGO_F32)
-        moe_route_kernel<float><<<(T + MOE_RT - 1) / MOE_RT, 128, smem, stream>>>((const float*)x, x_stride, wr, br, T, d,
-                                                                   E, top, ids, wts, counts, score_mode, correction, E_real, gate_out,
-                                                                  groups, keep, renorm, route_scale);
-    else
-        return TGO_E_BAD_ARG;
-    if ((rc = launch_status())) return rc;
-    rc = tgo_launch_pdl(moe_plan_kernel, dim3(1), dim3(32), 0, stream, (const int*)counts, E_real, offsets, fill,
+    *launches = 4;
+    const size_t smem = MOE_PW * per;
+    if (smem > 48 * 1024)                                // more than about 1000 router outputs
+        cudaFuncSetAttribute(moe_pick_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    rc = tgo_launch_pdl(moe_pick_kernel, dim3((T + MOE_PW - 1) / MOE_PW), dim3(32 * MOE_PW), smem, stream,
+                        (const float*)logits, rows, T, E, top, ids, wts, counts, score_mode, correction, E_real,
+                        gate_out, groups, keep, renorm, route_scale);
+    if (rc) return rc;
+    rc = tgo_launch_pdl(moe_plan_kernel, dim3(1), dim3(256), 0, stream, (const int*)counts, E_real, offsets, fill,
                         tile_info, tiles, max_tiles);
     if (rc) return rc;
     const int pairs = T * top;
@@ -544,10 +699,14 @@ TGO_API int tgo_moe_experts(const void* x, long long x_stride, int dtype, const 
     if (T <= 0) return 0;
     if (d <= 0 || ff <= 0 || top <= 0 || max_tiles <= 0 || max_tiles > 65535 || act < 0 || act > 3)
         return TGO_E_BAD_ARG;
+    const int comb_vec = d % 4 == 0 && x_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 &&
+                         (uintptr_t)extra % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)beside % 16 == 0;
+    const int comb_y = comb_vec && d > 512 ? (d / 512 < 16 ? d / 512 : 16) : 1;
     if (beside && beside_dtype != TGO_F32 && beside_dtype != TGO_BF16) return TGO_E_BAD_ARG;
 #define MOE_COMBINE_OF(TT, TB)                                                                             \
-    tgo_launch_pdl(moe_combine_kernel<TT, TB>, dim3(T), dim3(256), 0, stream, (const float*)y, wts, extra, out, \
-                   d, top, ids, E_real, (const TT*)x, x_stride, extra_gate, (const TB*)beside, accumulate)
+    tgo_launch_pdl(moe_combine_kernel<TT, TB>, dim3(T, comb_y), dim3(128), 0, stream, (const float*)y, wts, extra,  \
+                   out, d, top, ids, E_real, (const TT*)x, x_stride, extra_gate, (const TB*)beside, accumulate,     \
+                   comb_vec)
 #define MOE_COMBINE(TT) (beside && beside_dtype == TGO_BF16 ? MOE_COMBINE_OF(TT, bf16) : MOE_COMBINE_OF(TT, float))
     const dim3 g1((ff + MOE_TN - 1) / MOE_TN, max_tiles), g2((d + MOE_TN - 1) / MOE_TN, max_tiles);
     int rc;

@@ -51,6 +51,86 @@ causal_conv_act_kernel(const T* __restrict__ x, long long x_stride, const float*
     }
 }
 
+// The same with eight channels a thread (16-byte loads of x) and CV_TOK consecutive tokens, the
+// window of inputs in registers: for up to four taps, C, the row stride and x's address as
+// multiples of eight elements.
+#define CV_TOK 8
+__device__ __forceinline__ void cv_load(float* v, const bf16* p) {
+    const uint4 q = *(const uint4*)p;
+    const uint32_t* w = (const uint32_t*)&q;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)(w + k));
+        v[2 * k] = f.x;
+        v[2 * k + 1] = f.y;
+    }
+}
+__device__ __forceinline__ void cv_store(bf16* p, const float* v) {
+    uint4 q;
+    uint32_t* w = (uint32_t*)&q;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+        w[k] = *(const uint32_t*)&b;
+    }
+    *(uint4*)p = q;
+}
+__device__ __forceinline__ void cv_store(float* p, const float* v) {
+    *(float4*)p = make_float4(v[0], v[1], v[2], v[3]);
+    *(float4*)(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+
+template <typename TY, int TAPS>
+__global__ void __launch_bounds__(128)
+causal_conv_act_x8_kernel(const bf16* __restrict__ x, long long x_stride, const float* __restrict__ w,
+                          const float* __restrict__ bias, TY* __restrict__ y, int Tn, int C,
+                          const int* __restrict__ seq_ids, const int* __restrict__ q_start,
+                          const int* __restrict__ state_slots, const float* __restrict__ state,
+                          long long state_stride, long long conv_offset) {
+    pdl_wait();
+    const int c = 8 * (blockIdx.y * blockDim.x + threadIdx.x), t_lo = blockIdx.x * CV_TOK;
+    if (c >= C) return;
+    float wt[TAPS][8], bs[8], win[TAPS][8];              // win[j] meets wt[j]; the last is the token's own
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        bs[i] = bias ? bias[c + i] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[j][i] = w[(size_t)(c + i) * TAPS + j];
+    }
+    const int t_hi = t_lo + CV_TOK < Tn ? t_lo + CV_TOK : Tn;
+    for (int t = t_lo; t < t_hi; ++t) {
+        const int b = seq_ids[t], r = t - q_start[b];
+        if (t == t_lo || r == 0) {                       // a window from the start: rows of the step, then kept ones
+            const float* kept = state + (size_t)state_slots[b] * state_stride + conv_offset;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) {
+                const int back = TAPS - 1 - j;
+                if (back <= r) {
+                    cv_load(win[j], x + (size_t)(t - back) * x_stride + c);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) win[j][i] = kept[(size_t)(TAPS - 1 - (back - r)) * C + c + i];
+                }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+                for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
+        }
+        cv_load(win[TAPS - 1], x + (size_t)t * x_stride + c);
+        float o[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            float a = bs[i];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) a = fmaf(wt[j][i], win[j][i], a);
+            o[i] = __fdividef(a, 1.f + __expf(-a));
+        }
+        cv_store(y + (size_t)t * C + c, o);
+    }
+}
+
 // After the convolution has run: the kept inputs of every request become the last taps - 1
 // of (kept inputs, then the step's inputs). A thread per (request, channel).
 template <typename T>
@@ -90,11 +170,21 @@ TGO_API int tgo_causal_conv_act(const void* x, long long x_stride, int dtype, co
     tgo_launch_pdl(causal_conv_act_kernel<TT, TY>, dim3(T, cy), dim3(256), 0, stream, (const TT*)x, x_stride, w, \
                    bias, (TY*)y, C, taps, seq_ids, q_start, state_slots, (const float*)state, state_stride, \
                    conv_offset)
-    if (dtype == TGO_BF16 && y_dtype == TGO_F32) rc = CONV_GO(bf16, float);
+#define CONV_X8(TY, TAPS)                                                                                  \
+    tgo_launch_pdl(causal_conv_act_x8_kernel<TY, TAPS>, dim3((T + CV_TOK - 1) / CV_TOK, (C / 8 + 127) / 128),      \
+                   dim3(128), 0, stream, (const bf16*)x, x_stride, w, bias, (TY*)y, T, C, seq_ids, q_start,      \
+                   state_slots, (const float*)state, state_stride, conv_offset)
+#define CONV_TAPS(TY) (taps == 1 ? CONV_X8(TY, 1) : taps == 2 ? CONV_X8(TY, 2) : taps == 3 ? CONV_X8(TY, 3) : CONV_X8(TY, 4))
+    if (dtype == TGO_BF16 && (y_dtype == TGO_F32 || y_dtype == TGO_BF16) && taps <= 4 && C % 8 == 0 &&
+        x_stride % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0)
+        rc = y_dtype == TGO_F32 ? CONV_TAPS(float) : CONV_TAPS(bf16);
+    else if (dtype == TGO_BF16 && y_dtype == TGO_F32) rc = CONV_GO(bf16, float);
     else if (dtype == TGO_BF16 && y_dtype == TGO_BF16) rc = CONV_GO(bf16, bf16);
     else if (dtype == TGO_F32 && y_dtype == TGO_F32) rc = CONV_GO(float, float);
     else return TGO_E_BAD_ARG;
 #undef CONV_GO
+#undef CONV_X8
+#undef CONV_TAPS
     if (rc || taps == 1 || !keep) return rc;
     if (dtype == TGO_BF16)
         return tgo_launch_pdl(causal_conv_keep_kernel<bf16>, dim3(B, cy), dim3(256), 0, stream, (const bf16*)x,
@@ -289,21 +379,21 @@ TGO_API int tgo_selective_scan(const float* xbc, int C, const void* dt_raw, long
 }
 
 // ---------------------------------------------------------------------- scan per channel
-// A block per (request, CS_CH channels): L lanes share a channel and lane l keeps states
-// l * NS .. l * NS + NS - 1 of it in registers for the whole walk over the request's tokens,
-// CS_TOK at a time. A tile's inputs (x, raw dt, z, B, C) are loaded into registers while the
-// tile before it is walked, dt goes through softplus once per (token, channel) and lies in
-// shared memory beside dt * x, B and C as float32 rows. Four tokens are taken together: their
-// decays do not depend on the state, so only one FMA per state and token is a chain, and the
-// four sums over n are joined by a transposing exchange in the quad (three shuffles for four
-// tokens) and, for L > 4, by shuffles over the quads, the same order for every token. Tokens
-// past the end of a tile have dt = 0 and leave the state as it is. The thread that loaded a
-// (token, channel) pair adds D x, multiplies by silu(z) and stores. `a2` is A log2(e).
+// A block per (request, CS_CH channels) in two halves that work on different tiles of CS_TOK
+// tokens at the same time. The walking half: L lanes share a channel and lane l keeps states
+// l * NS .. l * NS + NS - 1 of it in registers for the whole walk over the request's tokens. Four
+// tokens are taken together: their decays do not depend on the state, so only one FMA per state
+// and token is a chain, and the four sums over n are joined by a transposing exchange in the
+// quad (three shuffles for four tokens) and, for L > 4, by shuffles over the quads, the same
+// order for every token. Tokens past the end of a tile have dt = 0 and leave the state as it is.
+// The serving half: while tile k is walked it puts tile k + 1 into shared memory (dt through
+// softplus once per (token, channel), beside dt * x; B and C as float32 rows), asks for tile
+// k + 2's inputs, and finishes tile k - 1 (D x added, times silu(z), stored). `a2` is A log2(e).
 //
 // The walk ends with the convolution's kept inputs: the last taps - 1 of (kept, then the
 // step's raw inputs `conv_in`), which the convolution has read before this kernel starts.
 #define CS_TOK 32
-#define CS_THREADS 128
+#define CS_HALF 128
 
 // One step of one state: 2^e S + add. A state that decays slowly is multiplied by nearly 1
 // thousands of times, and an exponential that is off by the same fraction of a unit in the last
@@ -311,15 +401,44 @@ TGO_API int tgo_selective_scan(const float* xbc, int C, const void* dt_raw, long
 // rounding is relative to the change, while the decay is slow.
 template <typename T> __device__ __forceinline__ float cs_step(float S, float e, float add);
 template <> __device__ __forceinline__ float cs_step<bf16>(float S, float e, float add) {
-    return fmaf(exp2f(e), S, add);
+    float d;                                             // a decay below 2^-126 is none
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(d) : "f"(e));
+    return fmaf(d, S, add);
 }
 template <> __device__ __forceinline__ float cs_step<float>(float S, float e, float add) {
     if (e < -0.5f) return fmaf(exp2f(e), S, add);
     return S + fmaf(expm1f(e * 0.69314718055994531f), S, add);
 }
 
+// softplus and silu: the library's functions in the float32 engine; in the bfloat16 engine the
+// special-function unit's exponential, logarithm and reciprocal (float32, a few units in the
+// last place), with log(1 + e) by its series where e is small.
+template <typename T> __device__ __forceinline__ float cs_softplus(float v);
+template <> __device__ __forceinline__ float cs_softplus<float>(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+template <> __device__ __forceinline__ float cs_softplus<bf16>(float v) {
+    const float e = __expf(v);
+    const float small = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333334f), -0.5f), 1.f);
+    return v > 20.f ? v : e < 0.03f ? small : __logf(1.f + e);
+}
+template <typename T> __device__ __forceinline__ float cs_silu(float z);
+template <> __device__ __forceinline__ float cs_silu<float>(float z) { return z / (1.f + expf(-z)); }
+template <> __device__ __forceinline__ float cs_silu<bf16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
+// The kept inputs of one channel of one request.
+template <typename T>
+__device__ __forceinline__ void cs_keep(float* kept, const T* __restrict__ conv_in, long long conv_in_stride,
+                                        int c, int C, int taps, int t0, int n_tok) {
+    const int keep = taps - 1;
+    // ascending i reads kept[n_tok + i] before any later write could reach it
+    for (int i = 0; i < keep; ++i) {
+        const int at = n_tok + i;                        // place in (kept, then new)
+        kept[(size_t)i * C + c] = at < keep ? kept[(size_t)at * C + c]
+                                            : to_f32(conv_in[(size_t)(t0 + at - keep) * conv_in_stride + c]);
+    }
+}
+
 template <typename T, int L, int NS>
-__global__ void __launch_bounds__(CS_THREADS)
+__global__ void __launch_bounds__(2 * CS_HALF)
 channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ z, long long z_stride,
                     const float* __restrict__ dt_raw, long long dt_stride, const float* __restrict__ dt_bias,
                     const float* __restrict__ a2, const T* __restrict__ bm, const T* __restrict__ cm,
@@ -327,152 +446,251 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
                     const int* __restrict__ q_start, const int* __restrict__ state_slots,
                     float* __restrict__ state, long long state_stride, long long ssm_offset,
                     const T* __restrict__ conv_in, long long conv_in_stride, int taps, long long conv_offset) {
-    constexpr int CH = CS_THREADS / L;                   // channels of this block
+    constexpr int CH = CS_HALF / L;                      // channels of this block
     constexpr int NP = L * NS;                           // N rounded up
-    constexpr int PER = CS_TOK * CH / CS_THREADS;        // (token, channel) pairs a thread loads
-    constexpr int RSTEP = CS_THREADS / CH;               // tokens between a thread's pairs (= L)
-    constexpr int PBC = (CS_TOK * NP + CS_THREADS - 1) / CS_THREADS;
+    constexpr int PER = CS_TOK * CH / CS_HALF;           // (token, channel) pairs a serving thread loads
+    constexpr int RSTEP = CS_HALF / CH;                  // tokens between a thread's pairs (= L)
+    constexpr int PBC = CS_TOK * NP / CS_HALF;
     extern __shared__ __align__(16) float cs_smem[];
-    float* s_b = cs_smem;                                // [CS_TOK][NP]
-    float* s_c = s_b + CS_TOK * NP;                      // [CS_TOK][NP]
-    float2* s_dt = (float2*)(s_c + CS_TOK * NP);         // [CS_TOK][CH + 1]: dt, dt x
-    float* s_y = (float*)(s_dt + CS_TOK * (CH + 1));     // [CS_TOK][CH + 1]
+    float* s_b = cs_smem;                                // [2][CS_TOK][NP]
+    float* s_c = s_b + 2 * CS_TOK * NP;                  // [2][CS_TOK][NP]
+    float2* s_dt = (float2*)(s_c + 2 * CS_TOK * NP);     // [2][CS_TOK][CH + 1]: dt, dt x
+    float* s_y = (float*)(s_dt + 2 * CS_TOK * (CH + 1)); // [2][CS_TOK][CH + 1]
     pdl_wait();
     const int b = blockIdx.x, c0 = blockIdx.y * CH;
     const int t0 = q_start[b], n_tok = q_start[b + 1] - t0;
-    const int tid = threadIdx.x;
+    const int n_tiles = (n_tok + CS_TOK - 1) / CS_TOK;
     float* row = state + (size_t)state_slots[b] * state_stride;
-    // the walking role: channel wc, states from n0
-    const int lane_l = tid % L, wc = c0 + tid / L, n0 = lane_l * NS;
-    const bool live = wc < C;
-    float S[NS], A[NS];
+    if (threadIdx.x < CS_HALF) {
+        // ---- walking
+        const int tid = threadIdx.x;
+        const int lane_l = tid % L, wch = tid / L, wc = c0 + wch, n0 = lane_l * NS;
+        const bool live = wc < C;
+        float S[NS], A[NS];
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {
-        const bool ok = live && n0 + i < N;
-        S[i] = ok ? row[ssm_offset + (size_t)wc * N + n0 + i] : 0.f;
-        A[i] = ok ? a2[(size_t)wc * N + n0 + i] : 0.f;
+        for (int i = 0; i < NS; ++i) {
+            const bool ok = live && n0 + i < N;
+            S[i] = ok ? row[ssm_offset + (size_t)wc * N + n0 + i] : 0.f;
+            A[i] = ok ? a2[(size_t)wc * N + n0 + i] : 0.f;
+        }
+        const bool odd = tid & 1, high = tid & 2;
+        __syncthreads();                                 // tile 0 is in shared memory
+        for (int k = 0; k < n_tiles; ++k) {
+            const int nt = n_tok - k * CS_TOK < CS_TOK ? n_tok - k * CS_TOK : CS_TOK;
+            const float2* dts = s_dt + (k & 1) * CS_TOK * (CH + 1) + wch;
+            const float* bs = s_b + (k & 1) * CS_TOK * NP + n0;
+            const float* cs = s_c + (k & 1) * CS_TOK * NP + n0;
+            float* ys = s_y + (k & 1) * CS_TOK * (CH + 1) + wch;
+#pragma unroll 2
+            for (int r = 0; r < nt; r += 4) {
+                float part[4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const float2 dd = dts[(r + u) * (CH + 1)];
+                    const float* br = bs + (r + u) * NP;
+                    const float* cr = cs + (r + u) * NP;
+                    float p = 0.f, p2 = 0.f;
+#pragma unroll
+                    for (int i = 0; i < NS; i += 4) {
+                        const float4 bq = *(const float4*)(br + i), cq = *(const float4*)(cr + i);
+                        S[i] = cs_step<T>(S[i], dd.x * A[i], dd.y * bq.x);
+                        S[i + 1] = cs_step<T>(S[i + 1], dd.x * A[i + 1], dd.y * bq.y);
+                        S[i + 2] = cs_step<T>(S[i + 2], dd.x * A[i + 2], dd.y * bq.z);
+                        S[i + 3] = cs_step<T>(S[i + 3], dd.x * A[i + 3], dd.y * bq.w);
+                        p = fmaf(S[i], cq.x, p);
+                        p2 = fmaf(S[i + 1], cq.y, p2);
+                        p = fmaf(S[i + 2], cq.z, p);
+                        p2 = fmaf(S[i + 3], cq.w, p2);
+                    }
+                    part[u] = p + p2;
+                }
+                // four sums over the quad, transposed: lane q of a quad ends with token r + q
+                const float s0 = odd ? part[0] : part[1], s1 = odd ? part[2] : part[3];
+                float k0 = odd ? part[1] : part[0], k1 = odd ? part[3] : part[2];
+                k0 += __shfl_xor_sync(0xffffffffu, s0, 1);
+                k1 += __shfl_xor_sync(0xffffffffu, s1, 1);
+                const float s2 = high ? k0 : k1;
+                float sum = high ? k1 : k0;
+                sum += __shfl_xor_sync(0xffffffffu, s2, 2);
+#pragma unroll
+                for (int o = 4; o < L; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+                if (lane_l < 4) ys[(r + (tid & 3)) * (CH + 1)] = sum;
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int i = 0; i < NS; ++i)
+            if (live && n0 + i < N) row[ssm_offset + (size_t)wc * N + n0 + i] = S[i];
+        return;
     }
-    // the loading role: channel lc, tokens lt + RSTEP k
+    // ---- serving: channel lc, tokens lt + RSTEP i of a tile
+    const int tid = threadIdx.x - CS_HALF;
     const int lcl = tid % CH, lc = c0 + lcl, lt = tid / CH;
     const bool lok = lc < C;
     const float bias = (lok && dt_bias) ? dt_bias[lc] : 0.f;
     const float skip = (lok && D) ? D[lc] : 0.f;
-    float xn[PER], zn[PER], dn[PER];
-    float bn[PBC], cn[PBC];
-    auto fetch = [&](int base) {
+    const T zero = from_f32<T>(0.f);
+    T xn[PER], bn[PBC], cn[PBC];                         // raw, so that nothing waits for them here
+    float dn[PER];
+    auto fetch = [&](int k) {
 #pragma unroll
-        for (int k = 0; k < PER; ++k) {
-            const int r = base + lt + RSTEP * k;
+        for (int i = 0; i < PER; ++i) {
+            const int r = k * CS_TOK + lt + RSTEP * i;
             const bool ok = lok && r < n_tok;
             const size_t t = (size_t)(t0 + r);
-            xn[k] = ok ? to_f32(x[t * x_stride + lc]) : 0.f;
-            zn[k] = ok ? to_f32(z[t * z_stride + lc]) : 0.f;
-            dn[k] = ok ? dt_raw[t * dt_stride + lc] : 0.f;
+            xn[i] = ok ? x[t * x_stride + lc] : zero;
+            dn[i] = ok ? dt_raw[t * dt_stride + lc] : 0.f;
         }
 #pragma unroll
-        for (int k = 0; k < PBC; ++k) {
-            const int i = tid + CS_THREADS * k;
-            const int r = base + i / NP, n = i % NP;
-            const bool ok = i < CS_TOK * NP && n < N && r < n_tok;
-            bn[k] = ok ? to_f32(bm[(size_t)(t0 + r) * bc_stride + n]) : 0.f;
-            cn[k] = ok ? to_f32(cm[(size_t)(t0 + r) * bc_stride + n]) : 0.f;
+        for (int i = 0; i < PBC; ++i) {
+            const int q = tid + CS_HALF * i;
+            const int r = k * CS_TOK + q / NP, n = q % NP;
+            const bool ok = n < N && r < n_tok;
+            bn[i] = ok ? bm[(size_t)(t0 + r) * bc_stride + n] : zero;
+            cn[i] = ok ? cm[(size_t)(t0 + r) * bc_stride + n] : zero;
+        }
+    };
+    auto stage = [&](int k) {                            // what fetch(k) has brought
+        float2* dts = s_dt + (k & 1) * CS_TOK * (CH + 1);
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = lt + RSTEP * i;
+            const float dt = k * CS_TOK + r < n_tok ? cs_softplus<T>(dn[i] + bias) : 0.f;
+            dts[r * (CH + 1) + lcl] = make_float2(dt, dt * to_f32(xn[i]));
+        }
+#pragma unroll
+        for (int i = 0; i < PBC; ++i) {
+            s_b[(k & 1) * CS_TOK * NP + tid + CS_HALF * i] = to_f32(bn[i]);
+            s_c[(k & 1) * CS_TOK * NP + tid + CS_HALF * i] = to_f32(cn[i]);
+        }
+    };
+    auto finish = [&](int k) {                           // the walked tile k: gate and store
+        const float* ys = s_y + (k & 1) * CS_TOK * (CH + 1);
+        T xr[PER], zr[PER];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = k * CS_TOK + lt + RSTEP * i;
+            const bool ok = lok && r < n_tok;
+            xr[i] = ok ? x[(size_t)(t0 + r) * x_stride + lc] : zero;
+            zr[i] = ok ? z[(size_t)(t0 + r) * z_stride + lc] : zero;
+        }
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = lt + RSTEP * i;
+            if (lok && k * CS_TOK + r < n_tok)
+                y[(size_t)(t0 + k * CS_TOK + r) * C + lc] =
+                    from_f32<T>(fmaf(skip, to_f32(xr[i]), ys[r * (CH + 1) + lcl]) * cs_silu<T>(to_f32(zr[i])));
         }
     };
     fetch(0);
-    for (int base = 0; base < n_tok; base += CS_TOK) {
-        const int nt = n_tok - base < CS_TOK ? n_tok - base : CS_TOK;
-        float xc[PER], zc[PER];
-#pragma unroll
-        for (int k = 0; k < PER; ++k) {
-            const int r = lt + RSTEP * k;
-            const float v = dn[k] + bias;
-            const float dt = r < nt ? (v > 20.f ? v : log1pf(expf(v))) : 0.f;
-            s_dt[r * (CH + 1) + lcl] = make_float2(dt, dt * xn[k]);
-            xc[k] = xn[k];
-            zc[k] = zn[k];
-        }
-#pragma unroll
-        for (int k = 0; k < PBC; ++k) {
-            const int i = tid + CS_THREADS * k;
-            if (i < CS_TOK * NP) { s_b[i] = bn[k]; s_c[i] = cn[k]; }
-        }
+    stage(0);
+    if (n_tiles > 1) fetch(1);
+    __syncthreads();
+    for (int k = 0; k < n_tiles; ++k) {
+        if (k + 1 < n_tiles) stage(k + 1);
+        if (k + 2 < n_tiles) fetch(k + 2);
+        if (k > 0) finish(k - 1);
         __syncthreads();
-        if (base + CS_TOK < n_tok) fetch(base + CS_TOK);
-        for (int r = 0; r < nt; r += 4) {
-            float part[4];
+    }
+    if (n_tiles > 0) finish(n_tiles - 1);
+    if (conv_in && tid < CH && c0 + tid < C)
+        cs_keep(row + conv_offset, conv_in, conv_in_stride, c0 + tid, C, taps, t0, n_tok);
+}
+
+// A step in which every request brings one token: nothing to stage, a thread takes NS states of
+// one channel of one request (L lanes a channel, four states a 16-byte access where they lie
+// that way), the lanes join their sums and the first of them gates and stores.
+template <typename T, int L, int NS, bool VEC>
+__global__ void __launch_bounds__(128)
+channel_scan_single_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ z, long long z_stride,
+                           const float* __restrict__ dt_raw, long long dt_stride, const float* __restrict__ dt_bias,
+                           const float* __restrict__ a2, const T* __restrict__ bm, const T* __restrict__ cm,
+                           long long bc_stride, const float* __restrict__ D, T* __restrict__ y, int C, int N,
+                           const int* __restrict__ q_start, const int* __restrict__ state_slots,
+                           float* __restrict__ state, long long state_stride, long long ssm_offset,
+                           const T* __restrict__ conv_in, long long conv_in_stride, int taps, long long conv_offset) {
+    constexpr int CH = 128 / L;
+    pdl_wait();
+    const int b = blockIdx.x, lane_l = threadIdx.x % L, n0 = lane_l * NS;
+    const int c = blockIdx.y * CH + threadIdx.x / L;
+    const bool live = c < C;
+    const int t = q_start[b];
+    float* row = state + (size_t)state_slots[b] * state_stride;
+    float* Sg = row + ssm_offset + (size_t)(live ? c : 0) * N + n0;
+    const float* Ag = a2 + (size_t)(live ? c : 0) * N + n0;
+    float S[NS], A[NS];
+    if (VEC) {
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const float2 dd = s_dt[(r + u) * (CH + 1) + tid / L];
-                const float* br = s_b + (r + u) * NP + n0;
-                const float* cr = s_c + (r + u) * NP + n0;
-                float p = 0.f;
-#pragma unroll
-                for (int i = 0; i < NS; i += 4) {
-                    const float4 bq = *(const float4*)(br + i), cq = *(const float4*)(cr + i);
-                    S[i] = cs_step<T>(S[i], dd.x * A[i], dd.y * bq.x);
-                    S[i + 1] = cs_step<T>(S[i + 1], dd.x * A[i + 1], dd.y * bq.y);
-                    S[i + 2] = cs_step<T>(S[i + 2], dd.x * A[i + 2], dd.y * bq.z);
-                    S[i + 3] = cs_step<T>(S[i + 3], dd.x * A[i + 3], dd.y * bq.w);
-                    p = fmaf(S[i], cq.x, p);
-                    p = fmaf(S[i + 1], cq.y, p);
-                    p = fmaf(S[i + 2], cq.z, p);
-                    p = fmaf(S[i + 3], cq.w, p);
-                }
-                part[u] = p;
-            }
-            // four sums over the quad, transposed: lane q of a quad ends with token r + q
-            const bool odd = tid & 1, high = tid & 2;
-            const float s0 = odd ? part[0] : part[1], s1 = odd ? part[2] : part[3];
-            float k0 = odd ? part[1] : part[0], k1 = odd ? part[3] : part[2];
-            k0 += __shfl_xor_sync(0xffffffffu, s0, 1);
-            k1 += __shfl_xor_sync(0xffffffffu, s1, 1);
-            const float s2 = high ? k0 : k1;
-            float sum = high ? k1 : k0;
-            sum += __shfl_xor_sync(0xffffffffu, s2, 2);
-#pragma unroll
-            for (int o = 4; o < L; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-            if (lane_l < 4) s_y[(r + (tid & 3)) * (CH + 1) + tid / L] = sum;
+        for (int i = 0; i < NS; i += 4) {
+            const bool ok = live && n0 + i < N;          // N % 4 == 0: the four are in or out together
+            const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 s4 = ok ? *(const float4*)(Sg + i) : zero4, a4 = ok ? *(const float4*)(Ag + i) : zero4;
+            S[i] = s4.x; S[i + 1] = s4.y; S[i + 2] = s4.z; S[i + 3] = s4.w;
+            A[i] = a4.x; A[i + 1] = a4.y; A[i + 2] = a4.z; A[i + 3] = a4.w;
         }
-        __syncthreads();
+    } else {
 #pragma unroll
-        for (int k = 0; k < PER; ++k) {
-            const int r = lt + RSTEP * k;
-            if (lok && r < nt) {
-                const float v = fmaf(skip, xc[k], s_y[r * (CH + 1) + lcl]);
-                y[(size_t)(t0 + base + r) * C + lc] = from_f32<T>(v * (zc[k] / (1.f + expf(-zc[k]))));
-            }
+        for (int i = 0; i < NS; ++i) {
+            const bool ok = live && n0 + i < N;
+            S[i] = ok ? Sg[i] : 0.f;
+            A[i] = ok ? Ag[i] : 0.f;
         }
     }
+    const float xv = live ? to_f32(x[(size_t)t * x_stride + c]) : 0.f;
+    const float zv = live ? to_f32(z[(size_t)t * z_stride + c]) : 0.f;
+    const float dv = live ? dt_raw[(size_t)t * dt_stride + c] + (dt_bias ? dt_bias[c] : 0.f) : 0.f;
+    const float dt = cs_softplus<T>(dv), dx = dt * xv;
+    float p = 0.f, p2 = 0.f;
 #pragma unroll
-    for (int i = 0; i < NS; ++i)
-        if (live && n0 + i < N) row[ssm_offset + (size_t)wc * N + n0 + i] = S[i];
-    if (conv_in && tid < CH && c0 + tid < C) {
-        const int c = c0 + tid, keep = taps - 1;
-        float* kept = row + conv_offset;
-        // ascending i reads kept[n_tok + i] before any later write could reach it
-        for (int i = 0; i < keep; ++i) {
-            const int at = n_tok + i;                    // place in (kept, then new)
-            kept[(size_t)i * C + c] = at < keep ? kept[(size_t)at * C + c]
-                                                : to_f32(conv_in[(size_t)(t0 + at - keep) * conv_in_stride + c]);
-        }
+    for (int i = 0; i < NS; ++i) {
+        const bool in = n0 + i < N;
+        const float bv = in ? to_f32(bm[(size_t)t * bc_stride + n0 + i]) : 0.f;
+        const float cv = in ? to_f32(cm[(size_t)t * bc_stride + n0 + i]) : 0.f;
+        S[i] = cs_step<T>(S[i], dt * A[i], dx * bv);
+        if (i & 1) p2 = fmaf(S[i], cv, p2); else p = fmaf(S[i], cv, p);
     }
+    if (VEC) {
+#pragma unroll
+        for (int i = 0; i < NS; i += 4)
+            if (live && n0 + i < N) *(float4*)(Sg + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < NS; ++i)
+            if (live && n0 + i < N) Sg[i] = S[i];
+    }
+    float sum = p + p2;
+#pragma unroll
+    for (int o = 1; o < L; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if (lane_l || !live) return;
+    const float skip = D ? D[c] : 0.f;
+    y[(size_t)t * C + c] = from_f32<T>(fmaf(skip, xv, sum) * cs_silu<T>(zv));
+    if (conv_in) cs_keep(row + conv_offset, conv_in, conv_in_stride, c, C, taps, t, 1);
 }
 
 template <typename T, int L, int NS>
 static int launch_channel_scan(const void* x, long long x_stride, const void* z, long long z_stride,
                                const float* dt_raw, long long dt_stride, const float* dt_bias, const float* a2,
-                               const void* bm, const void* cm, long long bc_stride, const float* D, void* y, int B,
-                               int C, int N, const int* q_start, const int* state_slots, float* state,
+                               const void* bm, const void* cm, long long bc_stride, const float* D, void* y, int Tn,
+                               int B, int C, int N, const int* q_start, const int* state_slots, float* state,
                                long long state_stride, long long ssm_offset, const void* conv_in,
                                long long conv_in_stride, int taps, long long conv_offset, cudaStream_t stream) {
-    constexpr int CH = CS_THREADS / L, NP = L * NS;
-    const size_t smem = (size_t)CS_TOK * (2 * NP + 3 * (CH + 1)) * sizeof(float);
+    constexpr int CH = CS_HALF / L, NP = L * NS;
+#define CS_LAUNCH(KERNEL, GRID, BLOCK, SMEM)                                                                  \
+    tgo_launch_pdl(KERNEL, GRID, dim3(BLOCK), SMEM, stream, (const T*)x, x_stride, (const T*)z, z_stride,     \
+                   dt_raw, dt_stride, dt_bias, a2, (const T*)bm, (const T*)cm, bc_stride, D, (T*)y, C, N, q_start, \
+                   state_slots, state, state_stride, ssm_offset, (const T*)conv_in, conv_in_stride, taps, conv_offset)
+    if (Tn == B) {                                       // every request brings one token
+        const dim3 grid(B, (C + 128 / L - 1) / (128 / L));
+        const bool vec = N % 4 == 0 && state_stride % 4 == 0 && ssm_offset % 4 == 0 && (uintptr_t)state % 16 == 0 &&
+                         (uintptr_t)a2 % 16 == 0;
+        if (vec) return CS_LAUNCH((channel_scan_single_kernel<T, L, NS, true>), grid, 128, 0);
+        return CS_LAUNCH((channel_scan_single_kernel<T, L, NS, false>), grid, 128, 0);
+    }
+    const size_t smem = (size_t)2 * CS_TOK * (2 * NP + 3 * (CH + 1)) * sizeof(float);
     auto kernel = channel_scan_kernel<T, L, NS>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return tgo_launch_pdl(kernel, dim3(B, (C + CH - 1) / CH), dim3(CS_THREADS), smem, stream, (const T*)x, x_stride,
-                          (const T*)z, z_stride, dt_raw, dt_stride, dt_bias, a2, (const T*)bm, (const T*)cm,
-                          bc_stride, D, (T*)y, C, N, q_start, state_slots, state, state_stride, ssm_offset,
-                          (const T*)conv_in, conv_in_stride, taps, conv_offset);
+    return CS_LAUNCH(kernel, dim3(B, (C + CH - 1) / CH), 2 * CS_HALF, smem);
+#undef CS_LAUNCH
 }
 
 // x, z column views [T, C], bm, cm column views [T, N] (row stride bc_stride) and conv_in a
@@ -481,22 +699,22 @@ static int launch_channel_scan(const void* x, long long x_stride, const void* z,
 // at `ssm_offset` of its state row, its kept inputs [taps - 1][C] at `conv_offset`.
 TGO_API int tgo_channel_scan(const void* x, long long x_stride, const void* z, long long z_stride, int dtype,
                              const float* dt_raw, long long dt_stride, const float* dt_bias, const float* a2,
-                             const void* bm, const void* cm, long long bc_stride, const float* D, void* y, int B,
-                             int C, int N, const int* q_start, const int* state_slots, float* state,
+                             const void* bm, const void* cm, long long bc_stride, const float* D, void* y, int T,
+                             int B, int C, int N, const int* q_start, const int* state_slots, float* state,
                              long long state_stride, long long ssm_offset, const void* conv_in,
                              long long conv_in_stride, int taps, long long conv_offset, cudaStream_t stream) {
-    if (B <= 0) return 0;
-    if (C <= 0 || N <= 0 || N > 256 || (dtype != TGO_BF16 && dtype != TGO_F32) ||
+    if (B <= 0 || T <= 0) return 0;
+    if (C <= 0 || N <= 0 || N > 256 || T < B || (dtype != TGO_BF16 && dtype != TGO_F32) ||
         state_stride < ssm_offset + (long long)C * N || (C + 3) / 4 > 65535 ||
         (conv_in && (taps < 1 || state_stride < conv_offset + (long long)(taps - 1) * C)))
         return TGO_E_BAD_ARG;
 #define CS_GO(L, NS)                                                                                          \
     (dtype == TGO_BF16                                                                                        \
          ? launch_channel_scan<bf16, L, NS>(x, x_stride, z, z_stride, dt_raw, dt_stride, dt_bias, a2, bm, cm,  \
-                                            bc_stride, D, y, B, C, N, q_start, state_slots, state, state_stride, \
+                                            bc_stride, D, y, T, B, C, N, q_start, state_slots, state, state_stride, \
                                             ssm_offset, conv_in, conv_in_stride, taps, conv_offset, stream)   \
          : launch_channel_scan<float, L, NS>(x, x_stride, z, z_stride, dt_raw, dt_stride, dt_bias, a2, bm, cm, \
-                                             bc_stride, D, y, B, C, N, q_start, state_slots, state, state_stride, \
+                                             bc_stride, D, y, T, B, C, N, q_start, state_slots, state, state_stride, \
                                              ssm_offset, conv_in, conv_in_stride, taps, conv_offset, stream))
     if (N <= 16) return CS_GO(4, 4);
     if (N <= 32) return CS_GO(4, 8);

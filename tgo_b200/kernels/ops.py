@@ -982,7 +982,7 @@ def channel_scan(x: torch.Tensor, z: torch.Tensor, dt_raw: torch.Tensor, dt_bias
     _check(lib.tgo_channel_scan(
         _ptr(x), c_ll(x.stride(0)), _ptr(z), c_ll(z.stride(0)), c_int(dtype_code(x.dtype)), _ptr(dt_raw),
         c_ll(dt_raw.stride(0)), _ptr(dt_bias), _ptr(a2), _ptr(bm), _ptr(cm), c_ll(bm.stride(0)),
-        _ptr(d_skip), _ptr(y), c_int(num_seqs), c_int(C), c_int(N), _ptr(q_start), _ptr(state_slots),
+        _ptr(d_skip), _ptr(y), c_int(T), c_int(num_seqs), c_int(C), c_int(N), _ptr(q_start), _ptr(state_slots),
         _ptr(state), c_ll(state.stride(0)), c_ll(ssm_offset), _ptr(conv_in),
         c_ll(conv_in.stride(0) if conv_in is not None else 0), c_int(taps), c_ll(conv_offset), _stream()),
         "channel_scan", f"(channels={C}, state={N})")
@@ -1055,6 +1055,8 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
     tile_info = ints[o + 3 * E + 1:o + 3 * E + 2]
     tiles = ints[o + 3 * E + 2:]
     wts = torch.empty(pairs, dtype=torch.float32, device=dev)
+    logits = torch.empty((T, w_router.shape[0]), dtype=torch.float32, device=dev)
+    launches = c_int(0)
     gate = torch.empty(T, dtype=torch.float32, device=dev) if extra_gated else None
     hidden = torch.empty((pairs, ff), dtype=x.dtype, device=dev)
     y = torch.empty((pairs, d), dtype=torch.float32, device=dev)
@@ -1062,10 +1064,10 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
     lib = load_library("moe")
     _check(lib.tgo_moe_route(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w_router), _ptr(b_router),
-        c_int(T), c_int(d), c_int(outputs), c_int(top), _ptr(ids), _ptr(wts), _ptr(counts), _ptr(fill),
+        c_int(T), c_int(d), c_int(outputs), c_int(top), _ptr(logits), _ptr(ids), _ptr(wts), _ptr(counts), _ptr(fill),
         _ptr(offsets), _ptr(perm), _ptr(place), _ptr(tile_info), _ptr(tiles), c_int(max_tiles),
         c_int(ROUTER_SCORES[scores]), _ptr(correction), c_int(E), _ptr(gate), c_int(groups), c_int(keep),
-        c_int(1 if renormalize else 0), c_float(route_scale), _stream()), "moe_route", f"(E={E}+{identity}, top={top})")
+        c_int(1 if renormalize else 0), c_float(route_scale), ctypes.byref(launches), _stream()), "moe_route", f"(E={E}+{identity}, top={top})")
     _check(lib.tgo_moe_experts(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w_gate), _ptr(w_up),
         _ptr(w_down), _ptr(hidden), _ptr(y), _ptr(wts), _ptr(extra), _ptr(out), c_int(T), c_int(d),
@@ -1073,7 +1075,7 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
         _ptr(tiles), c_int(max_tiles), _ptr(ids if identity else None), c_int(E), _ptr(gate),
         _ptr(beside), c_int(dtype_code(beside.dtype) if beside is not None else 0),
         c_int(1 if residual is not None else 0), _stream()), "moe_experts", f"(d={d}, ff={ff})")
-    LAUNCHES[0] += 4
+    LAUNCHES[0] += launches.value + 1            # beside the two that _check counted
     return None if residual is not None else out
 
 
