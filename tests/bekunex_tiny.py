@@ -25,6 +25,7 @@ import copy
 import numpy as np
 
 from derosun_tiny import bf16_values, bind_model, write_model_dir  # noqa: F401
+from plain_bekunex import choice_margin
 
 
 def _lat(H, dim, rot, vdim, rank, base, scale):
@@ -118,10 +119,28 @@ def changed(cfg, path, value):
     return cfg
 
 
+KINDS = 6
+
+
+def apart(rng, router, r):
+    """Corrections with which no choice is close, whatever the signs of the KINDS channels."""
+    E, g = r["experts"], r.get("groups") or {"count": 1, "keep": 1}
+    patterns = np.array(np.meshgrid(*[[-1.0, 1.0]] * KINDS)).reshape(KINDS, -1).T
+    scores = (patterns @ router[:, :KINDS].T > 0) * 1.0
+    for _ in range(20000):
+        c = bf16_values(rng.uniform(-1.0, 1.0, E))
+        if min(choice_margin(row, c, r["top"], g["count"], g["keep"]) for row in scores) > 0.03:
+            return c
+    raise ValueError("no corrections keep the choices apart")
+
+
 def make_weights(cfg, seed):
     """name -> float64 array of bfloat16-exact values; lively enough that tokens differ, that
     corrections change which experts are chosen, that sinks and gates matter and that states
-    decay at very different rates."""
+    decay at very different rates. Close calls between experts are rare: the first KINDS channels
+    of the stream carry a sign per token that no layer writes over, every expert's logit is one
+    of those channels, and the corrections keep the choices apart; so what a 16-bit
+    engine rounds decides no choice, and which experts a token takes still depends on it."""
     rng = np.random.default_rng(seed)
     d, V = cfg["width"], cfg["vocab"]
     W = {}
@@ -133,10 +152,12 @@ def make_weights(cfg, seed):
         W[name] = mean + sd * rng.normal(0, 1, n)
 
     W["embed"] = rng.normal(0, 1.0, (V, d))
+    W["embed"][:, :KINDS] = rng.choice([-3.0, 3.0], (V, KINDS)) * (1.0 + 0.05 * rng.normal(size=(V, KINDS)))
     for i, L in enumerate(cfg["layers"]):
         p, m = f"l{i}.", L["mixer"]
         vec(p + "norm1", d, 1.0)
         vec(p + "norm1.b", d, 0.1, 0.3)
+        W[p + "norm1"][:KINDS], W[p + "norm1.b"][:KINDS] = 1.0, 0.0
         p += "mix."
         if L["type"] == "mamba1":
             c, N, R = m["inner"], m["state"], m["dt_rank"]
@@ -165,8 +186,10 @@ def make_weights(cfg, seed):
         if mlp:
             p = f"l{i}.mlp."
             E, f = mlp["router"]["experts"], mlp["expert"]["ff"]
-            mat(p + "router", E, d, 2.0)
-            vec(p + "correction", E, 0.0, 0.3)
+            W[p + "router"] = np.zeros((E, d))
+            for e in range(E):
+                W[p + "router"][e, rng.integers(KINDS)] = rng.choice([-8.0, 8.0])
+            W[p + "correction"] = apart(rng, W[p + "router"], mlp["router"])
             for e in range(E):
                 mat(f"{p}e{e}.gate", f, d, 1.5)
                 mat(f"{p}e{e}.up", f, d)
@@ -176,6 +199,9 @@ def make_weights(cfg, seed):
                 mat(p + "shared.gate", f, d, 1.5)
                 mat(p + "shared.up", f, d)
                 mat(p + "shared.down", d, f)
+    for name in W:
+        if name.endswith(("mix.o", ".down")):
+            W[name][:KINDS] = 0.0
     vec("final.norm", d, 1.0)
     vec("final.norm.b", d, 0.0, 0.3)
     mat("head", V, d, 2.0)

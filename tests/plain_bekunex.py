@@ -158,12 +158,27 @@ def choose_experts(s, correction, top, groups, keep):
     return sorted(open_to, key=lambda e: (-choice[e], e))[:top]
 
 
-def routed(X, W, p, mlp, rnd=same):
+def choice_margin(s, correction, top, groups, keep):
+    """How far the choice of one token is from another one: the smaller of the gap between the
+    weakest open group and the strongest closed one and of the gap between the last expert
+    chosen and the next (infinite where nothing is left out)."""
+    choice = s + correction
+    runs = choice.reshape(groups, -1)
+    strength = np.sort([sum(sorted(run, reverse=True)[:2]) for run in runs])[::-1]
+    gap = strength[keep - 1] - strength[keep] if keep < groups else math.inf
+    best = sorted(range(groups), key=lambda g: -sum(sorted(runs[g], reverse=True)[:2]))[:keep]
+    inside = np.sort(runs[best].ravel())[::-1]
+    return min(gap, inside[top - 1] - inside[top] if len(inside) > top else math.inf)
+
+
+def routed(X, W, p, mlp, rnd=same, margins=None):
     r = mlp["router"]
     g = r.get("groups") or {"count": 1, "keep": 1}
     s = sigmoid(X @ W[p + "router"].T)
     out = np.zeros(X.shape)
     for t in range(len(X)):
+        if margins is not None:
+            margins[t] = min(margins[t], choice_margin(s[t], W[p + "correction"], r["top"], g["count"], g["keep"]))
         for e in choose_experts(s[t], W[p + "correction"], r["top"], g["count"], g["keep"]):
             out[t] += s[t, e] * r["scale"] * gated(X[t:t + 1], W, f"{p}e{e}.", rnd)[0]
     if mlp.get("shared"):
@@ -172,14 +187,17 @@ def routed(X, W, p, mlp, rnd=same):
 
 
 # ------------------------------------------------------------------------------------ model
-def forward(cfg, W, tokens, layer_outputs=None, rnd=same):
+def forward(cfg, W, tokens, layer_outputs=None, rnd=same, margins=None):
     """Logits [n, vocab] of a whole sequence. `layer_outputs`, a list, gets the stream after
-    every layer. With `rnd` (a rounding to a 16-bit type) the sublayers' inputs, the
+    every layer; `margins`, a list, gets for every token the closest call of any of its routers.
+    With `rnd` (a rounding to a 16-bit type) the sublayers' inputs, the
     projections' results and what the last products read are rounded, as a 16-bit engine
     stores them; the stream, the norms, the softmax, the router and the recurrence stay."""
     eps = cfg["norm"]["eps"]
     x = W["embed"][np.asarray(tokens)].astype(np.float64)
     latents = {}
+    if margins is not None:
+        margins[:] = [math.inf] * len(x)
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}.", layer["mixer"]
         h = rnd(layer_norm(x, W[p + "norm1"], W[p + "norm1.b"], eps))
@@ -189,7 +207,7 @@ def forward(cfg, W, tokens, layer_outputs=None, rnd=same):
             lent = latents[m["kv_from"]] if m.get("kv_from") is not None else None
             y, latents[i] = latent_attention(h, W, p + "mix.", m, eps, rnd, lent)
         if layer.get("mlp") is not None:
-            y = y + routed(h, W, p + "mlp.", layer["mlp"], rnd)
+            y = y + routed(h, W, p + "mlp.", layer["mlp"], rnd, margins)
         x = x + y
         if layer_outputs is not None:
             layer_outputs.append(x.copy())

@@ -1025,30 +1025,60 @@ attention_sink_wide_decode_kernel(const bf16* __restrict__ q, long long q_stride
 }
 
 // Joins the shares of a token's keys: out = sum_s O_s 2^(m_s - m) / (sum_s l_s 2^(m_s - m) +
-// 2^(sink - m)), m the largest of the maxima and the sink. A block per (token, head).
-__global__ void attention_sink_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                           const int* __restrict__ positions, const float* __restrict__ sinks,
-                                           bf16* __restrict__ out, long long out_stride, int H, int dv,
-                                           int n_splits) {
-    const int tok = blockIdx.x, head = blockIdx.y;
+// 2^(sink - m)), m the largest of the maxima and the sink. A block per (token, head). The shares'
+// factors are made side by side and lie in shared memory (AS_JOIN of them at a time); the sums over
+// shares are in share order.
+#define AS_JOIN 128
+__global__ void __launch_bounds__(128)
+attention_sink_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                           const int* __restrict__ positions, const float* __restrict__ sinks,
+                           bf16* __restrict__ out, long long out_stride, int H, int dv, int n_splits) {
+    __shared__ float s_w[AS_JOIN], s_l[AS_JOIN], s_m[33];
+    pdl_wait();
+    const int tok = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, n = blockDim.x;
     if (positions[tok] < 0) return;            // zeros were written by the tile kernel
     const size_t at = ((size_t)tok * H + head) * n_splits;
     const float sk2 = sinks ? sinks[head] * AS_LOG2E : -INFINITY;
     float m = sk2;
-    for (int s = 0; s < n_splits; ++s) m = fmaxf(m, part_ml[(at + s) * 2]);
-    float l = sinks ? exp2f(sk2 - m) : 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-        const float ms = part_ml[(at + s) * 2];
-        if (ms != -INFINITY) l += part_ml[(at + s) * 2 + 1] * exp2f(ms - m);
-    }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    for (int d = threadIdx.x; d < dv; d += blockDim.x) {
-        float a = 0.f;
-        for (int s = 0; s < n_splits; ++s) {
-            const float ms = part_ml[(at + s) * 2];
-            if (ms != -INFINITY) a += part_o[(at + s) * dv + d] * exp2f(ms - m);
+    for (int s = tid; s < n_splits; s += n) m = fmaxf(m, part_ml[(at + s) * 2]);
+    m = warp_max(m);
+    if ((tid & 31) == 0) s_m[tid >> 5] = m;
+    __syncthreads();
+    for (int w = 0; w < n / 32; ++w) m = fmaxf(m, s_m[w]);
+    float l = sk2 != -INFINITY ? exp2f(sk2 - m) : 0.f;
+    bf16* dst = out + (size_t)tok * out_stride + (size_t)head * dv;
+    const float* po = part_o + at * dv;
+    for (int d0 = 0; d0 < dv; d0 += 4 * n) {   // up to four columns a thread at a time
+        float a[4] = {0.f, 0.f, 0.f, 0.f}, sum = l;
+        for (int s0 = 0; s0 < n_splits; s0 += AS_JOIN) {
+            const int ns = n_splits - s0 < AS_JOIN ? n_splits - s0 : AS_JOIN;
+            __syncthreads();                   // the last factors are no longer read
+            for (int s = tid; s < ns; s += n) {
+                const float2 ml = *(const float2*)(part_ml + (at + s0 + s) * 2);
+                const float w = ml.x != -INFINITY ? exp2f(ml.x - m) : 0.f;
+                s_w[s] = w;
+                s_l[s] = w != 0.f ? ml.y * w : 0.f;
+            }
+            __syncthreads();
+#pragma unroll 4
+            for (int s = 0; s < ns; ++s) {
+                const float w = s_w[s];
+                sum += s_l[s];
+                if (w != 0.f) {                // a share without a key has left its O unwritten or zero
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const int d = d0 + tid + k * n;
+                        if (d < dv) a[k] = fmaf(po[(size_t)(s0 + s) * dv + d], w, a[k]);
+                    }
+                }
+            }
         }
-        out[(size_t)tok * out_stride + (size_t)head * dv + d] = __float2bfloat16_rn(a * inv);
+        const float inv = sum > 0.f ? 1.f / sum : 0.f;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int d = d0 + tid + k * n;
+            if (d < dv) dst[d] = __float2bfloat16_rn(a[k] * inv);
+        }
     }
 }
 
@@ -1094,9 +1124,9 @@ static int launch_sink(const bf16* q, long long q_stride, bf16* out, long long o
         rc = launch_status();
     }
     if (rc || n_splits <= 1) return rc;
-    attention_sink_join_kernel<<<dim3(n_tiles, H), 64, 0, stream>>>(part_o, part_ml, positions, sinks, out,
-                                                                   out_stride, H, dv, n_splits);
-    return launch_status();
+    return tgo_launch_pdl(attention_sink_join_kernel, dim3(n_tiles, H), dim3(dv > 64 ? 128 : 64), 0, stream,
+                          (const float*)part_o, (const float*)part_ml, positions, sinks, out, out_stride, H, dv,
+                          n_splits);
 }
 
 // q [T, >= H dk] and out [T, >= H dv] bfloat16 views with unit column stride, 16-byte aligned
@@ -1166,9 +1196,9 @@ static int launch_sink_wide(const bf16* q, long long q_stride, bf16* out, long l
                             dk, dv, scale * AS_LOG2E, window, sinks, n_splits, part_o, part_ml, cap_log2,
                             scale_over_cap);
         if (rc || n_splits <= 1) return rc;
-        attention_sink_join_kernel<<<dim3(n_tiles, H), 128, 0, stream>>>(part_o, part_ml, positions, sinks, out,
-                                                                        out_stride, H, dv, n_splits);
-        return launch_status();
+        return tgo_launch_pdl(attention_sink_join_kernel, dim3(n_tiles, H), dim3(128), 0, stream,
+                              (const float*)part_o, (const float*)part_ml, positions, sinks, out, out_stride, H,
+                              dv, n_splits);
     }
     auto kernel = attention_sink_wide_kernel<DK, DV>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -1177,9 +1207,9 @@ static int launch_sink_wide(const bf16* q, long long q_stride, bf16* out, long l
                             positions, seq_ids, tile_tok0, tile_ntok, H, Hkv, dk, dv, scale * AS_LOG2E, window,
                             sinks, n_splits, part_o, part_ml, cap_log2, scale_over_cap);
     if (rc || n_splits <= 1) return rc;
-    attention_sink_join_kernel<<<dim3(n_tiles, H), 128, 0, stream>>>(part_o, part_ml, positions, sinks, out,
-                                                                    out_stride, H, dv, n_splits);
-    return launch_status();
+    return tgo_launch_pdl(attention_sink_join_kernel, dim3(n_tiles, H), dim3(128), 0, stream,
+                          (const float*)part_o, (const float*)part_ml, positions, sinks, out, out_stride, H, dv,
+                          n_splits);
 }
 
 // As tgo_attention_sink for key rows up to 576 wide whose first dv (up to 512) channels are the

@@ -125,7 +125,8 @@ TGO_API int tgo_rope_slice(const void* src, long long src_stride, int src_head, 
 // one head; a thread sums one output's k in ascending order for one or several tokens, so an
 // output's bits do not depend on what else is in the step. HL_N is 64, or 16 when that gives
 // too few blocks to fill the device (few tokens, few outputs a head). x, y: rows with unit
-// column stride. With `gate` ([T, H N] in the storage type, rows gate_stride apart) every output is
+// column stride. The 32-bit engine's form (the bfloat16 engine takes the library's batched
+// product). With `gate` ([T, H N] in the storage type, rows gate_stride apart) every output is
 // multiplied by the logistic function of its place in it (an output gate on the heads).
 __device__ __forceinline__ float hl_gated(float v, float g) { return v / (1.f + expf(-g)); }
 
@@ -222,18 +223,12 @@ TGO_API int tgo_head_linear(const void* x, long long x_stride, int x_head, const
                             long long y_stride, int y_head, int dtype, int T, int H, int N, int K,
                             const void* gate, long long gate_stride, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (H <= 0 || N <= 0 || K <= 0 || H > 65535) return TGO_E_BAD_ARG;
+    if (H <= 0 || N <= 0 || K <= 0 || H > 65535 || dtype != TGO_F32) return TGO_E_BAD_ARG;
     if (T <= 16 && K <= 32 * HLF_PER && (N + 7) / 8 <= 0x7fffffff) {
         const dim3 fgrid((N + 7) / 8, H), fblock(256);
-        if (dtype == TGO_BF16)
-            return tgo_launch_pdl(head_linear_few_kernel<bf16>, fgrid, fblock, 0, stream, (const bf16*)x, x_stride,
-                                  x_head, (const bf16*)w, (bf16*)y, y_stride, y_head, T, N, K,
-                                  (const bf16*)gate, gate_stride);
-        if (dtype == TGO_F32)
-            return tgo_launch_pdl(head_linear_few_kernel<float>, fgrid, fblock, 0, stream, (const float*)x,
+        return tgo_launch_pdl(head_linear_few_kernel<float>, fgrid, fblock, 0, stream, (const float*)x,
                                   x_stride, x_head, (const float*)w, (float*)y, y_stride, y_head, T, N, K,
-                                  (const float*)gate, gate_stride);
-        return TGO_E_BAD_ARG;
+                              (const float*)gate, gate_stride);
     }
     const long long blocks64 = (long long)((T + HL_TOK - 1) / HL_TOK) * H * ((N + 63) / 64);
     const int hn = blocks64 < 600 ? 16 : 64;
@@ -242,16 +237,9 @@ TGO_API int tgo_head_linear(const void* x, long long x_stride, int x_head, const
 #define HL_GO(TT, NN)                                                                                       \
     return tgo_launch_pdl(head_linear_kernel<TT, NN>, grid, block, 0, stream, (const TT*)x, x_stride, x_head, \
                           (const TT*)w, (TT*)y, y_stride, y_head, T, N, K, (const TT*)gate, gate_stride)
-    if (dtype == TGO_BF16) {
-        if (hn == 16) HL_GO(bf16, 16);
-        HL_GO(bf16, 64);
-    }
-    if (dtype == TGO_F32) {
-        if (hn == 16) HL_GO(float, 16);
-        HL_GO(float, 64);
-    }
+    if (hn == 16) HL_GO(float, 16);
+    HL_GO(float, 64);
 #undef HL_GO
-    return TGO_E_BAD_ARG;
 }
 
 // ------------------------------------------------- a product's head-major rows, into token rows

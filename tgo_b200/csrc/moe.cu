@@ -37,11 +37,14 @@
 #define MOE_TK 16
 
 // ------------------------------------------------------------------------------ logits
-// A warp takes one router row (an expert) and up to ML_TOK tokens, lanes over the width four
-// channels at a time; a block's eight warps share the tokens, so x comes from the first-level
-// cache after the first. The order of a sum depends on the width alone. out [T, rows]; the last
-// row may have no bias (the gate of a shared expert). Block 0 also zeroes the experts' counts.
+// A block takes ML_TOK tokens and ML_EXP router rows (experts); its eight warps share the width,
+// four channels a thread and 1024 a round, so that the loads of a few tokens are all in flight
+// at once. A warp's 32 sums are joined by a transposing exchange (lane i ends with pair i), the
+// warps' through shared memory in warp order: the order of a sum depends on the width alone.
+// out [T, rows]; the last row may have no bias (the gate of a shared expert). Block 0 also zeroes
+// the experts' counts.
 #define ML_TOK 8
+#define ML_EXP 4
 template <typename T> struct Load4;
 template <> struct Load4<bf16> {
     static __device__ __forceinline__ float4 get(const bf16* p) {
@@ -60,45 +63,71 @@ __global__ void __launch_bounds__(256)
 moe_logits_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ wr,
                   const float* __restrict__ br, int Tn, int d, int rows, int E, float* __restrict__ out,
                   int* __restrict__ counts, int E_real) {
+    __shared__ float s_part[8][32];
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (blockIdx.x == 0 && blockIdx.y == 0)
         for (int i = threadIdx.x; i < E_real; i += 256) counts[i] = 0;
-    const int e = blockIdx.y * 8 + warp, t0 = blockIdx.x * ML_TOK;
-    if (e >= rows) return;
-    const int nt = Tn - t0 < ML_TOK ? Tn - t0 : ML_TOK;
-    const float* w = wr + (size_t)e * d;
-    const T* xt = x + (size_t)t0 * x_stride;
-    float a[ML_TOK];
+    const int e0 = blockIdx.y * ML_EXP, t0 = blockIdx.x * ML_TOK;
+    // tokens and rows past the end repeat the last one: their sums are not stored
+    const T* xr[ML_TOK];
+    const float* w[ML_EXP];
 #pragma unroll
-    for (int j = 0; j < ML_TOK; ++j) a[j] = 0.f;
+    for (int j = 0; j < ML_TOK; ++j) xr[j] = x + (size_t)(t0 + j < Tn ? t0 + j : Tn - 1) * x_stride;
+#pragma unroll
+    for (int k = 0; k < ML_EXP; ++k) w[k] = wr + (size_t)(e0 + k < rows ? e0 + k : rows - 1) * d;
+    float a[32];                                         // a[4 j + k]: token j, row k
+#pragma unroll
+    for (int q = 0; q < 32; ++q) a[q] = 0.f;
     if (VEC) {
-#pragma unroll 4
-        for (int i = 4 * lane; i < d; i += 128) {
-            const float4 wv = *(const float4*)(w + i);
+        for (int i = 4 * threadIdx.x; i < d; i += 1024) {
+            float4 wv[ML_EXP], xv[ML_TOK];
+#pragma unroll
+            for (int k = 0; k < ML_EXP; ++k) wv[k] = *(const float4*)(w[k] + i);
+#pragma unroll
+            for (int j = 0; j < ML_TOK; ++j) xv[j] = Load4<T>::get(xr[j] + i);
 #pragma unroll
             for (int j = 0; j < ML_TOK; ++j)
-                if (j < nt) {
-                    const float4 xv = Load4<T>::get(xt + (size_t)j * x_stride + i);
-                    a[j] = fmaf(wv.x, xv.x, a[j]);
-                    a[j] = fmaf(wv.y, xv.y, a[j]);
-                    a[j] = fmaf(wv.z, xv.z, a[j]);
-                    a[j] = fmaf(wv.w, xv.w, a[j]);
+#pragma unroll
+                for (int k = 0; k < ML_EXP; ++k) {
+                    float v = a[4 * j + k];
+                    v = fmaf(wv[k].x, xv[j].x, v);
+                    v = fmaf(wv[k].y, xv[j].y, v);
+                    v = fmaf(wv[k].z, xv[j].z, v);
+                    a[4 * j + k] = fmaf(wv[k].w, xv[j].w, v);
                 }
         }
     } else {
-        for (int i = lane; i < d; i += 32) {
-            const float wv = w[i];
+        for (int i = threadIdx.x; i < d; i += 256) {
+            float wv[ML_EXP];
 #pragma unroll
-            for (int j = 0; j < ML_TOK; ++j)
-                if (j < nt) a[j] = fmaf(wv, to_f32(xt[(size_t)j * x_stride + i]), a[j]);
+            for (int k = 0; k < ML_EXP; ++k) wv[k] = w[k][i];
+#pragma unroll
+            for (int j = 0; j < ML_TOK; ++j) {
+                const float v = to_f32(xr[j][i]);
+#pragma unroll
+                for (int k = 0; k < ML_EXP; ++k) a[4 * j + k] = fmaf(wv[k], v, a[4 * j + k]);
+            }
         }
     }
-    const float bias = (br && e < E) ? br[e] : 0.f;
+    // 32 sums over 32 lanes: with each round a lane keeps half of its values, lane i ends with sum i
 #pragma unroll
-    for (int j = 0; j < ML_TOK; ++j) {
-        const float v = warp_sum(a[j]);
-        if (lane == 0 && j < nt) out[(size_t)(t0 + j) * rows + e] = v + bias;
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int q = 0; q < o; ++q) {
+            const float give = up ? a[q] : a[q + o], have = up ? a[q + o] : a[q];
+            a[q] = have + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+    s_part[warp][lane] = a[0];
+    __syncthreads();
+    if (warp == 0) {
+        float v = 0.f;
+#pragma unroll
+        for (int q = 0; q < 8; ++q) v += s_part[q][lane];
+        const int t = t0 + lane / 4, e = e0 + lane % 4;
+        if (t < Tn && e < rows) out[(size_t)t * rows + e] = v + ((br && e < E) ? br[e] : 0.f);
     }
 }
 
@@ -117,22 +146,22 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg,
     if (gate_out && lane == 0) gate_out[t] = 1.f / (1.f + expf(-lg[E]));
     float first = 0.f, sum = 0.f, mine = 0.f;
     int mine_e = 0;
-    // the largest of n values in shared memory and its index (ties: the lower index), the same
-    // in every lane; with nothing above -inf the index is `fallback`
-    auto largest = [&](const float* v, int n, int fallback, float& best) {
-        best = -INFINITY;
+    // the largest of n values in shared memory below `limit` and its index (ties: the lower index),
+    // the same in every lane; with nothing above -inf the index is `fallback`
+    auto largest = [&](const float* v, int n, int fallback, float limit, float& best) {
+        float mine_v = -INFINITY;
         int be = 0x7fffffff;
         for (int e = lane; e < n; e += 32) {
             const float x = v[e];
-            if (x > best) { best = x; be = e; }
+            if (x > mine_v && x < limit) { mine_v = x; be = e; }
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-            if (ov > best || (ov == best && oe < be)) { best = ov; be = oe; }
-        }
-        return be < n ? be : fallback;
+        // a float's bits, reordered so that they compare as integers
+        const unsigned raw = __float_as_uint(mine_v);
+        const unsigned key = (raw & 0x80000000u) ? ~raw : raw | 0x80000000u;
+        const unsigned top_key = __reduce_max_sync(0xffffffffu, key);
+        best = __uint_as_float((top_key & 0x80000000u) ? top_key & 0x7fffffffu : ~top_key);
+        const unsigned bi = __reduce_min_sync(0xffffffffu, key == top_key ? (unsigned)be : 0x7fffffffu);
+        return (int)bi < n ? (int)bi : fallback;
     };
     if (score_mode != 0) {
         // scores: the softmax over every logit, or each logit's logistic; the choice adds the correction
@@ -168,18 +197,9 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg,
             __syncwarp();
             // the weakest groups - keep runs go: mark the strongest with +inf, then close the others
             for (int j = 0; j < keep; ++j) {
-                float best = -INFINITY;
-                int bg = 0x7fffffff;
-                for (int g = lane; g < groups; g += 32) {
-                    const float v = gs[g];
-                    if (v < INFINITY && v > best) { best = v; bg = g; }
-                }
-#pragma unroll
-                for (int o = 16; o > 0; o >>= 1) {
-                    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-                    const int og = __shfl_xor_sync(0xffffffffu, bg, o);
-                    if (ov > best || (ov == best && og < bg)) { best = ov; bg = og; }
-                }
+                float best;
+                const int bg = largest(gs, groups, groups, INFINITY, best);
+                __syncwarp();                            // every lane has read gs
                 if (lane == 0 && bg < groups) gs[bg] = INFINITY;
                 __syncwarp();
             }
@@ -189,7 +209,7 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg,
         }
         for (int j = 0; j < top; ++j) {
             float best;
-            const int be = largest(lg, E, j, best);
+            const int be = largest(lg, E, j, INFINITY, best);
             const float w = sc[be];
             sum += w;
             if (lane == j) { mine = w; mine_e = be; }
@@ -206,7 +226,7 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg,
     }
     for (int j = 0; j < top; ++j) {
         float best;
-        const int be = largest(lg, E, j, best);
+        const int be = largest(lg, E, j, INFINITY, best);
         if (j == 0) first = best;
         const float w = expf(best - first);
         sum += w;
@@ -238,72 +258,64 @@ moe_pick_kernel(const float* __restrict__ logits, int rows, int Tn, int E, int t
 }
 
 // -------------------------------------------------------------------------------- plan
-// One block: offsets [E + 1], tiles (expert, first place, rows) and their count in tile_info[0];
-// the fill counters go back to zero. Experts are taken blockDim at a time, the places and tiles
-// before each by a running sum over the block. `scan` is 2 x blockDim ints of shared memory.
+// One warp: offsets [E + 1], tiles (expert, first place, rows) and their count in tile_info[0]; the
+// fill counters go back to zero. A lane takes a run of experts, the places and tiles before it by
+// a running sum over the lanes.
 __device__ __forceinline__ void moe_plan(const int* counts, int E, int* __restrict__ offsets, int* fill,
-                                         int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles,
-                                         int* scan) {
-    const int n = blockDim.x, i = threadIdx.x;
-    int at = 0, nt = 0;                                  // places and tiles of the experts before
-    for (int e0 = 0; e0 < E; e0 += n) {
-        const int e = e0 + i;
-        const int c = e < E ? counts[e] : 0, mine = (c + MOE_TM - 1) / MOE_TM;
-        int pc = c, pt = mine;                           // inclusive sums
-        for (int o = 1; o < n; o <<= 1) {
-            scan[i] = pc;
-            scan[n + i] = pt;
-            __syncthreads();
-            if (i >= o) { pc += scan[i - o]; pt += scan[n + i - o]; }
-            __syncthreads();
-        }
-        if (e < E) {
-            offsets[e] = at + pc - c;
-            fill[e] = 0;
-            for (int k = 0; k < mine; ++k) {
-                const int q = nt + pt - mine + k;
-                if (q < max_tiles) {
-                    tiles[3 * q] = e;
-                    tiles[3 * q + 1] = at + pc - c + k * MOE_TM;
-                    tiles[3 * q + 2] = c - k * MOE_TM < MOE_TM ? c - k * MOE_TM : MOE_TM;
-                }
-            }
-        }
-        scan[i] = pc;
-        scan[n + i] = pt;
-        __syncthreads();
-        at += scan[n - 1];
-        nt += scan[2 * n - 1];
-        __syncthreads();
+                                         int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles) {
+    const int lane = threadIdx.x & 31, per = (E + 31) / 32;
+    const int e_lo = lane * per < E ? lane * per : E, e_hi = e_lo + per < E ? e_lo + per : E;
+    int c = 0, nt = 0;
+    for (int e = e_lo; e < e_hi; ++e) {
+        c += counts[e];
+        nt += (counts[e] + MOE_TM - 1) / MOE_TM;
     }
-    if (i == 0) {
+    int at = c, tile = nt;                               // inclusive sums over the lanes
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, at, o), b = __shfl_up_sync(0xffffffffu, tile, o);
+        if (lane >= o) { at += a; tile += b; }
+    }
+    if (lane == 31) {
         offsets[E] = at;
-        tile_info[0] = nt < max_tiles ? nt : max_tiles;
+        tile_info[0] = tile < max_tiles ? tile : max_tiles;
+    }
+    at -= c;
+    tile -= nt;
+    for (int e = e_lo; e < e_hi; ++e) {
+        const int n = counts[e];
+        offsets[e] = at;
+        fill[e] = 0;
+        for (int r = 0; r < n; r += MOE_TM, ++tile) {
+            if (tile >= max_tiles) break;
+            tiles[3 * tile] = e;
+            tiles[3 * tile + 1] = at + r;
+            tiles[3 * tile + 2] = n - r < MOE_TM ? n - r : MOE_TM;
+        }
+        at += n;
     }
 }
 
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(32)
 moe_plan_kernel(const int* __restrict__ counts, int E, int* __restrict__ offsets, int* __restrict__ fill,
                 int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles) {
-    __shared__ int scan[512];
     pdl_wait();
-    moe_plan(counts, E, offsets, fill, tile_info, tiles, max_tiles, scan);
+    moe_plan(counts, E, offsets, fill, tile_info, tiles, max_tiles);
 }
 
 // A step of few tokens: pick, plan and scatter by one block, the counts and fill counters in
 // shared memory.
-#define MOE_FEW_WARPS 16
+#define MOE_FEW_WARPS 32
 __global__ void __launch_bounds__(32 * MOE_FEW_WARPS)
 moe_route_few_kernel(const float* __restrict__ logits, int rows, int Tn, int E, int top, int* __restrict__ ids,
                      float* __restrict__ wts, int score_mode, const float* __restrict__ correction, int E_real,
                      float* __restrict__ gate_out, int groups, int keep, int renorm, float route_scale,
                      int* __restrict__ offsets, int* __restrict__ perm, int* __restrict__ place,
                      int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles) {
-    extern __shared__ float smem[];                      // [warps][2 E + 1 + groups], counts, fill, scan
+    extern __shared__ float smem[];                      // [warps][2 E + 1 + groups], counts, fill
     const int per = 2 * E + 1 + groups;
     int* counts = (int*)(smem + (size_t)MOE_FEW_WARPS * per);
     int* fill = counts + E_real;
-    int* scan = fill + E_real;
     const int warp = threadIdx.x >> 5, n = 32 * MOE_FEW_WARPS;
     for (int i = threadIdx.x; i < E_real; i += n) counts[i] = 0;
     pdl_wait();
@@ -315,7 +327,7 @@ moe_route_few_kernel(const float* __restrict__ logits, int rows, int Tn, int E, 
         __syncwarp();
     }
     __syncthreads();                                     // ids are in memory for the whole block
-    moe_plan(counts, E_real, offsets, fill, tile_info, tiles, max_tiles, scan);
+    if (warp == 0) moe_plan(counts, E_real, offsets, fill, tile_info, tiles, max_tiles);
     __syncthreads();
     for (int p = threadIdx.x; p < Tn * top; p += n) {
         const int e = ids[p];
@@ -651,7 +663,7 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
         (dtype != TGO_BF16 && dtype != TGO_F32))
         return TGO_E_BAD_ARG;
     const int rows = E + (gate_out ? 1 : 0);
-    const dim3 lgrid((T + ML_TOK - 1) / ML_TOK, (rows + 7) / 8);
+    const dim3 lgrid((T + ML_TOK - 1) / ML_TOK, (rows + ML_EXP - 1) / ML_EXP);
     const bool vec = d % 4 == 0 && x_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)wr % 16 == 0;
 #define LOGITS_GO(TT, V)                                                                                    \
     tgo_launch_pdl(moe_logits_kernel<TT, V>, lgrid, dim3(256), 0, stream, (const TT*)x, x_stride, wr, br, T, d, \
@@ -661,7 +673,7 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
 #undef LOGITS_GO
     if (rc) return rc;
     const size_t per = (size_t)(2 * E + 1 + groups) * sizeof(float);
-    const size_t few = MOE_FEW_WARPS * per + (size_t)(2 * E_real + 64 * MOE_FEW_WARPS) * sizeof(int);
+    const size_t few = MOE_FEW_WARPS * per + (size_t)2 * E_real * sizeof(int);
     if (T <= MOE_FEW_TOKENS && few <= 200 * 1024) {
         if (few > 48 * 1024)
             cudaFuncSetAttribute(moe_route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)few);
@@ -679,7 +691,7 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
                         (const float*)logits, rows, T, E, top, ids, wts, counts, score_mode, correction, E_real,
                         gate_out, groups, keep, renorm, route_scale);
     if (rc) return rc;
-    rc = tgo_launch_pdl(moe_plan_kernel, dim3(1), dim3(256), 0, stream, (const int*)counts, E_real, offsets, fill,
+    rc = tgo_launch_pdl(moe_plan_kernel, dim3(1), dim3(32), 0, stream, (const int*)counts, E_real, offsets, fill,
                         tile_info, tiles, max_tiles);
     if (rc) return rc;
     const int pairs = T * top;

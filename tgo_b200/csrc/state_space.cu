@@ -51,12 +51,12 @@ causal_conv_act_kernel(const T* __restrict__ x, long long x_stride, const float*
     }
 }
 
-// The same with eight channels a thread (16-byte loads of x) and CV_TOK consecutive tokens, the
-// window of inputs in registers: for up to four taps, C, the row stride and x's address as
-// multiples of eight elements.
+// The same with eight channels a thread (16-byte loads of x) and TOK consecutive tokens, whose
+// rows are asked for before the first is used, the window of inputs in registers: for up to four
+// taps, C, the row stride and x's address as multiples of eight elements. `kept4`: the kept rows
+// can be read 16 bytes at a time. One token a thread where the step has only single tokens.
 #define CV_TOK 8
-__device__ __forceinline__ void cv_load(float* v, const bf16* p) {
-    const uint4 q = *(const uint4*)p;
+__device__ __forceinline__ void cv_widen(float* v, uint4 q) {
     const uint32_t* w = (const uint32_t*)&q;
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
@@ -64,6 +64,11 @@ __device__ __forceinline__ void cv_load(float* v, const bf16* p) {
         v[2 * k] = f.x;
         v[2 * k + 1] = f.y;
     }
+}
+__device__ __forceinline__ void cv_load8(float* v, const float* p) {
+    const float4 a = *(const float4*)p, b = *(const float4*)(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 __device__ __forceinline__ void cv_store(bf16* p, const float* v) {
     uint4 q;
@@ -80,36 +85,52 @@ __device__ __forceinline__ void cv_store(float* p, const float* v) {
     *(float4*)(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
 }
 
-template <typename TY, int TAPS>
+template <typename TY, int TAPS, int TOK>
 __global__ void __launch_bounds__(128)
 causal_conv_act_x8_kernel(const bf16* __restrict__ x, long long x_stride, const float* __restrict__ w,
                           const float* __restrict__ bias, TY* __restrict__ y, int Tn, int C,
                           const int* __restrict__ seq_ids, const int* __restrict__ q_start,
                           const int* __restrict__ state_slots, const float* __restrict__ state,
-                          long long state_stride, long long conv_offset) {
+                          long long state_stride, long long conv_offset, int kept4) {
     pdl_wait();
-    const int c = 8 * (blockIdx.y * blockDim.x + threadIdx.x), t_lo = blockIdx.x * CV_TOK;
+    const int c = 8 * (blockIdx.y * blockDim.x + threadIdx.x), t_lo = blockIdx.x * TOK;
     if (c >= C) return;
-    float wt[TAPS][8], bs[8], win[TAPS][8];              // win[j] meets wt[j]; the last is the token's own
+    uint4 rows[TOK];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        bs[i] = bias ? bias[c + i] : 0.f;
+    for (int u = 0; u < TOK; ++u)
+        rows[u] = *(const uint4*)(x + (size_t)(t_lo + u < Tn ? t_lo + u : Tn - 1) * x_stride + c);
+    float wt[8 * TAPS], bs[8], win[TAPS][8];             // win[j] meets tap j; the last is the token's own
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) wt[j][i] = w[(size_t)(c + i) * TAPS + j];
+    for (int q = 0; q < TAPS; ++q) cv_load8(wt + 8 * q, w + (size_t)c * TAPS + 8 * q);    // [channel][tap]
+    if (bias) {
+        cv_load8(bs, bias + c);
+    } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) bs[i] = 0.f;
     }
-    const int t_hi = t_lo + CV_TOK < Tn ? t_lo + CV_TOK : Tn;
-    for (int t = t_lo; t < t_hi; ++t) {
-        const int b = seq_ids[t], r = t - q_start[b];
-        if (t == t_lo || r == 0) {                       // a window from the start: rows of the step, then kept ones
+    int q_at = -1, first = 0;
+#pragma unroll
+    for (int u = 0; u < TOK; ++u) {
+        const int t = t_lo + u;
+        if (t >= Tn) break;
+        const int b = seq_ids[t];
+        if (u == 0 || b != q_at) {                       // a window from the start: rows of the step, then kept ones
+            q_at = b;
+            first = q_start[b];
             const float* kept = state + (size_t)state_slots[b] * state_stride + conv_offset;
 #pragma unroll
             for (int j = 0; j < TAPS - 1; ++j) {
-                const int back = TAPS - 1 - j;
+                const int back = TAPS - 1 - j, r = t - first;
                 if (back <= r) {
-                    cv_load(win[j], x + (size_t)(t - back) * x_stride + c);
+                    cv_widen(win[j], *(const uint4*)(x + (size_t)(t - back) * x_stride + c));
                 } else {
+                    const float* k = kept + (size_t)(TAPS - 1 - (back - r)) * C + c;
+                    if (kept4) {
+                        cv_load8(win[j], k);
+                    } else {
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) win[j][i] = kept[(size_t)(TAPS - 1 - (back - r)) * C + c + i];
+                        for (int i = 0; i < 8; ++i) win[j][i] = k[i];
+                    }
                 }
             }
         } else {
@@ -118,13 +139,13 @@ causal_conv_act_x8_kernel(const bf16* __restrict__ x, long long x_stride, const 
 #pragma unroll
                 for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
         }
-        cv_load(win[TAPS - 1], x + (size_t)t * x_stride + c);
+        cv_widen(win[TAPS - 1], rows[u]);
         float o[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             float a = bs[i];
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) a = fmaf(wt[j][i], win[j][i], a);
+            for (int j = 0; j < TAPS; ++j) a = fmaf(wt[i * TAPS + j], win[j][i], a);
             o[i] = __fdividef(a, 1.f + __expf(-a));
         }
         cv_store(y + (size_t)t * C + c, o);
@@ -170,13 +191,16 @@ TGO_API int tgo_causal_conv_act(const void* x, long long x_stride, int dtype, co
     tgo_launch_pdl(causal_conv_act_kernel<TT, TY>, dim3(T, cy), dim3(256), 0, stream, (const TT*)x, x_stride, w, \
                    bias, (TY*)y, C, taps, seq_ids, q_start, state_slots, (const float*)state, state_stride, \
                    conv_offset)
-#define CONV_X8(TY, TAPS)                                                                                  \
-    tgo_launch_pdl(causal_conv_act_x8_kernel<TY, TAPS>, dim3((T + CV_TOK - 1) / CV_TOK, (C / 8 + 127) / 128),      \
+    const int kept4 = state_stride % 4 == 0 && conv_offset % 4 == 0 && (uintptr_t)state % 16 == 0;
+#define CONV_X8_AT(TY, TAPS, TOK)                                                                          \
+    tgo_launch_pdl(causal_conv_act_x8_kernel<TY, TAPS, TOK>, dim3((T + TOK - 1) / TOK, (C / 8 + 127) / 128),       \
                    dim3(128), 0, stream, (const bf16*)x, x_stride, w, bias, (TY*)y, T, C, seq_ids, q_start,      \
-                   state_slots, (const float*)state, state_stride, conv_offset)
+                   state_slots, (const float*)state, state_stride, conv_offset, kept4)
+#define CONV_X8(TY, TAPS) (T == B ? CONV_X8_AT(TY, TAPS, 1) : CONV_X8_AT(TY, TAPS, CV_TOK))
 #define CONV_TAPS(TY) (taps == 1 ? CONV_X8(TY, 1) : taps == 2 ? CONV_X8(TY, 2) : taps == 3 ? CONV_X8(TY, 3) : CONV_X8(TY, 4))
     if (dtype == TGO_BF16 && (y_dtype == TGO_F32 || y_dtype == TGO_BF16) && taps <= 4 && C % 8 == 0 &&
-        x_stride % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0)
+        x_stride % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+        (uintptr_t)bias % 16 == 0)
         rc = y_dtype == TGO_F32 ? CONV_TAPS(float) : CONV_TAPS(bf16);
     else if (dtype == TGO_BF16 && y_dtype == TGO_F32) rc = CONV_GO(bf16, float);
     else if (dtype == TGO_BF16 && y_dtype == TGO_BF16) rc = CONV_GO(bf16, bf16);
@@ -184,6 +208,7 @@ TGO_API int tgo_causal_conv_act(const void* x, long long x_stride, int dtype, co
     else return TGO_E_BAD_ARG;
 #undef CONV_GO
 #undef CONV_X8
+#undef CONV_X8_AT
 #undef CONV_TAPS
     if (rc || taps == 1 || !keep) return rc;
     if (dtype == TGO_BF16)
@@ -564,9 +589,8 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
             s_c[(k & 1) * CS_TOK * NP + tid + CS_HALF * i] = to_f32(cn[i]);
         }
     };
-    auto finish = [&](int k) {                           // the walked tile k: gate and store
-        const float* ys = s_y + (k & 1) * CS_TOK * (CH + 1);
-        T xr[PER], zr[PER];
+    T xr[PER], zr[PER];
+    auto recall = [&](int k) {                           // x and z of a walked tile, ahead of their use
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int r = k * CS_TOK + lt + RSTEP * i;
@@ -574,6 +598,9 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
             xr[i] = ok ? x[(size_t)(t0 + r) * x_stride + lc] : zero;
             zr[i] = ok ? z[(size_t)(t0 + r) * z_stride + lc] : zero;
         }
+    };
+    auto finish = [&](int k) {                           // the walked tile k: gate and store
+        const float* ys = s_y + (k & 1) * CS_TOK * (CH + 1);
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int r = lt + RSTEP * i;
@@ -587,12 +614,16 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
     if (n_tiles > 1) fetch(1);
     __syncthreads();
     for (int k = 0; k < n_tiles; ++k) {
+        if (k > 0) recall(k - 1);
         if (k + 1 < n_tiles) stage(k + 1);
         if (k + 2 < n_tiles) fetch(k + 2);
         if (k > 0) finish(k - 1);
         __syncthreads();
     }
-    if (n_tiles > 0) finish(n_tiles - 1);
+    if (n_tiles > 0) {
+        recall(n_tiles - 1);
+        finish(n_tiles - 1);
+    }
     if (conv_in && tid < CH && c0 + tid < C)
         cs_keep(row + conv_offset, conv_in, conv_in_stride, c0 + tid, C, taps, t0, n_tok);
 }

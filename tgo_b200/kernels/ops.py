@@ -855,27 +855,22 @@ def rope_slice(src: torch.Tensor, src_head: int, src_off: int, dst: torch.Tensor
         c_int(1 if interleaved else 0), _stream()), "rope_slice")
 
 
-HEAD_LINEAR_LIBRARY_ROWS = 65     # bfloat16 steps of this many rows or more: the library's
-                                  # batched product
-
-
 def head_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, y: torch.Tensor, y_head: int,
                 gate: Optional[torch.Tensor] = None) -> None:
     """A product per head: y[t, h * y_head + n] = sum_k x[t, h * x_head + k] w[h, n, k], with
     w [H, N, K]; x and y 2-D views with unit column stride. With `gate` (a 2-D view [T, H N] in
     x's type) every output is multiplied by the logistic function of gate[t, h * N + n].
-    float32, and bfloat16 with few
-    rows: this package's kernels (up to 16 rows and K up to 512: a warp an output, the lanes'
-    partial sums joined in a fixed order; else tiles, k summed in order); bfloat16 with many
-    rows: the library's batched product, where the dense products of as many rows take the
-    library too."""
+    bfloat16: the library's batched product, straight into y (at 16 heads of 128 x 512 it takes 9
+    to 11 us for 1 to 128 rows where this package's kernels take 12 to 54). float32: this
+    package's kernels (up to 16 rows and K up to 512: a warp an output, the lanes' partial sums
+    joined in a fixed order; else tiles, k summed in order)."""
     _need_cuda(x, w, y, gate)
     T = x.shape[0]
     H, N, K = w.shape
     assert gate is None or (gate.shape == (T, H * N) and gate.stride(1) == 1 and gate.dtype == x.dtype)
     assert w.is_contiguous() and x.stride(1) == 1 and y.stride(1) == 1
     assert x.dtype == w.dtype == y.dtype and y.shape[0] == T
-    if x.dtype == torch.bfloat16 and T >= HEAD_LINEAR_LIBRARY_ROWS:
+    if x.dtype == torch.bfloat16:
         xv = torch.as_strided(x, (H, T, K), (x_head, x.stride(0), 1))
         if gate is not None:
             lib = load_library("latent")
@@ -884,8 +879,7 @@ def head_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, y: torch.Tensor, 
                                           c_int(dtype_code(y.dtype)), c_int(T), c_int(H), c_int(N),
                                           _ptr(gate), c_ll(gate.stride(0)), _stream()), "head_rows_gate")
             return
-        yv = torch.as_strided(y, (H, T, N), (y_head, y.stride(0), 1))
-        yv.copy_(torch.bmm(xv, w.transpose(1, 2)))
+        torch.bmm(xv, w.transpose(1, 2), out=torch.as_strided(y, (H, T, N), (y_head, y.stride(0), 1)))
         return
     lib = load_library("latent")
     _check(lib.tgo_head_linear(_ptr(x), c_ll(x.stride(0)), c_int(x_head), _ptr(w), _ptr(y),
@@ -901,9 +895,9 @@ def causal_conv_act(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tenso
                     keep: bool = True) -> None:
     """y = silu(bias + causal convolution of x per channel): x a 2-D view [T, C] in the
     activation type, w float32 [C, taps] (the last column meets the current token), y [T, C]
-    float32 or in the activation type. The inputs before a request's portion come from its state row (float32
-    [slots, n]; the last taps - 1 inputs [taps - 1, C] at `conv_offset`), which is then moved
-    on by the step's inputs, unless `keep` is False (`channel_scan` moves them on)."""
+    float32 or in the activation type. The inputs before a request's portion come from its state
+    row (float32 [slots, n]; the last taps - 1 inputs [taps - 1, C] at `conv_offset`), which is
+    then moved on by the step's inputs, unless `keep` is False (`channel_scan` moves them on)."""
     _need_cuda(x, w, bias, y, seq_ids, q_start, state_slots, state)
     T, C = x.shape
     taps = w.shape[1]
