@@ -404,21 +404,22 @@ TGO_API int tgo_selective_scan(const float* xbc, int C, const void* dt_raw, long
 }
 
 // ---------------------------------------------------------------------- scan per channel
-// A block per (request, CS_CH channels) in two halves that work on different tiles of CS_TOK
-// tokens at the same time. The walking half: L lanes share a channel and lane l keeps states
+// A block per (request, CS_WALK / L channels) whose threads have two roles and work on different
+// tiles of TOK tokens at the same time. The walking warps: L lanes share a channel and lane l keeps states
 // l * NS .. l * NS + NS - 1 of it in registers for the whole walk over the request's tokens. Four
 // tokens are taken together: their decays do not depend on the state, so only one FMA per state
 // and token is a chain, and the four sums over n are joined by a transposing exchange in the
 // quad (three shuffles for four tokens) and, for L > 4, by shuffles over the quads, the same
 // order for every token. Tokens past the end of a tile have dt = 0 and leave the state as it is.
-// The serving half: while tile k is walked it puts tile k + 1 into shared memory (dt through
+// The serving warps: while tile k is walked it puts tile k + 1 into shared memory (dt through
 // softplus once per (token, channel), beside dt * x; B and C as float32 rows), asks for tile
 // k + 2's inputs, and finishes tile k - 1 (D x added, times silu(z), stored). `a2` is A log2(e).
 //
 // The walk ends with the convolution's kept inputs: the last taps - 1 of (kept, then the
 // step's raw inputs `conv_in`), which the convolution has read before this kernel starts.
-#define CS_TOK 32
-#define CS_HALF 128
+#define CS_WALK 128              // walking threads
+// serving threads: 256 where a tile has a (token, channel) pair for each, else 128
+#define CS_SERVE(TOK, L) ((TOK) * (CS_WALK / (L)) % 256 == 0 ? 256 : 128)
 
 // One step of one state: 2^e S + add. A state that decays slowly is multiplied by nearly 1
 // thousands of times, and an exponential that is off by the same fraction of a unit in the last
@@ -462,8 +463,8 @@ __device__ __forceinline__ void cs_keep(float* kept, const T* __restrict__ conv_
     }
 }
 
-template <typename T, int L, int NS>
-__global__ void __launch_bounds__(2 * CS_HALF)
+template <typename T, int L, int NS, int TOK>
+__global__ void __launch_bounds__(CS_WALK + CS_SERVE(TOK, L))
 channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ z, long long z_stride,
                     const float* __restrict__ dt_raw, long long dt_stride, const float* __restrict__ dt_bias,
                     const float* __restrict__ a2, const T* __restrict__ bm, const T* __restrict__ cm,
@@ -471,22 +472,24 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
                     const int* __restrict__ q_start, const int* __restrict__ state_slots,
                     float* __restrict__ state, long long state_stride, long long ssm_offset,
                     const T* __restrict__ conv_in, long long conv_in_stride, int taps, long long conv_offset) {
-    constexpr int CH = CS_HALF / L;                      // channels of this block
+    constexpr int CH = CS_WALK / L;                      // channels of this block
     constexpr int NP = L * NS;                           // N rounded up
-    constexpr int PER = CS_TOK * CH / CS_HALF;           // (token, channel) pairs a serving thread loads
-    constexpr int RSTEP = CS_HALF / CH;                  // tokens between a thread's pairs (= L)
-    constexpr int PBC = CS_TOK * NP / CS_HALF;
+    constexpr int SERVE = CS_SERVE(TOK, L);
+    constexpr int PER = TOK * CH / SERVE;                // (token, channel) pairs a serving thread loads
+    constexpr int RSTEP = SERVE / CH;                 // tokens between a thread's pairs
+    constexpr int PBC = TOK * NP / SERVE;
+    static_assert(TOK * CH % SERVE == 0 && TOK * NP % SERVE == 0, "tile");
     extern __shared__ __align__(16) float cs_smem[];
-    float* s_b = cs_smem;                                // [2][CS_TOK][NP]
-    float* s_c = s_b + 2 * CS_TOK * NP;                  // [2][CS_TOK][NP]
-    float2* s_dt = (float2*)(s_c + 2 * CS_TOK * NP);     // [2][CS_TOK][CH + 1]: dt, dt x
-    float* s_y = (float*)(s_dt + 2 * CS_TOK * (CH + 1)); // [2][CS_TOK][CH + 1]
+    float* s_b = cs_smem;                                // [2][TOK][NP]
+    float* s_c = s_b + 2 * TOK * NP;                  // [2][TOK][NP]
+    float2* s_dt = (float2*)(s_c + 2 * TOK * NP);     // [2][TOK][CH + 1]: dt, dt x
+    float* s_y = (float*)(s_dt + 2 * TOK * (CH + 1)); // [2][TOK][CH + 1]
     pdl_wait();
     const int b = blockIdx.x, c0 = blockIdx.y * CH;
     const int t0 = q_start[b], n_tok = q_start[b + 1] - t0;
-    const int n_tiles = (n_tok + CS_TOK - 1) / CS_TOK;
+    const int n_tiles = (n_tok + TOK - 1) / TOK;
     float* row = state + (size_t)state_slots[b] * state_stride;
-    if (threadIdx.x < CS_HALF) {
+    if (threadIdx.x < CS_WALK) {
         // ---- walking
         const int tid = threadIdx.x;
         const int lane_l = tid % L, wch = tid / L, wc = c0 + wch, n0 = lane_l * NS;
@@ -501,12 +504,11 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
         const bool odd = tid & 1, high = tid & 2;
         __syncthreads();                                 // tile 0 is in shared memory
         for (int k = 0; k < n_tiles; ++k) {
-            const int nt = n_tok - k * CS_TOK < CS_TOK ? n_tok - k * CS_TOK : CS_TOK;
-            const float2* dts = s_dt + (k & 1) * CS_TOK * (CH + 1) + wch;
-            const float* bs = s_b + (k & 1) * CS_TOK * NP + n0;
-            const float* cs = s_c + (k & 1) * CS_TOK * NP + n0;
-            float* ys = s_y + (k & 1) * CS_TOK * (CH + 1) + wch;
-#pragma unroll 2
+            const int nt = n_tok - k * TOK < TOK ? n_tok - k * TOK : TOK;
+            const float2* dts = s_dt + (k & 1) * TOK * (CH + 1) + wch;
+            const float* bs = s_b + (k & 1) * TOK * NP + n0;
+            const float* cs = s_c + (k & 1) * TOK * NP + n0;
+            float* ys = s_y + (k & 1) * TOK * (CH + 1) + wch;
             for (int r = 0; r < nt; r += 4) {
                 float part[4];
 #pragma unroll
@@ -549,7 +551,7 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
         return;
     }
     // ---- serving: channel lc, tokens lt + RSTEP i of a tile
-    const int tid = threadIdx.x - CS_HALF;
+    const int tid = threadIdx.x - CS_WALK;
     const int lcl = tid % CH, lc = c0 + lcl, lt = tid / CH;
     const bool lok = lc < C;
     const float bias = (lok && dt_bias) ? dt_bias[lc] : 0.f;
@@ -560,7 +562,7 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
     auto fetch = [&](int k) {
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
-            const int r = k * CS_TOK + lt + RSTEP * i;
+            const int r = k * TOK + lt + RSTEP * i;
             const bool ok = lok && r < n_tok;
             const size_t t = (size_t)(t0 + r);
             xn[i] = ok ? x[t * x_stride + lc] : zero;
@@ -568,44 +570,44 @@ channel_scan_kernel(const T* __restrict__ x, long long x_stride, const T* __rest
         }
 #pragma unroll
         for (int i = 0; i < PBC; ++i) {
-            const int q = tid + CS_HALF * i;
-            const int r = k * CS_TOK + q / NP, n = q % NP;
+            const int q = tid + SERVE * i;
+            const int r = k * TOK + q / NP, n = q % NP;
             const bool ok = n < N && r < n_tok;
             bn[i] = ok ? bm[(size_t)(t0 + r) * bc_stride + n] : zero;
             cn[i] = ok ? cm[(size_t)(t0 + r) * bc_stride + n] : zero;
         }
     };
     auto stage = [&](int k) {                            // what fetch(k) has brought
-        float2* dts = s_dt + (k & 1) * CS_TOK * (CH + 1);
+        float2* dts = s_dt + (k & 1) * TOK * (CH + 1);
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int r = lt + RSTEP * i;
-            const float dt = k * CS_TOK + r < n_tok ? cs_softplus<T>(dn[i] + bias) : 0.f;
+            const float dt = k * TOK + r < n_tok ? cs_softplus<T>(dn[i] + bias) : 0.f;
             dts[r * (CH + 1) + lcl] = make_float2(dt, dt * to_f32(xn[i]));
         }
 #pragma unroll
         for (int i = 0; i < PBC; ++i) {
-            s_b[(k & 1) * CS_TOK * NP + tid + CS_HALF * i] = to_f32(bn[i]);
-            s_c[(k & 1) * CS_TOK * NP + tid + CS_HALF * i] = to_f32(cn[i]);
+            s_b[(k & 1) * TOK * NP + tid + SERVE * i] = to_f32(bn[i]);
+            s_c[(k & 1) * TOK * NP + tid + SERVE * i] = to_f32(cn[i]);
         }
     };
     T xr[PER], zr[PER];
     auto recall = [&](int k) {                           // x and z of a walked tile, ahead of their use
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
-            const int r = k * CS_TOK + lt + RSTEP * i;
+            const int r = k * TOK + lt + RSTEP * i;
             const bool ok = lok && r < n_tok;
             xr[i] = ok ? x[(size_t)(t0 + r) * x_stride + lc] : zero;
             zr[i] = ok ? z[(size_t)(t0 + r) * z_stride + lc] : zero;
         }
     };
     auto finish = [&](int k) {                           // the walked tile k: gate and store
-        const float* ys = s_y + (k & 1) * CS_TOK * (CH + 1);
+        const float* ys = s_y + (k & 1) * TOK * (CH + 1);
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int r = lt + RSTEP * i;
-            if (lok && k * CS_TOK + r < n_tok)
-                y[(size_t)(t0 + k * CS_TOK + r) * C + lc] =
+            if (lok && k * TOK + r < n_tok)
+                y[(size_t)(t0 + k * TOK + r) * C + lc] =
                     from_f32<T>(fmaf(skip, to_f32(xr[i]), ys[r * (CH + 1) + lcl]) * cs_silu<T>(to_f32(zr[i])));
         }
     };
@@ -705,7 +707,7 @@ static int launch_channel_scan(const void* x, long long x_stride, const void* z,
                                int B, int C, int N, const int* q_start, const int* state_slots, float* state,
                                long long state_stride, long long ssm_offset, const void* conv_in,
                                long long conv_in_stride, int taps, long long conv_offset, cudaStream_t stream) {
-    constexpr int CH = CS_HALF / L, NP = L * NS;
+    constexpr int CH = CS_WALK / L, NP = L * NS;
 #define CS_LAUNCH(KERNEL, GRID, BLOCK, SMEM)                                                                  \
     tgo_launch_pdl(KERNEL, GRID, dim3(BLOCK), SMEM, stream, (const T*)x, x_stride, (const T*)z, z_stride,     \
                    dt_raw, dt_stride, dt_bias, a2, (const T*)bm, (const T*)cm, bc_stride, D, (T*)y, C, N, q_start, \
@@ -717,10 +719,11 @@ static int launch_channel_scan(const void* x, long long x_stride, const void* z,
         if (vec) return CS_LAUNCH((channel_scan_single_kernel<T, L, NS, true>), grid, 128, 0);
         return CS_LAUNCH((channel_scan_single_kernel<T, L, NS, false>), grid, 128, 0);
     }
-    const size_t smem = (size_t)2 * CS_TOK * (2 * NP + 3 * (CH + 1)) * sizeof(float);
-    auto kernel = channel_scan_kernel<T, L, NS>;
+    constexpr int TOK = NP <= 32 ? 64 : 32;              // tokens a tile: what shared memory has room for
+    const size_t smem = (size_t)2 * TOK * (2 * NP + 3 * (CH + 1)) * sizeof(float);
+    auto kernel = channel_scan_kernel<T, L, NS, TOK>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return CS_LAUNCH(kernel, dim3(B, (C + CH - 1) / CH), 2 * CS_HALF, smem);
+    return CS_LAUNCH(kernel, dim3(B, (C + CH - 1) / CH), CS_WALK + CS_SERVE(TOK, L), smem);
 #undef CS_LAUNCH
 }
 
