@@ -80,14 +80,14 @@ def _scan_case(c, N, taps, n, rng):
                                       (14, 256, 2)])
 def test_convolution_and_channel_scan_over_portions(c, N, taps, dtype):
     """Three requests in one batch, cut into portions that end before, on and after the kernel's
-    groups of 4 and tiles of 32 tokens (single tokens among them), their states in slots given
+    groups of 4 and tiles of 32 or 64 tokens (single tokens among them), their states in slots given
     out of order between rows of NaN; against the plain convolution and scan of the whole
     sequences. Decays from nearly none to nearly all; the loud first token shows a state that is
     lost on the way."""
     from tgo_b200.kernels import ops
     rng = np.random.default_rng(c + N)
-    lens = (103, 33, 1)
-    cuts = [[31, 1, 1, 2, 4, 32, 5, 27], [1, 5, 1, 26], [1]]
+    lens = (206, 33, 1)
+    cuts = [[31, 1, 1, 2, 4, 64, 65, 33, 5], [1, 5, 1, 26], [1]]
     data = [_scan_case(c, N, taps, n, rng) for n in lens]
     w, bias = rng.normal(size=(c, taps)) * 0.6, rng.normal(size=c) * 0.2
     dt_bias, D = rng.normal(size=c) - 1.0, rng.normal(size=c)
