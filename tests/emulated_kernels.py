@@ -31,6 +31,20 @@ def add_rmsnorm(h, delta, gain, eps, out, rows=None):
     out.copy_(((x * scale) * gain).to(out.dtype))
 
 
+def embed_rmsnorm(table, ids, gain, eps, out, copy=None, scale=1.0):
+    embed(table, ids, out, scale)
+    out.copy_(out * torch.rsqrt((out * out).mean(-1, keepdim=True) + eps) * gain)
+    if copy is not None:
+        copy.copy_(out)
+
+
+def norm_add_norm(h, y, gain_y, eps_y, gain, eps, out, extra=None):
+    h += y * torch.rsqrt((y * y).mean(-1, keepdim=True) + eps_y) * gain_y
+    if extra is not None:
+        h += extra
+    out.copy_((h * torch.rsqrt((h * h).mean(-1, keepdim=True) + eps) * gain).to(out.dtype))
+
+
 def add_layernorm(h, delta, gain, bias, eps, out, rows=None):
     if rows is None:
         if delta is not None:
@@ -100,7 +114,7 @@ def qk_norm_rope_cache(q, k, v, num_heads, num_kv_heads, head_dim, q_gain, k_gai
 
 def attention_generic(q, out, num_heads, num_kv_heads, head_dim, k_cache, v_cache, page_size,
                       block_tables, seq_ids, positions, scale, window, value_dim=None, sinks=None,
-                      softcap=0.0, value_row=0, keep_first=0, dist_bias=None):
+                      softcap=0.0, value_row=0, keep_first=0, dist_bias=None, gate=None):
     T = q.shape[0]
     group = num_heads // num_kv_heads
     dv = value_dim or head_dim
@@ -130,7 +144,10 @@ def attention_generic(q, out, num_heads, num_kv_heads, head_dim, k_cache, v_cach
                 w = torch.softmax(torch.cat([s, sinks[h:h + 1].float()]), dim=0)[:-1]
             else:
                 w = torch.softmax(s, dim=0)
-            out[t, h * dv:(h + 1) * dv] = (w @ V).to(out.dtype)
+            o = w @ V
+            if gate is not None:
+                o = o * torch.sigmoid(gate[t, h].float())
+            out[t, h * dv:(h + 1) * dv] = o.to(out.dtype)
 
 
 def paged_attention(q, out, num_heads, num_kv_heads, head_dim, cache, ctx, scale, window):
@@ -455,6 +472,59 @@ def selective_scan(xbc, dt_raw, dt_bias, a_log, d_skip, y, num_seqs, heads, grou
             y[t] = out.reshape(-1)
 
 
+def delta_prepare(x, w, b_raw, a_raw, dt_bias, decay, num_seqs, heads, groups, key_dim, value_dim, seq_ids,
+                  q_start, state_slots, state, conv_offset):
+    T, C = x.shape
+    rows = torch.empty((T, C), dtype=torch.float32)
+    causal_conv_act(x, w.t().contiguous(), None, rows, num_seqs, seq_ids, q_start, state_slots, state, conv_offset,
+                    keep=False)
+    kw = groups * key_dim
+    qk = torch.zeros((T, groups, 2, (key_dim + 31) // 32 * 32))
+    for j in range(2):
+        z = rows[:, j * kw:(j + 1) * kw].reshape(T, groups, key_dim)
+        qk[:, :, j, :key_dim] = z * torch.rsqrt((z * z).sum(-1, keepdim=True) + 1e-6) * \
+            (key_dim ** -0.5 if j == 0 else 1.0)
+    log_g = -decay * torch.nn.functional.softplus(a_raw.float() + dt_bias, threshold=1e9)
+    gates = torch.stack([torch.exp(log_g), torch.expm1(log_g), torch.sigmoid(b_raw.float()),
+                         torch.zeros_like(log_g)], dim=2).contiguous()
+    pairs = torch.zeros((T, groups, 4))              # of use to the kernels' pairs of tokens only
+    return qk, rows[:, 2 * kw:].contiguous(), gates, pairs
+
+
+def delta_scan(prepared, y, num_seqs, heads, groups, key_dim, value_dim, q_start, state_slots, state, mem_offset,
+               conv_in, taps, conv_offset):
+    qk, v, gates, _ = prepared
+    per, C = heads // groups, conv_in.shape[1]
+    for b in range(num_seqs):
+        t0, t1 = int(q_start[b]), int(q_start[b + 1])
+        row = state[int(state_slots[b])]
+        S = row[mem_offset:mem_offset + heads * key_dim * value_dim].view(heads, key_dim, value_dim)
+        for t in range(t0, t1):
+            q, k = (qk[t, :, j, :key_dim].repeat_interleave(per, dim=0) for j in range(2))
+            g, beta = gates[t, :, 0], gates[t, :, 2]
+            S.mul_(g[:, None, None])
+            u = beta[:, None] * (v[t].reshape(heads, value_dim) - torch.einsum("hkv,hk->hv", S, k))
+            S.add_(k[:, :, None] * u[:, None, :])
+            y[t] = torch.einsum("hkv,hk->hv", S, q).reshape(-1)
+        keep = taps - 1
+        if keep:
+            kept = row[conv_offset:conv_offset + keep * C].view(keep, C)
+            full = torch.cat([kept.clone(), conv_in[t0:t1].float()])
+            kept.copy_(full[full.shape[0] - keep:])
+
+
+def delta_step_supports(heads, groups, key_dim, value_dim, state, mem_offset):
+    return value_dim % 4 == 0
+
+
+def delta_step(prepared, z, gain, eps, out, num_seqs, heads, groups, key_dim, value_dim, q_start, state_slots,
+               state, mem_offset, conv_in, taps, conv_offset):
+    y = torch.empty(z.shape, dtype=torch.float32)
+    delta_scan(prepared, y, num_seqs, heads, groups, key_dim, value_dim, q_start, state_slots, state, mem_offset,
+               conv_in, taps, conv_offset)
+    gated_group_norm(y, z, gain.repeat(heads), out, heads, eps, "silu", False)
+
+
 def _plain_act(z, activation):
     if activation == "relu_squared":
         return torch.relu(z) ** 2
@@ -467,7 +537,7 @@ def _plain_act(z, activation):
 
 def moe_feed_forward(x, w_router, b_router, w_gate, w_up, w_down, top, activation, extra=None,
                      scores="chosen", correction=None, identity=0, extra_gated=False, groups=1, keep=1,
-                     renormalize=True, route_scale=1.0, beside=None, residual=None):
+                     renormalize=True, route_scale=1.0, beside=None, residual=None, group_best=2):
     T, d = x.shape
     E = w_up.shape[0]
     outputs = E + identity
@@ -481,7 +551,7 @@ def moe_feed_forward(x, w_router, b_router, w_gate, w_up, w_down, top, activatio
             choice = sc + (correction if correction is not None else 0.0)
             if groups > 1:
                 runs = choice.reshape(groups, -1)
-                strength = runs.topk(min(2, runs.shape[1]), dim=1).values.sum(1)
+                strength = runs.topk(min(group_best, runs.shape[1]), dim=1).values.sum(1)
                 best = sorted(range(groups), key=lambda g: (-float(strength[g]), g))[:keep]
                 closed = [g for g in range(groups) if g not in best]
                 runs = runs.clone()
@@ -744,7 +814,8 @@ def attention_sink_wide_supports(num_heads, num_kv_heads, key_dim, value_dim):
     return False
 
 
-NAMES = ["add_layernorm", "channel_scan", "act_rows", "stream_spread", "stream_read_norm", "stream_write", "qkv_conv_rope_norm_cache",
+NAMES = ["add_layernorm", "embed_rmsnorm", "norm_add_norm", "delta_prepare", "delta_scan", "delta_step",
+         "delta_step_supports", "channel_scan", "act_rows", "stream_spread", "stream_read_norm", "stream_write", "qkv_conv_rope_norm_cache",
          "scaled_add_norm", "add_bias", "qk_rownorm_rope_cache", "latent_row_cache", "rope_slice",
          "head_linear", "mlstm", "mlstm_chunked", "mlstm_chunk_tokens", "mlstm_chunked_supports",
          "gated_group_norm", "qkv_bias_rope_cache", "causal_conv_act", "selective_scan",

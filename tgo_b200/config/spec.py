@@ -82,6 +82,7 @@ class MixerSpec:
     decay: tuple = ()                    # linear-attention kinds: one decay per head
     output_gate: bool = False            # the mixer's output multiplied by a gate projection
     gate_activation: str = "silu"        # what the gate projection goes through: silu | sigmoid
+    gate_scope: str = "channel"          # a number of the gate per "channel" of the output or per "head"
     input_activation: Optional[str] = None   # linear-attention kinds: q, k, v through this (silu)
     # linear-attention kinds: how the heads' outputs are normed: "head_unit" (each head by its
     # own root mean square, no gain) or "joint_gain" (all heads as one row, times a gain)
@@ -89,6 +90,8 @@ class MixerSpec:
     bias: bool = False                   # attention kinds: q, k and v projections carry biases
     sink: bool = False                   # attention kinds: a learned term per head in the
                                          # softmax's denominator that stands for no token
+    sink_score: Optional[float] = None   # attention kinds: the sink is this constant, not learned
+    values_from_keys: bool = False       # attention kinds: the values are the keys before the rotation
     # state-space kinds: num_heads heads of value_dim channels, num_kv_heads groups of B and C,
     # head_dim the state size; taps of the causal convolution; parts of the output norm
     conv_taps: int = 0
@@ -159,6 +162,8 @@ class FeedForwardSpec:
     router_scale: float = 1.0            # the weights are multiplied by this
     router_groups: Optional[tuple] = None    # (count, keep): the router outputs in `count` equal
                                          # runs, of which only the best `keep` can be chosen from
+    # a run of router_groups counts as the sum of this many of its largest choice scores (1 or 2)
+    router_group_best: int = 2
     router_correction: bool = False      # a per-expert term added to the scores for the choice only
     identity_experts: int = 0            # router outputs past `experts` whose expert is the input itself
     shared_gate: bool = False            # the shared feed-forward times a logistic gate per token
@@ -194,6 +199,9 @@ class LayerCall:
     """
     layer: int
     cache_from: Optional[int] = None
+    # the embedding output (what the stream was before the first call) joins the stream once more
+    # ahead of this call
+    adds_embedding: bool = False
 
 
 @dataclass
@@ -213,6 +221,8 @@ class ModelSpec:
     logit_softcap: Optional[float] = None   # c: logits <- c tanh(logits / c)
     logit_scale: float = 1.0         # the logits are multiplied by this
     embedding_scale: float = 1.0     # the embedding rows are multiplied by this
+    embedding_norm: Optional[NormSpec] = None    # a norm of the embedding rows, after the factor
+    embedding_norm_name: str = ""
     source: dict = field(default_factory=dict)   # the config.json it came from
 
     @property
@@ -226,6 +236,8 @@ class ModelSpec:
             if not (0 <= call.layer < len(self.layers)):
                 raise ValueError(f"model spec: run_order[{i}] names layer {call.layer}, "
                                  f"there are {len(self.layers)}")
+            if call.adds_embedding and i == 0:
+                raise ValueError("model spec: run_order[0] adds the embedding output to itself")
             if call.cache_from is not None:
                 if not (0 <= call.cache_from < i):
                     raise ValueError(f"model spec: run_order[{i}] reads the cache of call "

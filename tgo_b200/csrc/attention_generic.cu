@@ -21,6 +21,8 @@
 // order of the sums still depends on (p, window, keep_first) alone.
 // `dist_bias` (float32 [n_dist][H]): dist_bias[min(p - j, n_dist - 1)][h] is added to the
 // scaled score of key j, unscaled (a learned bias by distance).
+// `gate` ([T, >= H] in the storage type, rows gate_stride apart): the output of head h at token t
+// is multiplied by the logistic function of gate[t][h].
 #include "common.cuh"
 
 #define AG_MAX_DH 256            // rows up to this wide take the instance with 8 sums a lane
@@ -35,7 +37,7 @@ __global__ void attention_generic_kernel(
     int page_size, const int* __restrict__ block_tables, int max_blocks,
     const int* __restrict__ seq_ids, const int* __restrict__ positions, float scale, int window,
     const float* __restrict__ sinks, float softcap, int v_row, int keep_first,
-    const float* __restrict__ dist_bias, int n_dist) {
+    const float* __restrict__ dist_bias, int n_dist, const T* __restrict__ gate, long long gate_stride) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
@@ -100,7 +102,8 @@ __global__ void attention_generic_kernel(
         for (int i = 0; i < NACC; ++i) acc[i] *= corr;
     }
     T* o = out + (size_t)t * out_stride + (size_t)h * dv;
-    const float inv = l > 0.f ? 1.f / l : 0.f;     // position < 0: no keys, zeros out
+    float inv = l > 0.f ? 1.f / l : 0.f;           // position < 0: no keys, zeros out
+    if (gate) inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)t * gate_stride + h])));
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
         const int d = lane + 32 * i;
@@ -114,7 +117,8 @@ TGO_API int tgo_attention_generic(const void* q, long long q_stride, void* out,
                                   const int* block_tables, int max_blocks, const int* seq_ids,
                                   const int* positions, float scale, int window,
                                   const float* sinks, float softcap, int v_row, int keep_first,
-                                  const float* dist_bias, int n_dist, cudaStream_t stream) {
+                                  const float* dist_bias, int n_dist, const void* gate, long long gate_stride,
+                                  cudaStream_t stream) {
     if (T <= 0) return 0;
     if (v_row <= 0) v_row = dv;
     if (dh <= 0 || dh > AG_MAX_WIDEST || dv <= 0 || dv > AG_MAX_WIDEST || H <= 0 || Hkv <= 0 || H % Hkv ||
@@ -128,7 +132,7 @@ TGO_API int tgo_attention_generic(const void* q, long long q_stride, void* out,
     attention_generic_kernel<TT, NACC><<<grid, AG_WARPS * 32, smem, stream>>>(                         \
         (const TT*)q, q_stride, (TT*)out, out_stride, H, Hkv, dh, dv, (const TT*)k_cache,              \
         (const TT*)v_cache, page_size, block_tables, max_blocks, seq_ids, positions, scale, window,   \
-        sinks, softcap, v_row, keep_first, dist_bias, n_dist)
+        sinks, softcap, v_row, keep_first, dist_bias, n_dist, (const TT*)gate, gate_stride)
     if (dtype == TGO_BF16) {
         if (widest) AG_GO(bf16, AG_MAX_WIDEST / 32); else if (wide) AG_GO(bf16, AG_MAX_WIDE / 32); else AG_GO(bf16, AG_MAX_DH / 32);
     } else if (dtype == TGO_F32) {

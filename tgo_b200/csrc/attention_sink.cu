@@ -26,6 +26,8 @@
 // window's first tile are walked first, then the window's tiles (one list of tiles, which is
 // also what `n_splits` cuts). `dist_bias` (float32 [n_dist][H]): dist_bias[min(i - j, n_dist
 // - 1)][h] is added to the scaled score, unscaled (a learned bias by distance).
+// `gate` (bfloat16 [T, >= H], rows gate_stride apart): the finished output of head h at token t is
+// multiplied by the logistic function of gate[t][h].
 #include "common.cuh"
 
 #define AS_BN 64                 // keys per tile
@@ -53,6 +55,10 @@ __device__ __forceinline__ float as_scored(float qk, float scale_log2, float cap
     return fmaf(-2.f * cap_log2, r, cap_log2);
 }
 
+__device__ __forceinline__ float as_gate(const bf16* __restrict__ gate, long long gate_stride, int tok, int head) {
+    return gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)tok * gate_stride + head]))) : 1.f;
+}
+
 template <int DK, int DV>
 __global__ void __launch_bounds__(AS_WARPS * 32)
 attention_sink_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __restrict__ out,
@@ -64,7 +70,8 @@ attention_sink_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __re
                       int Hkv, int dk, int dv, float scale_log2, int window,
                       const float* __restrict__ sinks, int n_splits, float* __restrict__ part_o,
                       float* __restrict__ part_ml, float cap_log2, float scale_over_cap, int v_row,
-                      int keep_first, const float* __restrict__ dist_bias, int n_dist) {
+                      int keep_first, const float* __restrict__ dist_bias, int n_dist,
+                      const bf16* __restrict__ gate, long long gate_stride) {
     constexpr int LDK = DK + AS_PAD, LDV = DV + AS_PAD;
     constexpr int KS = DK / 16;
     constexpr int CHK = DK / 8, CHV = DV / 8;  // 16-byte chunks per padded row
@@ -311,7 +318,7 @@ attention_sink_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __re
                 corr = exp2f(m - mn);          // m = -inf cannot happen here: a row sees itself
                 l = l * corr + exp2f(sk2 - mn);
             }
-            const float inv = l > 0.f ? corr / l : 0.f;
+            const float inv = (l > 0.f ? corr / l : 0.f) * as_gate(gate, gate_stride, tok0 + r / G, head);
             bf16* dst = out + (size_t)(tok0 + r / G) * out_stride + (size_t)head * dv + col;
 #pragma unroll
             for (int i = 0; i < DV / 8; ++i)
@@ -336,7 +343,8 @@ attention_sink_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                              int Hkv, int dk, int dv, float scale_log2, int window,
                              const float* __restrict__ sinks, int n_splits, float* __restrict__ part_o,
                              float* __restrict__ part_ml, float cap_log2, float scale_over_cap, int v_row,
-                             int keep_first, const float* __restrict__ dist_bias, int n_dist) {
+                             int keep_first, const float* __restrict__ dist_bias, int n_dist,
+                             const bf16* __restrict__ gate, long long gate_stride) {
     constexpr int LDK = DK + AS_PAD, LDV = DV + AS_PAD;
     constexpr int KS = DK / 16;
     constexpr int CHK = DK / 8, CHV = DV / 8;
@@ -557,7 +565,8 @@ attention_sink_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                 part_ml[at * 2 + 1] = l;
             }
         } else {
-            out[(size_t)tok * out_stride + (size_t)head * dv + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+            const float gv = as_gate(gate, gate_stride, tok, head);
+            out[(size_t)tok * out_stride + (size_t)head * dv + d] = __float2bfloat16_rn(l > 0.f ? acc / l * gv : 0.f);
         }
     }
 }
@@ -1032,7 +1041,8 @@ attention_sink_wide_decode_kernel(const bf16* __restrict__ q, long long q_stride
 __global__ void __launch_bounds__(128)
 attention_sink_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                            const int* __restrict__ positions, const float* __restrict__ sinks,
-                           bf16* __restrict__ out, long long out_stride, int H, int dv, int n_splits) {
+                           bf16* __restrict__ out, long long out_stride, int H, int dv, int n_splits,
+                           const bf16* __restrict__ gate, long long gate_stride) {
     __shared__ float s_w[AS_JOIN], s_l[AS_JOIN], s_m[33];
     pdl_wait();
     const int tok = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, n = blockDim.x;
@@ -1046,6 +1056,7 @@ attention_sink_join_kernel(const float* __restrict__ part_o, const float* __rest
     __syncthreads();
     for (int w = 0; w < n / 32; ++w) m = fmaxf(m, s_m[w]);
     float l = sk2 != -INFINITY ? exp2f(sk2 - m) : 0.f;
+    const float gv = as_gate(gate, gate_stride, tok, head);
     bf16* dst = out + (size_t)tok * out_stride + (size_t)head * dv;
     const float* po = part_o + at * dv;
     for (int d0 = 0; d0 < dv; d0 += 4 * n) {   // up to four columns a thread at a time
@@ -1073,7 +1084,7 @@ attention_sink_join_kernel(const float* __restrict__ part_o, const float* __rest
                 }
             }
         }
-        const float inv = sum > 0.f ? 1.f / sum : 0.f;
+        const float inv = (sum > 0.f ? 1.f / sum : 0.f) * gv;
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
             const int d = d0 + tid + k * n;
@@ -1096,7 +1107,7 @@ static int launch_sink(const bf16* q, long long q_stride, bf16* out, long long o
                        const int* tile_ntok, int n_tiles, int H, int Hkv, int dk, int dv, float scale,
                        int window, const float* sinks, int n_splits, float* part_o, float* part_ml,
                        float softcap, int v_row, int keep_first, const float* dist_bias, int n_dist,
-                       cudaStream_t stream) {
+                       const bf16* gate, long long gate_stride, cudaStream_t stream) {
     const float cap_log2 = softcap > 0.f ? softcap * AS_LOG2E : 0.f;
     const float scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
     const size_t smem = ((size_t)AS_BM * (DK + AS_PAD) + 2 * AS_BN * (DK + AS_PAD) + 2 * AS_BN * (DV + AS_PAD)) *
@@ -1113,20 +1124,20 @@ static int launch_sink(const bf16* q, long long q_stride, bf16* out, long long o
         rc = tgo_launch_pdl(dec, dim3(n_tiles, Hkv, n_splits), dim3(128), dsm, stream, q, q_stride, out,
                             out_stride, k_cache, v_cache, page_size, block_tables, max_blocks, positions, seq_ids,
                             H, Hkv, dk, dv, scale * AS_LOG2E, window, sinks, n_splits, part_o, part_ml,
-                            cap_log2, scale_over_cap, v_row, keep_first, dist_bias, n_dist);
+                            cap_log2, scale_over_cap, v_row, keep_first, dist_bias, n_dist, gate, gate_stride);
     } else {
         auto kernel = attention_sink_kernel<DK, DV>;
         if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         kernel<<<dim3(n_tiles, Hkv, n_splits), AS_WARPS * 32, smem, stream>>>(
             q, q_stride, out, out_stride, k_cache, v_cache, page_size, block_tables, max_blocks, positions,
             seq_ids, tile_tok0, tile_ntok, H, Hkv, dk, dv, scale * AS_LOG2E, window, sinks, n_splits, part_o,
-            part_ml, cap_log2, scale_over_cap, v_row, keep_first, dist_bias, n_dist);
+            part_ml, cap_log2, scale_over_cap, v_row, keep_first, dist_bias, n_dist, gate, gate_stride);
         rc = launch_status();
     }
     if (rc || n_splits <= 1) return rc;
     return tgo_launch_pdl(attention_sink_join_kernel, dim3(n_tiles, H), dim3(dv > 64 ? 128 : 64), 0, stream,
                           (const float*)part_o, (const float*)part_ml, positions, sinks, out, out_stride, H, dv,
-                          n_splits);
+                          n_splits, gate, gate_stride);
 }
 
 // q [T, >= H dk] and out [T, >= H dv] bfloat16 views with unit column stride, 16-byte aligned
@@ -1141,7 +1152,7 @@ TGO_API int tgo_attention_sink(const void* q, long long q_stride, void* out, lon
                                int n_tiles, int H, int Hkv, int dk, int dv, float scale, int window,
                                const float* sinks, int n_splits, float* part_o, float* part_ml,
                                float softcap, int v_row, int keep_first, const float* dist_bias,
-                               int n_dist, cudaStream_t stream) {
+                               int n_dist, const void* gate, long long gate_stride, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (v_row <= 0) v_row = dv;
     if (v_row < dv || (v_row % 8) || !(softcap >= 0.f) || keep_first < 0 || (dist_bias && n_dist <= 0))
@@ -1158,7 +1169,7 @@ TGO_API int tgo_attention_sink(const void* q, long long q_stride, void* out, lon
                                           block_tables, max_blocks, positions, seq_ids, tile_tok0,        \
                                           tile_ntok, n_tiles, H, Hkv, dk, dv, scale, window, sinks,   \
                                           n_splits, part_o, part_ml, softcap, v_row, keep_first, dist_bias, \
-                                          n_dist, stream)
+                                          n_dist, (const bf16*)gate, gate_stride, stream)
     if (dk <= 64) return dv <= 64 ? AS_GO(64, 64) : AS_GO(64, 128);
     return dv <= 64 ? AS_GO(128, 64) : AS_GO(128, 128);
 #undef AS_GO
@@ -1198,7 +1209,7 @@ static int launch_sink_wide(const bf16* q, long long q_stride, bf16* out, long l
         if (rc || n_splits <= 1) return rc;
         return tgo_launch_pdl(attention_sink_join_kernel, dim3(n_tiles, H), dim3(128), 0, stream,
                               (const float*)part_o, (const float*)part_ml, positions, sinks, out, out_stride, H,
-                              dv, n_splits);
+                              dv, n_splits, (const bf16*)nullptr, 0LL);
     }
     auto kernel = attention_sink_wide_kernel<DK, DV>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -1209,7 +1220,7 @@ static int launch_sink_wide(const bf16* q, long long q_stride, bf16* out, long l
     if (rc || n_splits <= 1) return rc;
     return tgo_launch_pdl(attention_sink_join_kernel, dim3(n_tiles, H), dim3(128), 0, stream,
                           (const float*)part_o, (const float*)part_ml, positions, sinks, out, out_stride, H, dv,
-                          n_splits);
+                          n_splits, (const bf16*)nullptr, 0LL);
 }
 
 // As tgo_attention_sink for key rows up to 576 wide whose first dv (up to 512) channels are the

@@ -35,6 +35,51 @@ TGO_API int tgo_embed(const void* table, int dtype, const int* ids, float* out, 
     return launch_status();
 }
 
+// The gather with an RMS norm behind it: out[t, :] = gain * rmsnorm(table[ids[t], :] * scale),
+// float32, and the same rows in `copy` (may be null). An id outside [0, V) writes zeros. A block a
+// token; the scaled row waits in `out` between the sum of squares and the scaling (each thread
+// reads back only what it wrote).
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_rmsnorm_kernel(const T* __restrict__ table, const int* __restrict__ ids, const float* __restrict__ gain,
+                     float eps, float* out, float* copy, int d, int V, float scale) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < V;
+    const T* row = table + (size_t)(ok ? id : 0) * d;
+    float* o = out + (size_t)t * d;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        const float v = ok ? to_f32(row[i]) * scale : 0.f;
+        o[i] = v;
+        ss += v * v;
+    }
+    ss = block_sum(ss, scratch);
+    const float r = rsqrtf(ss / (float)d + eps);
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        const float v = (o[i] * r) * gain[i];
+        o[i] = v;
+        if (copy) copy[(size_t)t * d + i] = v;
+    }
+}
+
+TGO_API int tgo_embed_rmsnorm(const void* table, int dtype, const int* ids, const float* gain, float eps,
+                              float* out, float* copy, int T, int d, int V, float scale,
+                              cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (d <= 0 || V <= 0) return TGO_E_BAD_ARG;
+    const int threads = d >= 1024 ? 256 : 128;
+    if (dtype == TGO_BF16)
+        return tgo_launch_pdl(embed_rmsnorm_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16*)table,
+                              ids, gain, eps, out, copy, d, V, scale);
+    if (dtype == TGO_F32)
+        return tgo_launch_pdl(embed_rmsnorm_kernel<float>, dim3(T), dim3(threads), 0, stream,
+                              (const float*)table, ids, gain, eps, out, copy, d, V, scale);
+    return TGO_E_BAD_ARG;
+}
+
 // ------------------------------------------------------- residual add + RMSNorm
 // For output row i: r = rows ? rows[i] : i;  x = h[r] (+ delta[r]);  if rows is null the
 // sum is written back to h (the residual stream moves on);  out[i] = x * rsqrt(mean x^2

@@ -120,6 +120,125 @@ TGO_API int tgo_group_norm_scale_add(float* h, const void* y, int y_dtype, const
     return TGO_E_BAD_ARG;
 }
 
+// ------------------------------- a sublayer's result normed into the stream, and the next norm
+//   h <- h + extra + gain_y * rmsnorm(y);   out = gain * rmsnorm(h)
+// One pass over the row for a block that norms each sublayer's output and its next input. h, y and
+// extra (may be null) are float32, out in TO. A block
+// a row, the row in registers (CH quads a thread) or, with CH = 0, through h itself.
+template <typename TO> struct NnStore;
+template <> struct NnStore<float> {
+    static __device__ __forceinline__ void put(float* p, float4 v) { *(float4*)p = v; }
+};
+template <> struct NnStore<bf16> {
+    static __device__ __forceinline__ void put(bf16* p, float4 v) {
+        uint2 q;
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        q.x = *(uint32_t*)&lo;
+        q.y = *(uint32_t*)&hi;
+        *(uint2*)p = q;
+    }
+};
+
+template <typename TO, int CH>
+__global__ void __launch_bounds__(512)
+norm_add_norm_vec_kernel(float* __restrict__ h, const float* __restrict__ y, const float* __restrict__ gain_y,
+                         const float* __restrict__ extra, const float* __restrict__ gain, float eps_y,
+                         float eps, TO* __restrict__ out, int d) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * d;
+    float4 x[CH], s[CH];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int j = 4 * (threadIdx.x + c * blockDim.x);
+        x[c] = s[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < d) {
+            x[c] = *(const float4*)(y + base + j);
+            s[c] = *(const float4*)(h + base + j);
+            if (extra) {
+                const float4 e = *(const float4*)(extra + base + j);
+                s[c].x += e.x; s[c].y += e.y; s[c].z += e.z; s[c].w += e.w;
+            }
+            ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float ry = rsqrtf(ss / (float)d + eps_y);
+    ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int j = 4 * (threadIdx.x + c * blockDim.x);
+        if (j < d) {
+            const float4 g = *(const float4*)(gain_y + j);
+            s[c].x += (x[c].x * ry) * g.x; s[c].y += (x[c].y * ry) * g.y;
+            s[c].z += (x[c].z * ry) * g.z; s[c].w += (x[c].w * ry) * g.w;
+            *(float4*)(h + base + j) = s[c];
+            ss += s[c].x * s[c].x + s[c].y * s[c].y + s[c].z * s[c].z + s[c].w * s[c].w;
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float r = rsqrtf(ss / (float)d + eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int j = 4 * (threadIdx.x + c * blockDim.x);
+        if (j < d) {
+            const float4 g = *(const float4*)(gain + j);
+            NnStore<TO>::put(out + base + j, make_float4((s[c].x * r) * g.x, (s[c].y * r) * g.y,
+                                                         (s[c].z * r) * g.z, (s[c].w * r) * g.w));
+        }
+    }
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(256)
+norm_add_norm_kernel(float* __restrict__ h, const float* __restrict__ y, const float* __restrict__ gain_y,
+                     const float* __restrict__ extra, const float* __restrict__ gain, float eps_y, float eps,
+                     TO* __restrict__ out, int d) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * d;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) ss += y[base + i] * y[base + i];
+    ss = block_sum(ss, scratch);
+    const float ry = rsqrtf(ss / (float)d + eps_y);
+    ss = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        float s = h[base + i];
+        if (extra) s += extra[base + i];
+        s += (y[base + i] * ry) * gain_y[i];
+        h[base + i] = s;
+        ss += s * s;
+    }
+    ss = block_sum(ss, scratch);
+    const float r = rsqrtf(ss / (float)d + eps);
+    for (int i = threadIdx.x; i < d; i += blockDim.x) out[base + i] = from_f32<TO>((h[base + i] * r) * gain[i]);
+}
+
+TGO_API int tgo_norm_add_norm(float* h, const float* y, const float* gain_y, float eps_y, const float* extra,
+                              const float* gain, float eps, void* out, int out_dtype, int T, int d,
+                              cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (d <= 0 || (out_dtype != TGO_BF16 && out_dtype != TGO_F32)) return TGO_E_BAD_ARG;
+    const bool bf = out_dtype == TGO_BF16;
+    const bool aligned = d % 4 == 0 && d <= 8192 && !((uintptr_t)h & 15) && !((uintptr_t)y & 15) &&
+                         !((uintptr_t)gain_y & 15) && !((uintptr_t)extra & 15) && !((uintptr_t)gain & 15) &&
+                         !((uintptr_t)out & 15);
+    if (!aligned)
+        return bf ? tgo_launch_pdl(norm_add_norm_kernel<bf16>, dim3(T), dim3(256), 0, stream, h, y, gain_y, extra,
+                                   gain, eps_y, eps, (bf16*)out, d)
+                  : tgo_launch_pdl(norm_add_norm_kernel<float>, dim3(T), dim3(256), 0, stream, h, y, gain_y, extra,
+                                   gain, eps_y, eps, (float*)out, d);
+    const int quads = d / 4, vt = quads <= 256 ? 128 : quads <= 1024 ? 256 : 512, ch = (quads + vt - 1) / vt;
+#define NN_GO(TO, CH)                                                                                     \
+    tgo_launch_pdl(norm_add_norm_vec_kernel<TO, CH>, dim3(T), dim3(vt), 0, stream, h, y, gain_y, extra, gain, eps_y, \
+                   eps, (TO*)out, d)
+    if (ch <= 1) return bf ? NN_GO(bf16, 1) : NN_GO(float, 1);
+    if (ch <= 2) return bf ? NN_GO(bf16, 2) : NN_GO(float, 2);
+    return bf ? NN_GO(bf16, 4) : NN_GO(float, 4);
+#undef NN_GO
+}
+
 // --------------------------------------------- out = gain * group_rmsnorm(h[rows]) (no add)
 template <typename TO>
 __global__ void group_norm_rows_kernel(const float* __restrict__ h, const int* __restrict__ rows,

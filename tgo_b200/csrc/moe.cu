@@ -25,8 +25,8 @@
 // row itself; they get no place and no tile, the combine adds weight * x for them.
 // `score_mode` 2 takes the logistic function of each logit as its score; with `groups` > 1 the
 // experts are that many equal runs of neighbours, a run's strength is the sum of its two largest
-// choice scores, and only experts of the `keep` strongest runs can be chosen; without `renorm`
-// the weights are the chosen scores themselves; `route_scale` multiplies the weights. One more
+// choice scores (`run_best` 2) or its largest alone (`run_best` 1), and only experts of the `keep`
+// strongest runs can be chosen; without `renorm` the weights are the chosen scores themselves; `route_scale` multiplies the weights. One more
 // router row after all experts (`gate_out`) gives a logistic gate per token that multiplies
 // `extra` in the combine. Experts without a gate matrix (wg null) are W_down act(W_up x);
 // activation 3 is the square of relu.
@@ -139,7 +139,7 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg,
                                          float* __restrict__ wts, int* counts, int score_mode,
                                          const float* __restrict__ correction, int E_real,
                                          float* __restrict__ gate_out, int groups, int keep, int renorm,
-                                         float route_scale) {
+                                         float route_scale, int run_best) {
     const int lane = threadIdx.x & 31;
     for (int e = lane; e < E + (gate_out ? 1 : 0); e += 32) lg[e] = z[e];
     __syncwarp();
@@ -192,7 +192,7 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ z, float* lg,
                     const float v = lg[e];
                     if (v > a) { c = a; a = v; } else if (v > c) { c = v; }
                 }
-                gs[g] = size > 1 ? a + c : a;
+                gs[g] = size > 1 && run_best > 1 ? a + c : a;
             }
             __syncwarp();
             // the weakest groups - keep runs go: mark the strongest with +inf, then close the others
@@ -247,14 +247,14 @@ __global__ void __launch_bounds__(32 * MOE_PW)
 moe_pick_kernel(const float* __restrict__ logits, int rows, int Tn, int E, int top, int* __restrict__ ids,
                 float* __restrict__ wts, int* __restrict__ counts, int score_mode,
                 const float* __restrict__ correction, int E_real, float* __restrict__ gate_out, int groups,
-                int keep, int renorm, float route_scale) {
+                int keep, int renorm, float route_scale, int run_best) {
     extern __shared__ float smem[];                      // [MOE_PW][2 E + 1 + groups]
     pdl_wait();
     const int warp = threadIdx.x >> 5, t = blockIdx.x * MOE_PW + warp;
     if (t >= Tn) return;
     float* lg = smem + (size_t)warp * (2 * E + 1 + groups);
     moe_pick(logits + (size_t)t * rows, lg, lg + E + 1, lg + 2 * E + 1, t, E, top, ids, wts, counts, score_mode,
-             correction, E_real, gate_out, groups, keep, renorm, route_scale);
+             correction, E_real, gate_out, groups, keep, renorm, route_scale, run_best);
 }
 
 // -------------------------------------------------------------------------------- plan
@@ -310,7 +310,7 @@ __global__ void __launch_bounds__(32 * MOE_FEW_WARPS)
 moe_route_few_kernel(const float* __restrict__ logits, int rows, int Tn, int E, int top, int* __restrict__ ids,
                      float* __restrict__ wts, int score_mode, const float* __restrict__ correction, int E_real,
                      float* __restrict__ gate_out, int groups, int keep, int renorm, float route_scale,
-                     int* __restrict__ offsets, int* __restrict__ perm, int* __restrict__ place,
+                     int run_best, int* __restrict__ offsets, int* __restrict__ perm, int* __restrict__ place,
                      int* __restrict__ tile_info, int* __restrict__ tiles, int max_tiles) {
     extern __shared__ float smem[];                      // [warps][2 E + 1 + groups], counts, fill
     const int per = 2 * E + 1 + groups;
@@ -323,7 +323,7 @@ moe_route_few_kernel(const float* __restrict__ logits, int rows, int Tn, int E, 
     float* lg = smem + (size_t)warp * per;
     for (int t = warp; t < Tn; t += MOE_FEW_WARPS) {
         moe_pick(logits + (size_t)t * rows, lg, lg + E + 1, lg + 2 * E + 1, t, E, top, ids, wts, counts, score_mode,
-                 correction, E_real, gate_out, groups, keep, renorm, route_scale);
+                 correction, E_real, gate_out, groups, keep, renorm, route_scale, run_best);
         __syncwarp();
     }
     __syncthreads();                                     // ids are in memory for the whole block
@@ -655,12 +655,12 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
                           int* counts, int* fill, int* offsets, int* perm, int* place,
                           int* tile_info, int* tiles, int max_tiles, int score_mode,
                           const float* correction, int E_real, float* gate_out, int groups, int keep,
-                          int renorm, float route_scale, int* launches, cudaStream_t stream) {
+                          int renorm, float route_scale, int run_best, int* launches, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0 || E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || max_tiles <= 0 ||
         E_real < 0 || E_real > E || score_mode < 0 || score_mode > 2 || groups < 1 || E % groups ||
         keep < 1 || keep > groups || (long long)keep * (E / groups) < top || (groups > 1 && score_mode == 0) ||
-        (dtype != TGO_BF16 && dtype != TGO_F32))
+        run_best < 1 || run_best > 2 || (dtype != TGO_BF16 && dtype != TGO_F32))
         return TGO_E_BAD_ARG;
     const int rows = E + (gate_out ? 1 : 0);
     const dim3 lgrid((T + ML_TOK - 1) / ML_TOK, (rows + ML_EXP - 1) / ML_EXP);
@@ -680,8 +680,8 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
         *launches = 2;
         return tgo_launch_pdl(moe_route_few_kernel, dim3(1), dim3(32 * MOE_FEW_WARPS), few, stream,
                               (const float*)logits, rows, T, E, top, ids, wts, score_mode, correction, E_real,
-                              gate_out, groups, keep, renorm, route_scale, offsets, perm, place, tile_info, tiles,
-                              max_tiles);
+                              gate_out, groups, keep, renorm, route_scale, run_best, offsets, perm, place, tile_info,
+                              tiles, max_tiles);
     }
     *launches = 4;
     const size_t smem = MOE_PW * per;
@@ -689,7 +689,7 @@ TGO_API int tgo_moe_route(const void* x, long long x_stride, int dtype, const fl
         cudaFuncSetAttribute(moe_pick_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     rc = tgo_launch_pdl(moe_pick_kernel, dim3((T + MOE_PW - 1) / MOE_PW), dim3(32 * MOE_PW), smem, stream,
                         (const float*)logits, rows, T, E, top, ids, wts, counts, score_mode, correction, E_real,
-                        gate_out, groups, keep, renorm, route_scale);
+                        gate_out, groups, keep, renorm, route_scale, run_best);
     if (rc) return rc;
     rc = tgo_launch_pdl(moe_plan_kernel, dim3(1), dim3(32), 0, stream, (const int*)counts, E_real, offsets, fill,
                         tile_info, tiles, max_tiles);

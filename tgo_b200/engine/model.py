@@ -15,7 +15,7 @@ from ..cache.pages import GroupLayout
 from ..cache.storage import CacheStorage
 from ..config.spec import ModelSpec
 from ..kernels import ops
-from ..parts.base import LayerCache, StepContext, offered
+from ..parts.base import LayerCache, NormedDelta, StepContext, offered
 from ..registry import BLOCKS, NORMS
 from ..weights.binder import WeightSpec
 
@@ -32,6 +32,10 @@ class Model:
                        for ls in spec.layers]
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm, spec.hidden_size,
                                                           spec.final_norm_name)
+        self.embedding_norm = None
+        if spec.embedding_norm is not None:
+            self.embedding_norm = NORMS.get(spec.embedding_norm.kind)(spec.embedding_norm, spec.hidden_size,
+                                                                      spec.embedding_norm_name)
         if spec.logit_scale != 1.0 and not hasattr(self.final_norm, "fold_scale"):
             raise ValueError(f"model: the final norm {spec.final_norm.kind!r} takes no factor for the "
                              "logits (no fold_scale)")
@@ -43,6 +47,8 @@ class Model:
     def weight_specs(self) -> List[WeightSpec]:
         s = self.spec
         out = [WeightSpec(s.embedding_name, (s.vocab_size, s.hidden_size), "table")]
+        if self.embedding_norm is not None:
+            out += self.embedding_norm.weight_specs()
         for b in self.blocks:
             out += b.weight_specs()
         out += self.final_norm.weight_specs()
@@ -60,6 +66,8 @@ class Model:
         s = self.spec
         self.embedding = weights[s.embedding_name].contiguous()
         self.head = self.embedding if s.head_name is None else weights[s.head_name].contiguous()
+        if self.embedding_norm is not None:
+            self.embedding_norm.bind(weights)
         for b in self.blocks:
             b.bind(weights)
         self.final_norm.bind(weights)
@@ -138,7 +146,9 @@ class Model:
             names.append("layer_ops")
         for b in self.blocks:
             names += offered(b, "libraries")(self.dtype, page_size)
-        names += offered(self.final_norm, "libraries")(self.dtype, page_size)
+        for norm in (self.embedding_norm, self.final_norm):
+            if norm is not None:
+                names += offered(norm, "libraries")(self.dtype, page_size)
         return list(dict.fromkeys(names))
 
     def prepare_capture(self, ctx: StepContext, storage: CacheStorage, group_tables,
@@ -179,19 +189,47 @@ class Model:
             lc.state = storage.state[owner]
         return lc
 
+    def _embed(self, ctx: StepContext):
+        """(the stream, float32 [T, d]; a copy of it where a later call adds it again, else None)."""
+        s = self.spec
+        h = torch.empty((ctx.num_tokens, s.hidden_size), dtype=torch.float32, device=self.device)
+        again = any(call.adds_embedding for call in s.run_order)
+        scale = float(s.embedding_scale)
+        if hasattr(self.embedding_norm, "of_embedding"):
+            first = torch.empty_like(h) if again else None
+            self.embedding_norm.of_embedding(self.embedding, ctx.token_ids, scale, h, first)
+            return h, first
+        if scale != 1.0:
+            ops.embed(self.embedding, ctx.token_ids, h, scale)
+        else:
+            ops.embed(self.embedding, ctx.token_ids, h)
+        if self.embedding_norm is not None:
+            h = self.embedding_norm.forward(h, None, torch.float32)
+        return h, h.clone() if again else None
+
     def forward(self, ctx: StepContext, storage: CacheStorage, group_tables,
                 group_slots) -> torch.Tensor:
         """Run the step's tokens through every call; logits (float32) at ctx.logit_rows."""
         s = self.spec
-        h = torch.empty((ctx.num_tokens, s.hidden_size), dtype=torch.float32, device=self.device)
-        if s.embedding_scale != 1.0:
-            ops.embed(self.embedding, ctx.token_ids, h, float(s.embedding_scale))
-        else:
-            ops.embed(self.embedding, ctx.token_ids, h)
+        h, first = self._embed(ctx)
         pending = None
         for ci, call in enumerate(s.run_order):
             cache = self.layer_cache(ci, ctx, storage, group_tables, group_slots)
-            h, pending = self.blocks[call.layer].forward(h, pending, ctx, cache)
+            block = self.blocks[call.layer]
+            if isinstance(pending, NormedDelta) and not getattr(block, "takes_normed", False):
+                pending.settle(h)
+                pending = None
+            if call.adds_embedding:
+                if isinstance(pending, NormedDelta):
+                    pending.extra = first
+                else:
+                    if pending is not None:
+                        ops.residual_add(h, pending)
+                    pending = first
+            h, pending = block.forward(h, pending, ctx, cache)
+        if isinstance(pending, NormedDelta):
+            pending.settle(h)
+            pending = None
         n_want = ctx.logit_rows.numel()
         if n_want == 0:
             return torch.empty((0, s.vocab_size), dtype=torch.float32, device=self.device)

@@ -36,6 +36,7 @@ LIBRARIES = {
     "latent": (["latent.cu"], []),
     "layer_ops": (["layer_ops.cu"], []),
     "state_space": (["state_space.cu"], []),
+    "delta": (["delta.cu"], []),
     "attention_sink": (["attention_sink.cu"], []),
     "moe": (["moe.cu"], []),
     "attention_flash": (["attention_flash.cu"], []),

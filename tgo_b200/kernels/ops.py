@@ -68,6 +68,20 @@ def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: floa
                          c_int(T), c_int(d), c_int(table.shape[0]), c_float(scale), _stream()), "embed")
 
 
+def embed_rmsnorm(table: torch.Tensor, ids: torch.Tensor, gain: torch.Tensor, eps: float,
+                  out: torch.Tensor, copy: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+    """out[t] = gain * rmsnorm(table[ids[t]] * scale), float32, and the same rows in `copy`."""
+    _need_cuda(table, ids, gain, out, copy)
+    T, d = out.shape
+    assert ids.dtype == torch.int32 and ids.numel() == T and table.is_contiguous() and table.shape[1] == d
+    assert out.dtype == gain.dtype == torch.float32 and out.is_contiguous() and gain.numel() == d
+    assert copy is None or (copy.dtype == torch.float32 and copy.shape == out.shape and copy.is_contiguous())
+    lib = load_library("elementwise")
+    _check(lib.tgo_embed_rmsnorm(_ptr(table), c_int(dtype_code(table.dtype)), _ptr(ids), _ptr(gain),
+                                 c_float(eps), _ptr(out), _ptr(copy), c_int(T), c_int(d),
+                                 c_int(table.shape[0]), c_float(scale), _stream()), "embed_rmsnorm")
+
+
 def add_rmsnorm(h: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
                 out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
     """h += delta (if given, and rows is None), out = rmsnorm(h) * gain.
@@ -188,7 +202,8 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv
                       scale: float, window: int, value_dim: Optional[int] = None,
                       sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
                       value_row: int = 0, keep_first: int = 0,
-                      dist_bias: Optional[torch.Tensor] = None) -> None:
+                      dist_bias: Optional[torch.Tensor] = None,
+                      gate: Optional[torch.Tensor] = None) -> None:
     """Paged causal attention, one warp per (token, head). q is a 2-D view [T, >= H*dh]
     with unit column stride; out likewise. window 0 = every earlier key. `value_dim`: width
     of a value row where it differs from the keys'; `sinks`: float32 [H], a term exp(sink_h)
@@ -197,8 +212,12 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv
     that is not `value_dim` (values that are the first channels of their key rows: v_cache is
     k_cache and value_row the key rows' width); `keep_first`: with a window, the first keys of
     a request that every later query still reads; `dist_bias`: float32 [n, H], row
-    min(distance, n - 1) is added to the scaled scores of the keys at that distance."""
-    _need_cuda(q, out, k_cache, v_cache, block_tables, seq_ids, positions, sinks, dist_bias)
+    min(distance, n - 1) is added to the scaled scores of the keys at that distance; `gate`: a
+    2-D view [T, H] in q's type, head h's output is multiplied by the logistic function of
+    gate[t, h]."""
+    _need_cuda(q, out, k_cache, v_cache, block_tables, seq_ids, positions, sinks, dist_bias, gate)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape == (q.shape[0], num_heads) and
+                            (gate.stride(1) == 1 or num_heads == 1))
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.dim() == 2 and
                                  dist_bias.shape[1] == num_heads and dist_bias.is_contiguous())
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == num_heads and
@@ -216,8 +235,9 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv
         _ptr(v_cache), c_int(page_size), _ptr(block_tables), c_int(block_tables.shape[1]),
         _ptr(seq_ids), _ptr(positions), c_float(scale), c_int(window), _ptr(sinks),
         c_float(softcap or 0.0), c_int(value_row), c_int(keep_first if window else 0),
-        _ptr(dist_bias), c_int(dist_bias.shape[0] if dist_bias is not None else 0), _stream()),
-        "attention_generic", f"(head_dim={head_dim}, heads={num_heads}/{num_kv_heads})")
+        _ptr(dist_bias), c_int(dist_bias.shape[0] if dist_bias is not None else 0), _ptr(gate),
+        c_ll(gate.stride(0) if gate is not None else 0), _stream()), "attention_generic",
+        f"(head_dim={head_dim}, heads={num_heads}/{num_kv_heads})")
 
 
 def cast_rows(h: torch.Tensor, out: torch.Tensor) -> None:
@@ -247,6 +267,23 @@ def group_norm_scale_add(h: torch.Tensor, y: torch.Tensor, gain: torch.Tensor,
         _ptr(h), _ptr(y), c_int(dtype_code(y.dtype)), _ptr(gain), _ptr(scale), c_float(eps),
         c_int(groups), _ptr(act), c_int(dtype_code(act.dtype) if act is not None else 0),
         c_int(T), c_int(d), _stream()), "group_norm_scale_add", f"(d={d}, groups={groups})")
+
+
+def norm_add_norm(h: torch.Tensor, y: torch.Tensor, gain_y: torch.Tensor, eps_y: float,
+                  gain: torch.Tensor, eps: float, out: torch.Tensor,
+                  extra: Optional[torch.Tensor] = None) -> None:
+    """h <- h + extra + gain_y * rmsnorm(y), then out = gain * rmsnorm(h): h, y, extra float32
+    [T, d], out [T, d] in the activation type."""
+    _need_cuda(h, y, gain_y, gain, out, extra)
+    T, d = h.shape
+    assert h.dtype == y.dtype == gain_y.dtype == gain.dtype == torch.float32
+    assert y.shape == out.shape == h.shape and gain_y.numel() == gain.numel() == d
+    assert all(t.is_contiguous() for t in (h, y, gain_y, gain, out))
+    assert extra is None or (extra.dtype == torch.float32 and extra.shape == h.shape and extra.is_contiguous())
+    lib = load_library("layer_ops")
+    _check(lib.tgo_norm_add_norm(_ptr(h), _ptr(y), _ptr(gain_y), c_float(eps_y), _ptr(extra), _ptr(gain),
+                                 c_float(eps), _ptr(out), c_int(dtype_code(out.dtype)), c_int(T), c_int(d),
+                                 _stream()), "norm_add_norm", f"(d={d})")
 
 
 def group_norm_rows(h: torch.Tensor, rows: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
@@ -407,15 +444,18 @@ def attention_sink_tile(q: torch.Tensor, out: torch.Tensor, num_heads: int, num_
                         sinks: Optional[torch.Tensor], tile_tok0: Optional[torch.Tensor] = None,
                         tile_ntok: Optional[torch.Tensor] = None, n_splits: int = 1,
                         softcap: float = 0.0, value_row: int = 0, keep_first: int = 0,
-                        dist_bias: Optional[torch.Tensor] = None) -> None:
-    """`softcap`, `value_row`, `keep_first` and `dist_bias` as in `attention_generic`.
+                        dist_bias: Optional[torch.Tensor] = None,
+                        gate: Optional[torch.Tensor] = None) -> None:
+    """`softcap`, `value_row`, `keep_first`, `dist_bias` and `gate` as in `attention_generic`.
     Paged causal attention with keys `key_dim` and values `value_dim` wide, a window (0:
     none) and a sink per head (float32 [H] or None), bfloat16 on the tensor cores: a block per
     tile of consecutive tokens of one request (tile_tok0, tile_ntok: int32; None: every token
     is a tile of its own) and kv head. Without tile lists, `n_splits` > 1 cuts every token's
     keys over as many blocks and a second kernel joins their shares."""
     _need_cuda(q, out, k_cache, v_cache, block_tables, seq_ids, positions, sinks, tile_tok0, tile_ntok,
-               dist_bias)
+               dist_bias, gate)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape == (q.shape[0], num_heads) and
+                            (gate.stride(1) == 1 or num_heads == 1))
     assert q.dtype == out.dtype == k_cache.dtype == v_cache.dtype == torch.bfloat16
     assert q.stride(1) == 1 and out.stride(1) == 1
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and block_tables.is_contiguous()
@@ -442,7 +482,8 @@ def attention_sink_tile(q: torch.Tensor, out: torch.Tensor, num_heads: int, num_
         c_int(num_kv_heads), c_int(key_dim), c_int(value_dim), c_float(scale), c_int(window),
         _ptr(sinks), c_int(n_splits), _ptr(part_o), _ptr(part_ml), c_float(softcap or 0.0),
         c_int(value_row), c_int(keep_first), _ptr(dist_bias),
-        c_int(dist_bias.shape[0] if dist_bias is not None else 0), _stream()), "attention_sink",
+        c_int(dist_bias.shape[0] if dist_bias is not None else 0), _ptr(gate),
+        c_ll(gate.stride(0) if gate is not None else 0), _stream()), "attention_sink",
         f"(heads={num_heads}/{num_kv_heads}, dk={key_dim}, dv={value_dim})")
     if n_splits > 1:
         LAUNCHES[0] += 1
@@ -982,6 +1023,112 @@ def channel_scan(x: torch.Tensor, z: torch.Tensor, dt_raw: torch.Tensor, dt_bias
         "channel_scan", f"(channels={C}, state={N})")
 
 
+def delta_prepare(x: torch.Tensor, w: torch.Tensor, b_raw: torch.Tensor, a_raw: torch.Tensor,
+                  dt_bias: torch.Tensor, decay: torch.Tensor, num_seqs: int, heads: int, groups: int,
+                  key_dim: int, value_dim: int, seq_ids: torch.Tensor, q_start: torch.Tensor,
+                  state_slots: torch.Tensor, state: torch.Tensor, conv_offset: int) -> tuple:
+    """What the gated delta rule reads of a step's projections: x [T, C] holds q, k (groups *
+    key_dim each) and v (heads * value_dim), which pass a causal convolution (w float32 [taps, C],
+    the last row meets the current token; earlier inputs from the state row's [taps - 1, C] at
+    `conv_offset`) and SiLU; q and k become unit vectors per head (q times key_dim^-1/2). b_raw and
+    a_raw [T, heads]: the step size sigmoid(b) and the decay exp(-decay softplus(a + dt_bias)). All
+    float32: (qk [T, groups, 2, key_dim rounded up to 32], v [T, heads * value_dim], gates [T, heads,
+    4] = (g, g - 1, beta, 0), pairs [T, groups, 4] = k.q of a token and, for the second of a pair
+    counted from a request's first token of the step, k and q with the first one's k)."""
+    _need_cuda(x, w, b_raw, a_raw, dt_bias, decay, seq_ids, q_start, state_slots, state)
+    T, C = x.shape
+    taps = w.shape[0]
+    assert C == 2 * groups * key_dim + heads * value_dim and x.stride(1) == 1
+    assert w.dtype == torch.float32 and w.is_contiguous() and w.shape == (taps, C)
+    for t in (b_raw, a_raw):
+        assert t.shape == (T, heads) and t.dtype == x.dtype and (t.stride(1) == 1 or heads == 1)
+    assert b_raw.stride(0) == a_raw.stride(0)
+    for t in (dt_bias, decay):
+        assert t.dtype == torch.float32 and t.numel() == heads and t.is_contiguous()
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+    assert seq_ids.dtype == q_start.dtype == state_slots.dtype == torch.int32
+    assert q_start.numel() == num_seqs + 1 and state_slots.numel() == num_seqs and seq_ids.numel() == T
+    wide = (key_dim + 31) // 32 * 32
+    n_qk, n_v = T * groups * 2 * wide, (T * heads * value_dim + 3) // 4 * 4
+    buf = torch.empty(n_qk + n_v + 4 * T * (heads + groups), dtype=torch.float32, device=x.device)
+    qk = buf[:n_qk].view(T, groups, 2, wide)
+    v = buf[n_qk:n_qk + T * heads * value_dim].view(T, heads * value_dim)
+    at = n_qk + n_v
+    gates = buf[at:at + 4 * T * heads].view(T, heads, 4)
+    pairs = buf[at + 4 * T * heads:].view(T, groups, 4)
+    lib = load_library("delta")
+    _check(lib.tgo_delta_prepare(
+        _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w), _ptr(b_raw), _ptr(a_raw),
+        c_ll(a_raw.stride(0)), _ptr(dt_bias), _ptr(decay), _ptr(qk), _ptr(v), _ptr(gates), _ptr(pairs),
+        c_int(T), c_int(num_seqs), c_int(heads), c_int(groups), c_int(key_dim), c_int(value_dim), c_int(taps),
+        _ptr(seq_ids), _ptr(q_start), _ptr(state_slots), _ptr(state), c_ll(state.stride(0)),
+        c_ll(conv_offset), _stream()), "delta_prepare",
+        f"(heads={heads}/{groups}, dk={key_dim}, dv={value_dim}, taps={taps})")
+    return qk, v, gates, pairs
+
+
+def _delta_args(prepared, conv_in, heads, groups, key_dim, value_dim, num_seqs, q_start, state_slots, state):
+    qk, v, gates, pairs = prepared
+    T = qk.shape[0]
+    _need_cuda(qk, v, gates, pairs, conv_in, q_start, state_slots, state)
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in prepared)
+    assert qk.shape == (T, groups, 2, (key_dim + 31) // 32 * 32) and v.shape == (T, heads * value_dim)
+    assert gates.shape == (T, heads, 4) and pairs.shape == (T, groups, 4)
+    assert conv_in.shape == (T, 2 * groups * key_dim + heads * value_dim) and conv_in.stride(1) == 1
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+    assert q_start.dtype == state_slots.dtype == torch.int32
+    assert q_start.numel() == num_seqs + 1 and state_slots.numel() == num_seqs
+
+
+def delta_scan(prepared: tuple, y: torch.Tensor, num_seqs: int, heads: int, groups: int, key_dim: int,
+               value_dim: int, q_start: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor,
+               mem_offset: int, conv_in: torch.Tensor, taps: int, conv_offset: int) -> None:
+    """The gated delta rule S <- g S; u = beta (v - S^T k); S <- S + k u^T; y = S^T q per head over
+    each request's tokens, from and into its state row (float32 [slots, n]; S [heads, key_dim,
+    value_dim] at `mem_offset`). `prepared` is what `delta_prepare` returned, y float32 [T, heads *
+    value_dim]. The convolution's kept inputs [taps - 1, C] at `conv_offset` are moved on by the raw
+    inputs `conv_in` [T, C]."""
+    _delta_args(prepared, conv_in, heads, groups, key_dim, value_dim, num_seqs, q_start, state_slots, state)
+    qk, v, gates, pairs = prepared
+    assert y.dtype == torch.float32 and y.is_contiguous() and y.shape == v.shape and y.is_cuda
+    lib = load_library("delta")
+    _check(lib.tgo_delta_scan(
+        _ptr(qk), _ptr(v), _ptr(gates), _ptr(pairs), _ptr(y), c_int(num_seqs), c_int(heads), c_int(groups),
+        c_int(key_dim), c_int(value_dim), _ptr(q_start), _ptr(state_slots), _ptr(state),
+        c_ll(state.stride(0)), c_ll(mem_offset), _ptr(conv_in), c_ll(conv_in.stride(0)),
+        c_int(dtype_code(conv_in.dtype)), c_int(taps), c_ll(conv_offset), _stream()), "delta_scan",
+        f"(heads={heads}/{groups}, dk={key_dim}, dv={value_dim})")
+
+
+def delta_step_supports(heads: int, groups: int, key_dim: int, value_dim: int, state: torch.Tensor,
+                        mem_offset: int) -> bool:
+    """Whether the kernel for requests of one token each takes these sizes."""
+    return bool(load_library("delta").tgo_delta_step_supports(
+        c_int(heads), c_int(groups), c_int(key_dim), c_int(value_dim), c_ll(state.stride(0)), c_ll(mem_offset)))
+
+
+def delta_step(prepared: tuple, z: torch.Tensor, gain: torch.Tensor, eps: float, out: torch.Tensor,
+               num_seqs: int, heads: int, groups: int, key_dim: int, value_dim: int, q_start: torch.Tensor,
+               state_slots: torch.Tensor, state: torch.Tensor, mem_offset: int, conv_in: torch.Tensor,
+               taps: int, conv_offset: int) -> None:
+    """`delta_scan` for requests of one token each, with what follows it: out = gain * rmsnorm of
+    each head's row * silu(z), z [T, heads * value_dim] a 2-D view and out contiguous, both in the
+    activation type, gain float32 [value_dim]."""
+    _delta_args(prepared, conv_in, heads, groups, key_dim, value_dim, num_seqs, q_start, state_slots, state)
+    qk, v, gates, pairs = prepared
+    _need_cuda(z, gain, out)
+    assert z.shape == out.shape == v.shape and z.stride(1) == 1 and out.is_contiguous()
+    assert z.dtype == out.dtype == conv_in.dtype and num_seqs == v.shape[0]
+    assert gain.dtype == torch.float32 and gain.numel() == value_dim and gain.is_contiguous()
+    lib = load_library("delta")
+    _check(lib.tgo_delta_step(
+        _ptr(qk), _ptr(v), _ptr(gates), _ptr(pairs), _ptr(z), c_ll(z.stride(0)), _ptr(gain), c_float(eps),
+        _ptr(out), c_int(num_seqs), c_int(heads), c_int(groups), c_int(key_dim), c_int(value_dim),
+        _ptr(q_start), _ptr(state_slots), _ptr(state), c_ll(state.stride(0)), c_ll(mem_offset),
+        _ptr(conv_in), c_ll(conv_in.stride(0)), c_int(dtype_code(conv_in.dtype)), c_int(taps),
+        c_ll(conv_offset), _stream()), "delta_step", f"(heads={heads}/{groups}, dk={key_dim}, dv={value_dim})")
+
+
 # how a router's logits become scores
 ROUTER_SCORES = {"chosen": 0, "all": 1, "sigmoid": 2}
 
@@ -998,7 +1145,8 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
                      identity: int = 0, extra_gated: bool = False, groups: int = 1, keep: int = 1,
                      renormalize: bool = True, route_scale: float = 1.0,
                      beside: Optional[torch.Tensor] = None,
-                     residual: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                     residual: Optional[torch.Tensor] = None,
+                     group_best: int = 2) -> Optional[torch.Tensor]:
     """A routed feed-forward: each row of x [T, d] goes to the `top` experts with the largest
     router scores (w_router float32 [E, d], b_router float32 [E]; float32 sums); expert e is
     w_down[e] (act(w_gate[e] x) * (w_up[e] x)), or, with w_gate None, w_down[e] act(w_up[e] x).
@@ -1014,7 +1162,8 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
 
     `scores` "sigmoid": as "all" with each logit's logistic function as its score. With either,
     `groups` > 1 cuts the router outputs into equal runs of neighbours and only those of the
-    `keep` runs whose two largest choice scores sum highest can be chosen; without `renormalize`
+    `keep` runs whose two largest choice scores sum highest (`group_best` 1: whose largest choice
+    score is highest) can be chosen; without `renormalize`
     the weights are the chosen scores as they are. `route_scale` multiplies the weights.
 
     `beside` ([T, d], float32 or bfloat16) is added to the result; with `residual` (float32
@@ -1061,7 +1210,8 @@ def moe_feed_forward(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional
         c_int(T), c_int(d), c_int(outputs), c_int(top), _ptr(logits), _ptr(ids), _ptr(wts), _ptr(counts), _ptr(fill),
         _ptr(offsets), _ptr(perm), _ptr(place), _ptr(tile_info), _ptr(tiles), c_int(max_tiles),
         c_int(ROUTER_SCORES[scores]), _ptr(correction), c_int(E), _ptr(gate), c_int(groups), c_int(keep),
-        c_int(1 if renormalize else 0), c_float(route_scale), ctypes.byref(launches), _stream()), "moe_route", f"(E={E}+{identity}, top={top})")
+        c_int(1 if renormalize else 0), c_float(route_scale), c_int(group_best), ctypes.byref(launches),
+        _stream()), "moe_route", f"(E={E}+{identity}, top={top})")
     _check(lib.tgo_moe_experts(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w_gate), _ptr(w_up),
         _ptr(w_down), _ptr(hidden), _ptr(y), _ptr(wts), _ptr(extra), _ptr(out), c_int(T), c_int(d),

@@ -17,6 +17,10 @@
   - `qk_unit_norm`: every q and k head is divided by its root mean square after the rotation;
   - `keep_first`: beside the window a query reads the first keep_first keys of its request;
   - `query_temperature` (coef, every): q at position p times 1 + coef ln(floor((p+1)/every) + 1);
+  - `values_from_keys`: there is no value projection; a token's values are its keys as projected,
+    before the rotation (value_dim = head_dim);
+  - `sink_score` s: the sink is the constant s for every head instead of a learned number;
+  - `output_gate` with scope "head": head h's output is multiplied by sigmoid(W_g x)_h;
   - `distance_bias_max` D: a learned table [rows, heads] adds table[bucket(i - j), h] to the
     scaled score, bucket(n) = n below rows/2, then min(rows - 1, rows/2 + floor(ln(n / (rows/2))
     / ln(D / (rows/2)) * (rows - rows/2))).
@@ -26,8 +30,8 @@
     out_i       = Wo concat_h sum_j w_h(i, j) v_kv(h)(j)
 
 Scores, softmax and sums are float32. Tensor roles: q, k, v, o and, with `bias`, q_bias, k_bias,
-v_bias; with `sink`, sink; with the row norm, q_norm, k_norm; with the convolution, q_conv,
-k_conv, v_conv ([channels, taps]); with the distance bias, distance_bias.
+v_bias; with `sink`, sink; with the head gate, gate; with the row norm, q_norm, k_norm; with the
+convolution, q_conv, k_conv, v_conv ([channels, taps]); with the distance bias, distance_bias.
 """
 from __future__ import annotations
 
@@ -105,7 +109,21 @@ class SinkAttention(Part):
                              "not offered together with biases or the row norm")
         if self.temperature is not None and not self.row_norm:
             raise ValueError("attention: the query temperature is applied by the row norm's kernel")
-        roles = ["q", "k", "v", "o"] + (["q_bias", "k_bias", "v_bias"] if self.bias else []) + \
+        self.values_from_keys = bool(getattr(spec, "values_from_keys", False))
+        if self.values_from_keys and (self.dv != self.dk or self.bias or self.taps or self.unit_norm):
+            raise ValueError("attention: values that are the keys are as wide as they are, and are not "
+                             "offered with biases, the convolution or the unit norm")
+        self.sink_score = getattr(spec, "sink_score", None)
+        if self.sink and self.sink_score is not None:
+            raise ValueError("attention: the sink is learned or a constant, not both")
+        self.head_gate = bool(spec.output_gate)
+        if self.head_gate and (spec.gate_scope != "head" or spec.gate_activation != "sigmoid"):
+            raise ValueError("attention: this mixer's output gate is one logistic number per head "
+                             "(gate_scope 'head', gate_activation 'sigmoid')")
+        if self.head_gate and (self.taps or self.unit_norm):
+            raise ValueError("attention: the head gate is not offered with the convolution or the unit norm")
+        roles = ["q", "k", "o"] + ([] if self.values_from_keys else ["v"]) + \
+            (["q_bias", "k_bias", "v_bias"] if self.bias else []) + (["gate"] if self.head_gate else []) + \
             (["sink"] if self.sink else []) + (["q_norm", "k_norm"] if self.row_norm else []) + \
             (["q_conv", "k_conv", "v_conv"] if self.taps else []) + \
             (["distance_bias"] if self.bias_max is not None else [])
@@ -116,8 +134,12 @@ class SinkAttention(Part):
     def weight_specs(self):
         n, d = self.names, self.hidden
         qw, kw, vw = self.H * self.dk, self.Hkv * self.dk, self.Hkv * self.dv
-        out = [WeightSpec(n["q"], (qw, d)), WeightSpec(n["k"], (kw, d)), WeightSpec(n["v"], (vw, d)),
+        out = [WeightSpec(n["q"], (qw, d)), WeightSpec(n["k"], (kw, d)),
                WeightSpec(n["o"], (d, self.H * self.dv))]
+        if not self.values_from_keys:
+            out.insert(2, WeightSpec(n["v"], (vw, d)))
+        if self.head_gate:
+            out.append(WeightSpec(n["gate"], (self.H, d)))
         if self.bias:
             out += [WeightSpec(n["q_bias"], (qw,), "gain"), WeightSpec(n["k_bias"], (kw,), "gain"),
                     WeightSpec(n["v_bias"], (vw,), "gain")]
@@ -145,14 +167,20 @@ class SinkAttention(Part):
 
     def bind(self, weights):
         n = self.names
-        self.w_qkv = torch.cat([weights.pop(n["q"]), weights.pop(n["k"]), weights.pop(n["v"])],
-                               dim=0).contiguous()
+        rows = [weights.pop(n[r]) for r in ("q", "k") + (() if self.values_from_keys else ("v",)) +
+                (("gate",) if self.head_gate else ())]
+        if self.head_gate and self.H % 8:            # whole 16-byte rows for the products
+            rows.append(rows[0].new_zeros((8 - self.H % 8, self.hidden)))
+        self.w_qkv = torch.cat(rows, dim=0).contiguous()
         self.w_o = weights.pop(n["o"]).contiguous()
         if self.bias:
             self.b_q, self.b_k, self.b_v = (weights.pop(n[r]).to(torch.float32).contiguous()
                                             for r in ("q_bias", "k_bias", "v_bias"))
         if self.sink:
             self.sinks = weights.pop(n["sink"]).to(torch.float32).contiguous()
+        elif self.sink_score is not None:
+            self.sinks = torch.full((self.H,), float(self.sink_score), dtype=torch.float32,
+                                    device=self.w_o.device)
         if self.row_norm:
             self.q_gain = weights.pop(n["q_norm"]).to(torch.float32).contiguous()
             self.k_gain = weights.pop(n["k_norm"]).to(torch.float32).contiguous()
@@ -177,7 +205,8 @@ class SinkAttention(Part):
     def flops(self, extents, first_positions, writes_cache: bool = True) -> float:
         n = sum(extents)
         qw, kw, vw = self.H * self.dk, self.Hkv * self.dk, self.H * self.dv
-        total = 2.0 * n * self.hidden * (qw + kw + self.Hkv * self.dv) + 2.0 * n * vw * self.hidden
+        rows = qw + kw + (0 if self.values_from_keys else self.Hkv * self.dv) + (self.H if self.head_gate else 0)
+        total = 2.0 * n * self.hidden * rows + 2.0 * n * vw * self.hidden
         keys = 0
         for first, extent in zip(first_positions, extents):
             if self.window:
@@ -195,7 +224,14 @@ class SinkAttention(Part):
         qw, kw = H * dk, Hkv * dk
         x = ops.rows_of(x)
         qkv = ops.linear(x, self.w_qkv)
-        q, k, v = qkv[:, :qw], qkv[:, qw:qw + kw], qkv[:, qw + kw:]
+        q, k = qkv[:, :qw], qkv[:, qw:qw + kw]
+        at = qw + kw
+        if self.values_from_keys:
+            v = k                                    # read before the rotation: k goes to the cache only
+        else:
+            v = qkv[:, at:at + Hkv * dv]
+            at += Hkv * dv
+        gate = qkv[:, at:at + H] if self.head_gate else None
         table, rot, interleaved = None, 0, False
         if self.position is not None:
             table, rot = self.position.table(ctx), self.position.rotary_dim
@@ -216,7 +252,7 @@ class SinkAttention(Part):
                                     rot, interleaved, cache.slots, cache.k, cache.v, cache.page_size)
         a = torch.empty((x.shape[0], H * dv), dtype=q.dtype, device=q.device)
         sink_attention(q, a, H, Hkv, dk, dv, cache, ctx, self.scale, self.window or 0, self.sinks,
-                       softcap=self.softcap, keep_first=self.keep_first, dist_bias=self.dist_bias)
+                       softcap=self.softcap, keep_first=self.keep_first, dist_bias=self.dist_bias, gate=gate)
         return ops.linear(a, self.w_o, out_dtype=self.out_dtype)
 
 
@@ -237,10 +273,11 @@ def tile_form(H, Hkv, dk, dv, value_row, dtype):
 
 
 def sink_attention(q, out, H, Hkv, dk, dv, cache, ctx, scale, window, sinks, softcap=0.0,
-                   value_row=0, keep_first=0, dist_bias=None) -> None:
+                   value_row=0, keep_first=0, dist_bias=None, gate=None) -> None:
     """`keep_first`: the first keys of a request that stay visible beside the window; `dist_bias`
-    [n, H]: added to the scores by distance. `softcap` bounds the scores; `value_row` > 0 says that a value is the first dv channels
-    of its key row, `value_row` wide (one cache plane serves as keys and values).
+    [n, H]: added to the scores by distance; `gate` [T, H]: every head's output times the logistic
+    function of its number. `softcap` bounds the scores; `value_row` > 0 says that a value is the first
+    dv channels of its key row, `value_row` wide (one cache plane serves as keys and values).
     Which kernel runs the attention of a step. bfloat16 at sizes a tensor-core kernel takes
     (`tile_form`): that kernel, over tiles of consecutive tokens for steps with prompt portions
     (single tokens beside them are tiles of one), a tile a token for steps of single tokens, whose
@@ -248,8 +285,8 @@ def sink_attention(q, out, H, Hkv, dk, dv, cache, ctx, scale, window, sinks, sof
     and other sizes: the generic kernel (a warp per token and head, keys in a fixed order)."""
     v_cache = cache.k if value_row else cache.v
     form, tokens = tile_form(H, Hkv, dk, dv, value_row, q.dtype)
-    if form == "wide" and (keep_first or dist_bias is not None):
-        form = None                     # the kernel for wide rows knows neither
+    if form == "wide" and (keep_first or dist_bias is not None or gate is not None):
+        form = None                     # the kernel for wide rows knows none of them
     if form is not None and ops.attention_sink_takes(q, out):
         tok0, ntok = (None, None) if ctx.decode_only else step_tiles(ctx, tokens)
         if form == "wide":
@@ -265,12 +302,12 @@ def sink_attention(q, out, H, Hkv, dk, dv, cache, ctx, scale, window, sinks, sof
         ops.attention_sink_tile(q, out, H, Hkv, dk, dv, cache.k, v_cache, cache.page_size,
                                 cache.block_tables, ctx.seq_ids, ctx.positions, scale, window, sinks,
                                 tok0, ntok, n_splits=splits, softcap=softcap, value_row=value_row,
-                                keep_first=keep_first, dist_bias=dist_bias)
+                                keep_first=keep_first, dist_bias=dist_bias, gate=gate)
         return
     ops.attention_generic(q, out, H, Hkv, dk, cache.k, v_cache, cache.page_size,
                           cache.block_tables, ctx.seq_ids, ctx.positions, scale, window,
                           value_dim=dv, sinks=sinks, softcap=softcap, value_row=value_row,
-                          keep_first=keep_first, dist_bias=dist_bias)
+                          keep_first=keep_first, dist_bias=dist_bias, gate=gate)
 
 
 MIXERS.register("sink_attention", SinkAttention)

@@ -26,7 +26,9 @@ Interfaces (duck-typed; `Part` only supplies the defaults):
                   `ops.NormedRows` (it passes x to `ops.linear` / `ops.gated_linear`, or asks
                   `ops.rows_of(x)` for the tensor); without it a part always gets a tensor.
   block           forward(h, pending, ctx, cache) -> (h, pending): `pending` is a delta
-                  not yet added to h, so the add can be fused into the next norm.
+                  not yet added to h, so the add can be fused into the next norm. A block whose
+                  class sets `takes_normed = True` also accepts and may hand on a `NormedDelta`
+                  (rows that join the stream through a norm); the model settles it for others.
 
 A part's constructor gets (its spec, the hidden width, the layer's tensor-name prefix, the
 device); the checkpoint names of its weights are in its spec's `tensors` table, which the
@@ -52,6 +54,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
+from ..kernels import ops
 from ..weights.binder import WeightSpec
 
 
@@ -143,6 +146,20 @@ class StepContext:
     max_context: int = 0
     decode_only: bool = False        # every request brings exactly one token
     aux: Dict[str, object] = field(default_factory=dict)   # per-step device tensors made once
+
+
+@dataclass
+class NormedDelta:
+    """A sublayer's result that is to join the stream through a norm, h += extra + norm(y), and has
+    not yet: the next block may do it in the kernel of its own norm."""
+    norm: object                     # a norm part with `add_scaled` (and `join`)
+    y: torch.Tensor                  # float32 [T, d]
+    extra: Optional[torch.Tensor] = None     # float32 [T, d] that joins the stream too
+
+    def settle(self, h: torch.Tensor) -> None:
+        self.norm.add_scaled(h, self.y, None)
+        if self.extra is not None:
+            ops.residual_add(h, self.extra)
 
 
 class Part:

@@ -20,7 +20,7 @@ from ..config.spec import LayerSpec, tensor_names
 from ..kernels import ops
 from ..registry import BLOCKS, FEED_FORWARDS, MIXERS, NORMS
 from ..weights.binder import WeightSpec
-from .base import Part, offered
+from .base import NormedDelta, Part, offered
 
 
 class PreNormResidual(Part):
@@ -207,9 +207,13 @@ class SandwichNormResidual(Part):
         h = h + norm1b(mixer(norm1(h)));  h = h + norm2b(feed_forward(norm2(h)))
 
     The stream, the four norms and the adds are float32; the sublayers read the normed rows
-    in the activation type and hand back float32 rows. A layer may have no feed-forward (it
-    then has no second pair of norms). Tensor roles of the layer spec: mixer_norm,
+    in the activation type and hand back float32 rows. Norms that offer `join` (plain RMS norms) are
+    run two at a time, a sublayer's output norm with the next one's input norm; the last one of the
+    layer is then left to the block that follows (NormedDelta). A layer may have no feed-forward
+    (it then has no second pair of norms). Tensor roles of the layer spec: mixer_norm,
     mixer_out_norm, ffn_norm, ffn_out_norm."""
+
+    takes_normed = True
 
     def __init__(self, spec: LayerSpec, hidden: int, device=None):
         p = spec.prefix
@@ -272,11 +276,27 @@ class SandwichNormResidual(Part):
         return offered(self.mixer, "cache_bytes_read")(context_len, width)
 
     def forward(self, h, pending, ctx, cache):
-        y = self.mixer.forward(self.norm1.forward(h, pending, ctx.act_dtype), ctx, cache)
-        self.norm1b.add_scaled(h, y, None)
+        if isinstance(pending, NormedDelta):
+            if hasattr(pending.norm, "join") and hasattr(self.norm1, "join"):
+                n = pending.norm.join(h, pending.y, self.norm1, ctx.act_dtype, pending.extra)
+            else:
+                pending.settle(h)
+                n = self.norm1.forward(h, None, ctx.act_dtype)
+        else:
+            n = self.norm1.forward(h, pending, ctx.act_dtype)
+        y = self.mixer.forward(n, ctx, cache)
+        joins = hasattr(self.norm1b, "join") and y.dtype == torch.float32
+        last = self.norm1b
         if self.feed_forward is not None:
-            y = self.feed_forward.forward(self.norm2.forward(h, None, ctx.act_dtype), ctx)
-            self.norm2b.add_scaled(h, y, None)
+            if joins:
+                n = self.norm1b.join(h, y, self.norm2, ctx.act_dtype)
+            else:
+                self.norm1b.add_scaled(h, y, None)
+                n = self.norm2.forward(h, None, ctx.act_dtype)
+            y, last = self.feed_forward.forward(n, ctx), self.norm2b
+        if joins and y.dtype == torch.float32:
+            return h, NormedDelta(last, y)
+        last.add_scaled(h, y, None)
         return h, None
 
 

@@ -176,7 +176,8 @@ class RoutedExperts(Part):
     the router matrix's last row, so its logit is a float32 sum too); `router_scores` "sigmoid",
     as "all" with the logistic function of each logit as its score; `router_groups` (count, keep),
     the router outputs fall into `count` equal runs of neighbours, a run counts as the sum of its
-    two largest choice scores, and only the outputs of the best `keep` runs can be chosen;
+    two largest choice scores (`router_group_best` 1: as its largest alone), and only the outputs of
+    the best `keep` runs can be chosen;
     `router_renormalize` False, the weights are the chosen scores as they are; `router_scale`, a
     factor on the weights.
 
@@ -197,7 +198,10 @@ class RoutedExperts(Part):
         self.renormalize = bool(getattr(spec, "router_renormalize", True))
         self.route_scale = float(getattr(spec, "router_scale", 1.0))
         self.groups, self.keep = getattr(spec, "router_groups", None) or (1, 1)
+        self.group_best = int(getattr(spec, "router_group_best", 2))
         outputs = self.E + self.identity
+        if self.group_best not in (1, 2):
+            raise ValueError(f"routed feed-forward: a group counted by {self.group_best} scores; 1 or 2")
         if self.groups < 1 or outputs % self.groups or not 0 < self.keep <= self.groups or \
                 self.keep * (outputs // self.groups) < self.top:
             raise ValueError(f"routed feed-forward: {self.keep} of {self.groups} groups of "
@@ -295,7 +299,7 @@ class RoutedExperts(Part):
                                  self.w_down, self.top, self.activation, extra, self.scores,
                                  self.router_correction, self.identity, self.shared_gate,
                                  self.groups, self.keep, self.renormalize, self.route_scale,
-                                 beside, residual)
+                                 beside, residual, self.group_best)
         if residual is not None:
             return None
         want = self.out_dtype or ctx.act_dtype

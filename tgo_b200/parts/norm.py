@@ -56,6 +56,25 @@ class RMSNorm(Part):
         ops.add_rmsnorm(h, delta, self.gain, self.eps, out, rows)
         return out
 
+    def of_embedding(self, table: torch.Tensor, ids: torch.Tensor, scale: float, h: torch.Tensor,
+                     copy: Optional[torch.Tensor] = None) -> None:
+        """h = norm(table[ids] * scale), float32, in the gather's kernel; the same rows in `copy`."""
+        ops.embed_rmsnorm(table, ids, self.gain, self.eps, h, copy, scale)
+
+    def add_scaled(self, h: torch.Tensor, y: torch.Tensor, scale: Optional[torch.Tensor],
+                   act: Optional[torch.Tensor] = None) -> None:
+        """h += scale * gain * norm(y), the stream h in float32; `act` also gets the new stream in
+        the activation type."""
+        ops.group_norm_scale_add(h, y, self.gain, scale, self.eps, 1, act)
+
+    def join(self, h: torch.Tensor, y: torch.Tensor, after, out_dtype: torch.dtype,
+             extra: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """h <- h + extra + norm(y), and back come the rows that `after`, another plain RMS norm,
+        makes of the new stream: two norms in one kernel."""
+        out = torch.empty(h.shape, dtype=out_dtype, device=h.device)
+        ops.norm_add_norm(h, y, self.gain, self.eps, after.gain, after.eps, out, extra)
+        return out
+
     def scaled_add_norm(self, h: torch.Tensor, y: torch.Tensor, bias: Optional[torch.Tensor],
                         alpha: float, act: Optional[torch.Tensor] = None) -> None:
         """h <- gain * norm(alpha * h + y + bias): the stream itself is normed, in place, for

@@ -79,6 +79,9 @@ def _register_builtin() -> None:
     from .config import bekunex
     if bekunex.ARCHITECTURE not in ARCHITECTURES:
         ARCHITECTURES.register(bekunex.ARCHITECTURE, bekunex.bekunex_model_spec)
+    from .config import kesozen
+    if kesozen.ARCHITECTURE not in ARCHITECTURES:
+        ARCHITECTURES.register(kesozen.ARCHITECTURE, kesozen.kesozen_model_spec)
 
 
 _register_builtin()
