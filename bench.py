@@ -567,6 +567,57 @@ def bekunex_beside_totatar(args):
     return 0
 
 
+def kesozen_config(width, heads, kv, dim, ff, layers, vocab=32768):
+    """(delta, delta, attention) repeated over `layers` layer runs, the first layer run twice in a
+    row: delta heads of 128 x 128 and 32 experts in 4 groups of which 2 stay open, top 4, after them;
+    attention of the given heads with a rotation of half of every head and a dense feed-forward."""
+    delta = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4},
+             "mlp": {"kind": "moe", "router": {"experts": 32, "top": 4, "groups": {"count": 4, "keep": 2}},
+                     "expert": {"ff": ff // 8}}}
+    att = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+           "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                     "rot": {"dims": dim // 2, "base": 5e5}}}
+    runs = [att if i % 3 == 2 else delta for i in range(layers)]
+    return {"architecture": "Kesozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": runs[1:], "loop": {"start": 0, "stop": 1, "times": 2}}
+
+
+def kesozen_beside_totatar(args):
+    """One JSON line per measurement: prefill of 2,048 tokens and decode at batch 8 and 64 for
+    Kesozen and for Totatar (the closest model the engine has: norms around both sublayers, a
+    recurrence with a 32-bit matrix state, attention with a sink, routed experts) at each size; then
+    Kesozen's kernels one by one beside their like kernels."""
+    import torch
+
+    import tgo_b200
+    from tgo_b200.engine.measure import load_peaks, measure_decode, measure_prefill
+    from tgo_b200.engine.measure_kernels import measure_kesozen_kernels
+    peaks = load_peaks()
+    layers = args.layers or 6
+    steps = min(args.steps, 64)
+    for name, (width, heads, kv, dim, ff) in DESIGN_SIZES.items():
+        for arch, make in (("kesozen", kesozen_config), ("totatar", totatar_config)):
+            model = tgo_b200.open_random(make(width, heads, kv, dim, ff, layers), seed=SEED,
+                                         dtype="bfloat16", sigma=0.02, gain_sigma=0.05)
+            pre = measure_prefill(model, PREFILL_TOKENS, warmup=2, steps=3, seed=SEED, page_size=PAGE)
+            rec = {"size": name, "model": arch, "layers": layers,
+                   "prefill_ms": round(pre["ms"], 3), "prefill_tokens_per_s": round(pre["tokens_per_s"]),
+                   "prefill_frac_of_library_peak": round(pre["tflops"] / peaks["bf16_tflops"], 3)}
+            for b in (8, 64):
+                r = measure_decode(model, b, PROMPT, steps, warmup=max(args.warmup, 3), seed=SEED,
+                                   page_size=PAGE)
+                rec[f"decode_b{b}_ms"] = round(r["ms_per_step"], 4)
+                rec[f"decode_b{b}_tokens_per_s"] = round(r["tokens_per_s"])
+                rec[f"decode_b{b}_hbm_frac"] = round(r["gbs"] / peaks["hbm_gbs"], 3)
+            print(json.dumps(rec), flush=True)
+            del model
+            torch.cuda.empty_cache()
+        for rec in measure_kesozen_kernels(width, heads, kv, dim, heads, heads, 128, 128, 4, 32, 4, 4, 2, ff // 8):
+            rec["size"] = name
+            print(json.dumps(rec), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -582,7 +633,7 @@ def main():
     ap.add_argument("--rows", default="256,512,1024,2048", help="with --only products: row counts")
     ap.add_argument("--only", default="", choices=["", "prefill", "decode", "serve", "check", "products",
                                                    "gafonex", "totatar", "derosun", "vimelorn",
-                                                   "bekunex"],
+                                                   "bekunex", "kesozen"],
                     help="run just the 2,048-token prefill, just the decode steps, the "
                          "continuous-batching workload, or the exactness check at real layer "
                          "sizes (float32 against bfloat16, alone against cut and mixed; 4 layers "
@@ -599,7 +650,9 @@ def main():
                          "a bias by distance, routed small experts) beside Totatar and Qwen3 in "
                          "the same way; bekunex: the Bekunex design (latent attention with a "
                          "window and lent latents, scans with a decay per channel, experts in "
-                         "groups beside the mixer) beside Totatar and Derosun in the same way")
+                         "groups beside the mixer) beside Totatar and Derosun in the same way; "
+                         "kesozen: the Kesozen design (a gated delta rule, attention whose values are "
+                         "its keys, experts in groups, a loop of layers) beside Totatar in the same way")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -626,6 +679,8 @@ def main():
         return vimelorn_beside_totatar(args)
     if args.only == "bekunex":
         return bekunex_beside_totatar(args)
+    if args.only == "kesozen":
+        return kesozen_beside_totatar(args)
     config, seed = dict(SHAPES[args.shape][0]), SHAPES[args.shape][1]
     if args.layers:
         config["num_hidden_layers"] = args.layers

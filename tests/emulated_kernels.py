@@ -479,21 +479,22 @@ def delta_prepare(x, w, b_raw, a_raw, dt_bias, decay, num_seqs, heads, groups, k
     causal_conv_act(x, w.t().contiguous(), None, rows, num_seqs, seq_ids, q_start, state_slots, state, conv_offset,
                     keep=False)
     kw = groups * key_dim
-    qk = torch.zeros((T, groups, 2, (key_dim + 31) // 32 * 32))
+    qk = torch.zeros((T, groups, 2, key_dim))
     for j in range(2):
         z = rows[:, j * kw:(j + 1) * kw].reshape(T, groups, key_dim)
         qk[:, :, j, :key_dim] = z * torch.rsqrt((z * z).sum(-1, keepdim=True) + 1e-6) * \
             (key_dim ** -0.5 if j == 0 else 1.0)
     log_g = -decay * torch.nn.functional.softplus(a_raw.float() + dt_bias, threshold=1e9)
-    gates = torch.stack([torch.exp(log_g), torch.expm1(log_g), torch.sigmoid(b_raw.float()),
-                         torch.zeros_like(log_g)], dim=2).contiguous()
-    pairs = torch.zeros((T, groups, 4))              # of use to the kernels' pairs of tokens only
-    return qk, rows[:, 2 * kw:].contiguous(), gates, pairs
+    beta = torch.sigmoid(b_raw.float())
+    v = (rows[:, 2 * kw:].reshape(T, heads, value_dim) * beta[:, :, None]).reshape(T, -1).contiguous()
+    records = torch.zeros((T, heads, 12))            # as for a token without others beside it
+    records[:, :, 0], records[:, :, 8] = beta * torch.exp(log_g), torch.exp(log_g)
+    return qk, v, records
 
 
 def delta_scan(prepared, y, num_seqs, heads, groups, key_dim, value_dim, q_start, state_slots, state, mem_offset,
                conv_in, taps, conv_offset):
-    qk, v, gates, _ = prepared
+    qk, v, records = prepared
     per, C = heads // groups, conv_in.shape[1]
     for b in range(num_seqs):
         t0, t1 = int(q_start[b]), int(q_start[b + 1])
@@ -501,10 +502,8 @@ def delta_scan(prepared, y, num_seqs, heads, groups, key_dim, value_dim, q_start
         S = row[mem_offset:mem_offset + heads * key_dim * value_dim].view(heads, key_dim, value_dim)
         for t in range(t0, t1):
             q, k = (qk[t, :, j, :key_dim].repeat_interleave(per, dim=0) for j in range(2))
-            g, beta = gates[t, :, 0], gates[t, :, 2]
-            S.mul_(g[:, None, None])
-            u = beta[:, None] * (v[t].reshape(heads, value_dim) - torch.einsum("hkv,hk->hv", S, k))
-            S.add_(k[:, :, None] * u[:, None, :])
+            u = v[t].reshape(heads, value_dim) - records[t, :, 0, None] * torch.einsum("hkv,hk->hv", S, k)
+            S.mul_(records[t, :, 8, None, None]).add_(k[:, :, None] * u[:, None, :])
             y[t] = torch.einsum("hkv,hk->hv", S, q).reshape(-1)
         keep = taps - 1
         if keep:

@@ -8,16 +8,20 @@
 // dt_bias)) and beta = sigmoid(b) are one number per head and token. Head h uses the q and k of head
 // floor(h / (H / G)). Everything after the projections is float32 whatever their storage type.
 //
-// Tokens are taken in pairs (0 1)(2 3).. from a request's first token of the step, so that the two
-// reads of the memory by k and the two by q meet the same S. With c = k0.k1, d_ij = k_i.q_j:
+// Tokens are taken four at a time, (0 1 2 3)(4 5 6 7).. from a request's first token of the step, so
+// that the reads of the memory by four k and four q meet the same S and the exchanges between
+// threads are paid once. With P_j = g_0 .. g_j, E_j = g_j+1 .. g_last and S as it was before the four:
 //
-//   u0 = b0 (v0 - g0 S^T k0)                   o0 = g0 S^T q0 + d00 u0
-//   u1 = b1 (v1 - g1 (g0 S^T k1 + c u0))       o1 = g1 (g0 S^T q1 + d01 u0) + d11 u1
-//   S' = g1 g0 S + k0 (g1 u0)^T + k1 u1^T
+//   u_j = b_j v_j - b_j P_j S^T k_j - sum_(m<j) b_j (P_j / P_m) (k_m.k_j) u_m
+//   o_j = P_j S^T q_j + sum_(m<=j) (P_j / P_m) (k_m.q_j) u_m
+//   S'  = P_last S + sum_j k_j (E_j u_j)^T
 //
-//   prepare   rows [T, G, 2, DKP] float32 (q, then k, unit vectors, padded with zeros to DKP = dk
-//             rounded up to 32), values [T, H, dv] float32, gates [T, H] (g, g - 1, beta, 0) and
-//             pairs [T, G] (k.q of the token; k and q of a pair's second token with the first's k)
+// where the ratios are exponentials of sums of the tokens' log decays, and every factor that does not
+// depend on S is made ahead:
+//
+//   prepare   rows [T, G, 2, DKP] float32 (q, then k, unit vectors, padded with zeros to DKP = 32, 64,
+//             128 or 256), values b v [T, H, dv] float32 and records [T, H, 12]: for token j of a four
+//             (b P_j, b x the three k_m.k_j terms; the four k_m.q_j terms; P_j, E_j, P_last, P_last - 1)
 //   scan      the rule over requests of any number of tokens; y [T, H dv] float32
 //   step      the rule for requests of one token each, with the norm and the gate behind it
 //
@@ -26,6 +30,8 @@
 // dk + H dv channels in the order q, k, v. The prepare kernel reads the kept inputs, the kernel
 // after it moves them on.
 #include "common.cuh"
+
+static int delta_row_width(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 128 ? 128 : 256; }
 
 template <typename T> __device__ __forceinline__ float dl_exp(float x);
 template <> __device__ __forceinline__ float dl_exp<float>(float x) { return expf(x); }
@@ -57,156 +63,241 @@ template <> __device__ __forceinline__ void dl_store<4>(float* p, const float* v
 }
 
 // --------------------------------------------------------------------------------- prepare
-// The convolution and SiLU of VEC channels from c on for a pair: token t0 (place r0 of its portion)
-// and the next one. Rows before the portion are the request's kept inputs. w [taps][C].
-template <typename T, int VEC>
-__device__ __forceinline__ void dl_conv_pair(float* y0, float* y1, bool two, const T* __restrict__ x,
-                                             long long x_stride, const float* __restrict__ w, int C, int c,
-                                             int taps, int t0, int r0, const float* __restrict__ kept) {
+// The convolution and SiLU of VEC channels from c on for up to four tokens: t0 (place r0 of its
+// portion) and the `count - 1` after it. Rows before the portion are the request's kept inputs. w
+// [taps][C]. Tokens past `count` come out as zeros.
+#define DP_GROUP 4
+template <typename T, int VEC, int TAPS>
+__device__ __forceinline__ void dl_conv(float (*y)[VEC], int count, const T* __restrict__ x, long long x_stride,
+                                        const float* __restrict__ w, int C, int c, int taps, int t0, int r0,
+                                        const float* __restrict__ kept) {
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) y0[i] = y1[i] = 0.f;
-    for (int j = 0; j <= taps; ++j) {
-        const int back = taps - 1 - j;                   // tokens before t0; -1: the pair's second token
-        if (back < 0 && !two) break;
-        float v[VEC], wj[VEC];
+    for (int u = 0; u < DP_GROUP; ++u)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[u][i] = 0.f;
+    auto input = [&](float* v, int back) {               // `back` tokens before t0; negative: after it
         if (back <= r0) dl_load<T, VEC>(v, x + (long long)(t0 - back) * x_stride + c);
         else dl_load<float, VEC>(v, kept + (size_t)(taps - 1 - (back - r0)) * C + c);
-        if (j < taps) {
-            dl_load<float, VEC>(wj, w + (size_t)j * C + c);
+    };
+    if (TAPS > 0) {                                      // every load ahead of the sums
+        float v[TAPS + DP_GROUP - 1][VEC], wt[TAPS > 0 ? TAPS : 1][VEC];
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) y0[i] = fmaf(wj[i], v[i], y0[i]);
+        for (int j = 0; j < TAPS + DP_GROUP - 1; ++j) {
+            if (j - (TAPS - 1) < count) {
+                input(v[j], TAPS - 1 - j);
+            } else {
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) v[j][i] = 0.f;
+            }
         }
-        if (j > 0) {
-            dl_load<float, VEC>(wj, w + (size_t)(j - 1) * C + c);
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) y1[i] = fmaf(wj[i], v[i], y1[i]);
+        for (int q = 0; q < TAPS; ++q) dl_load<float, VEC>(wt[q], w + (size_t)q * C + c);
+#pragma unroll
+        for (int u = 0; u < DP_GROUP; ++u)
+#pragma unroll
+            for (int q = 0; q < TAPS; ++q)
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) y[u][i] = fmaf(wt[q][i], v[u + q][i], y[u][i]);
+    } else {
+        for (int j = 0; j < taps + DP_GROUP - 1 && j - (taps - 1) < count; ++j) {
+            float v[VEC];
+            input(v, taps - 1 - j);
+#pragma unroll
+            for (int u = 0; u < DP_GROUP; ++u) {         // this input meets tap j - u of token u
+                if (j < u || j - u >= taps) continue;
+                float wj[VEC];
+                dl_load<float, VEC>(wj, w + (size_t)(j - u) * C + c);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) y[u][i] = fmaf(wj[i], v[i], y[u][i]);
+            }
         }
     }
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) {
-        y0[i] = dl_silu<T>(y0[i]);
-        y1[i] = dl_silu<T>(y1[i]);                       // of no use without a second token
-    }
+    for (int u = 0; u < DP_GROUP; ++u)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[u][i] = u < count ? dl_silu<T>(y[u][i]) : 0.f;
 }
 
-// A warp takes a pair and a unit: unit u < G is q and k of head u, the next `v_units` are runs of
-// 32 VEC value channels, the rest 32 heads' gates each. NV rounds of 32 VEC channels cover DKP.
-#define DP_WARPS 8
-template <typename T, int VEC, int NV>
-__global__ void __launch_bounds__(32 * DP_WARPS)
-delta_prepare_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ w,
-                     const T* __restrict__ b_raw, const T* __restrict__ a_raw, long long gate_stride,
-                     const float* __restrict__ dt_bias, const float* __restrict__ A, float* __restrict__ qk,
-                     float* __restrict__ v_out, float4* __restrict__ gates, float4* __restrict__ pairs, int Tn,
-                     int H, int G, int dk, int dv, int dkp, int taps, float q_scale, int v_units,
-                     const int* __restrict__ seq_ids, const int* __restrict__ q_start,
-                     const int* __restrict__ state_slots, const float* __restrict__ state,
-                     long long state_stride, long long conv_offset) {
-    pdl_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x * DP_WARPS + warp;
-    if (t >= Tn) return;
-    const int b = seq_ids[t], r = t - q_start[b];
-    if (r & 1) return;                                   // the second of a pair
-    const bool two = t + 1 < q_start[b + 1];
+// A warp takes four tokens and a unit: unit u < G is q and k of head u and the records of
+// its group's heads, the others are runs of 32 VEC value channels. NV rounds of 32 VEC channels cover DKP.
+// A warp looks for the first tokens of fours among `per` consecutive ones: 4 in prompts, 1 in steps of
+// single tokens.
+#define DP_WARPS 4
+template <typename T, int VEC, int NV, int TAPS>
+__device__ __forceinline__ void
+delta_prepare_four(int t, int b, int r, const T* __restrict__ x, long long x_stride, const float* __restrict__ w,
+                   const T* __restrict__ b_raw, const T* __restrict__ a_raw, long long gate_stride,
+                   const float* __restrict__ dt_bias, const float* __restrict__ A, float* __restrict__ qk,
+                   float* __restrict__ v_out, float4* __restrict__ records,
+                   int H, int G, int dk, int dv, int dkp, int taps, float q_scale,
+                   const int* __restrict__ q_start, const int* __restrict__ state_slots,
+                   const float* __restrict__ state, long long state_stride, long long conv_offset) {
+    const int lane = threadIdx.x & 31;
+    const int left = q_start[b + 1] - t, count = left < DP_GROUP ? left : DP_GROUP;
     const int C = 2 * G * dk + H * dv;
     const float* kept = state + (size_t)state_slots[b] * state_stride + conv_offset;
     const int unit = blockIdx.y;
-    if (unit >= G + v_units) {                           // gates
-        const int h = (unit - G - v_units) * 32 + lane;
-        if (h >= H) return;
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-            if (j && !two) break;
-            const float z = to_f32(a_raw[(size_t)(t + j) * gate_stride + h]) + dt_bias[h];
-            const float sp = z > 20.f ? z : log1pf(expf(z));
-            const float l = -A[h] * sp;
-            gates[(size_t)(t + j) * H + h] =
-                make_float4(expf(l), expm1f(l), dl_sigmoid<float>(to_f32(b_raw[(size_t)(t + j) * gate_stride + h])), 0.f);
-        }
-        return;
-    }
-    if (unit >= G) {                                     // values
+    if (unit >= G) {                                     // values, times their steps
         const int c = ((unit - G) * 32 + lane) * VEC;
         if (c >= H * dv) return;
-        float y0[VEC], y1[VEC];
-        dl_conv_pair<T, VEC>(y0, y1, two, x, x_stride, w, C, 2 * G * dk + c, taps, t, r, kept);
-        dl_store<VEC>(v_out + (size_t)t * H * dv + c, y0);
-        if (two) dl_store<VEC>(v_out + (size_t)(t + 1) * H * dv + c, y1);
+        float y[DP_GROUP][VEC];
+        dl_conv<T, VEC, TAPS>(y, count, x, x_stride, w, C, 2 * G * dk + c, taps, t, r, kept);
+#pragma unroll
+        for (int u = 0; u < DP_GROUP; ++u)
+            if (u < count) {
+                const float beta = dl_sigmoid<T>(to_f32(b_raw[(size_t)(t + u) * gate_stride + c / dv]));
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) y[u][i] *= beta;
+                dl_store<VEC>(v_out + (size_t)(t + u) * H * dv + c, y[u]);
+            }
         return;
     }
-    float q[2][NV * VEC], k[2][NV * VEC];
-    float s[8];                                          // q0q0 q1q1 k0k0 k1k1 k0q0 k1q1 k0k1 k0q1
+    float q[NV][DP_GROUP][VEC], k[NV][DP_GROUP][VEC];
+    // sums 0-3 q_j.q_j, 4-7 k_j.k_j, 8-11 k_j.q_j, 12-17 c_ij, 18-23 d_ij for ij = 01 02 12 03 13 23
+    float s[32];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) s[i] = 0.f;
+    for (int i = 0; i < 32; ++i) s[i] = 0.f;
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
         const int c = (n * 32 + lane) * VEC;
-        float* q0 = q[0] + n * VEC;
-        float* q1 = q[1] + n * VEC;
-        float* k0 = k[0] + n * VEC;
-        float* k1 = k[1] + n * VEC;
         if (c < dk) {
-            dl_conv_pair<T, VEC>(q0, q1, two, x, x_stride, w, C, unit * dk + c, taps, t, r, kept);
-            dl_conv_pair<T, VEC>(k0, k1, two, x, x_stride, w, C, (G + unit) * dk + c, taps, t, r, kept);
+            dl_conv<T, VEC, TAPS>(q[n], count, x, x_stride, w, C, unit * dk + c, taps, t, r, kept);
+            dl_conv<T, VEC, TAPS>(k[n], count, x, x_stride, w, C, (G + unit) * dk + c, taps, t, r, kept);
         } else {
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) q0[i] = q1[i] = k0[i] = k1[i] = 0.f;
+            for (int u = 0; u < DP_GROUP; ++u)
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) q[n][u][i] = k[n][u][i] = 0.f;
         }
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
-            s[0] = fmaf(q0[i], q0[i], s[0]);
-            s[1] = fmaf(q1[i], q1[i], s[1]);
-            s[2] = fmaf(k0[i], k0[i], s[2]);
-            s[3] = fmaf(k1[i], k1[i], s[3]);
-            s[4] = fmaf(k0[i], q0[i], s[4]);
-            s[5] = fmaf(k1[i], q1[i], s[5]);
-            s[6] = fmaf(k0[i], k1[i], s[6]);
-            s[7] = fmaf(k0[i], q1[i], s[7]);
+            int at = 0;
+#pragma unroll
+            for (int u = 0; u < DP_GROUP; ++u) {
+                s[u] = fmaf(q[n][u][i], q[n][u][i], s[u]);
+                s[4 + u] = fmaf(k[n][u][i], k[n][u][i], s[4 + u]);
+                s[8 + u] = fmaf(k[n][u][i], q[n][u][i], s[8 + u]);
+#pragma unroll
+                for (int m = 0; m < u; ++m, ++at) {
+                    s[12 + at] = fmaf(k[n][m][i], k[n][u][i], s[12 + at]);
+                    s[18 + at] = fmaf(k[n][m][i], q[n][u][i], s[18 + at]);
+                }
+            }
         }
     }
-    // eight sums over 32 lanes: with each of the first rounds a lane keeps half of its values; sum i
-    // ends in the lanes whose bits 4, 3, 2 spell i
+    // 32 sums over 32 lanes: with each round a lane keeps half of its values, lane i ends with sum i
 #pragma unroll
-    for (int o = 4; o > 0; o >>= 1) {
-        const bool up = lane & (o * 4);
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool up = lane & o;
 #pragma unroll
         for (int i = 0; i < o; ++i) {
             const float give = up ? s[i] : s[i + o], have = up ? s[i + o] : s[i];
-            s[i] = have + __shfl_xor_sync(0xffffffffu, give, o * 4);
+            s[i] = have + __shfl_xor_sync(0xffffffffu, give, o);
         }
     }
-    float sum = s[0];
-    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-    float f[8];
+    const float inv = 1.f / sqrtf(s[0] + 1e-6f);         // lanes 0-7: one over the lengths of q_j, k_j
+    float rq[DP_GROUP], rk[DP_GROUP];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) f[i] = __shfl_sync(0xffffffffu, sum, 4 * i);
-    const float rq0 = q_scale / sqrtf(f[0] + 1e-6f), rq1 = q_scale / sqrtf(f[1] + 1e-6f);
-    const float rk0 = 1.f / sqrtf(f[2] + 1e-6f), rk1 = 1.f / sqrtf(f[3] + 1e-6f);
-    float* row = qk + ((size_t)t * G + unit) * 2 * dkp;
+    for (int u = 0; u < DP_GROUP; ++u) {
+        rq[u] = __shfl_sync(0xffffffffu, inv, u) * q_scale;
+        rk[u] = __shfl_sync(0xffffffffu, inv, 4 + u);
+    }
     const size_t next = (size_t)G * 2 * dkp;
+    float* row = qk + ((size_t)t * G + unit) * 2 * dkp;
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
         const int c = (n * 32 + lane) * VEC;
         if (c >= dkp) break;
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) {
-            q[0][n * VEC + i] *= rq0;
-            q[1][n * VEC + i] *= rq1;
-            k[0][n * VEC + i] *= rk0;
-            k[1][n * VEC + i] *= rk1;
-        }
-        dl_store<VEC>(row + c, q[0] + n * VEC);
-        dl_store<VEC>(row + dkp + c, k[0] + n * VEC);
-        if (two) {
-            dl_store<VEC>(row + next + c, q[1] + n * VEC);
-            dl_store<VEC>(row + next + dkp + c, k[1] + n * VEC);
+        for (int u = 0; u < DP_GROUP; ++u) {
+            if (u >= count) break;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) {
+                q[n][u][i] *= rq[u];
+                k[n][u][i] *= rk[u];
+            }
+            dl_store<VEC>(row + u * next + c, q[n][u]);
+            dl_store<VEC>(row + u * next + dkp + c, k[n][u]);
         }
     }
-    if (lane == 0) {
-        pairs[(size_t)t * G + unit] = make_float4(f[4] * rk0 * rq0, 0.f, 0.f, 0.f);
-        if (two) pairs[(size_t)(t + 1) * G + unit] = make_float4(f[5] * rk1 * rq1, f[6] * rk0 * rk1, f[7] * rk0 * rq1, 0.f);
+    // The records of the group's heads: lane 4 i + u is token u of the i-th of eight heads. Lanes 8 + j
+    // have k_j.q_j, lanes 12 + p and 18 + p the products of tokens m < j, p = j (j - 1) / 2 + m.
+    const int u = lane & 3, per_group = H / G;
+    const float rku = u == 0 ? rk[0] : u == 1 ? rk[1] : u == 2 ? rk[2] : rk[3];
+    const float rqu = u == 0 ? rq[0] : u == 1 ? rq[1] : u == 2 ? rq[2] : rq[3];
+    const float own = __shfl_sync(0xffffffffu, s[0], 8 + u) * rku * rqu;
+    float ck[3], cq[3];
+#pragma unroll
+    for (int m = 0; m < 3; ++m) {
+        const int at = u > m ? u * (u - 1) / 2 + m : 0;
+        ck[m] = __shfl_sync(0xffffffffu, s[0], 12 + at) * rk[m] * rku;
+        cq[m] = __shfl_sync(0xffffffffu, s[0], 18 + at) * rk[m] * rqu;
+    }
+    for (int h0 = 0; h0 < per_group; h0 += 8) {
+        const int hh = h0 + lane / 4, h = unit * per_group + (hh < per_group ? hh : per_group - 1);
+        float l = 0.f, beta = 0.f;
+        if (u < count) {
+            const float zz = to_f32(a_raw[(size_t)(t + u) * gate_stride + h]) + dt_bias[h];
+            l = -A[h] * (zz > 20.f ? zz : log1pf(expf(zz)));
+            beta = dl_sigmoid<T>(to_f32(b_raw[(size_t)(t + u) * gate_stride + h]));
+        }
+        // log decays: of the tokens up to this one, of those between m and this one, of those after it
+        float at[4], ratio[3];
+#pragma unroll
+        for (int m = 0; m < 4; ++m) at[m] = __shfl_sync(0xffffffffu, l, (lane & ~3) + m);
+        const float upto = at[0] + (u > 0 ? at[1] : 0.f) + (u > 1 ? at[2] : 0.f) + (u > 2 ? at[3] : 0.f);
+        const float all = at[0] + at[1] + at[2] + at[3];
+        const float later = (u < 1 ? at[1] : 0.f) + (u < 2 ? at[2] : 0.f) + (u < 3 ? at[3] : 0.f);
+        ratio[0] = (u > 0 ? at[1] : 0.f) + (u > 1 ? at[2] : 0.f) + (u > 2 ? at[3] : 0.f);
+        ratio[1] = (u > 1 ? at[2] : 0.f) + (u > 2 ? at[3] : 0.f);
+        ratio[2] = u > 2 ? at[3] : 0.f;
+        float pk[3], pq[4];
+#pragma unroll
+        for (int m = 0; m < 3; ++m) {
+            const float e = m < u ? expf(ratio[m]) : 0.f;
+            pk[m] = beta * e * ck[m];
+            pq[m] = e * cq[m];
+        }
+        pq[3] = 0.f;
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+            if (m == u) pq[m] = own;
+        if (u < count && hh < per_group) {
+            float4* rec = records + ((size_t)(t + u) * H + h) * 3;
+            const float p = expf(upto);
+            rec[0] = make_float4(beta * p, pk[0], pk[1], pk[2]);
+            rec[1] = make_float4(pq[0], pq[1], pq[2], pq[3]);
+            rec[2] = make_float4(p, expf(later), expf(all), expm1f(all));
+        }
+    }
+}
+
+template <typename T, int VEC, int NV, int TAPS>
+__global__ void __launch_bounds__(32 * DP_WARPS, VEC * NV <= 4 ? 6 : 4)
+delta_prepare_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ w,
+                     const T* __restrict__ b_raw, const T* __restrict__ a_raw, long long gate_stride,
+                     const float* __restrict__ dt_bias, const float* __restrict__ A, float* __restrict__ qk,
+                     float* __restrict__ v_out, float4* __restrict__ records, int Tn,
+                     int per, int H, int G, int dk, int dv, int dkp, int taps, float q_scale,
+                     const int* __restrict__ seq_ids, const int* __restrict__ q_start,
+                     const int* __restrict__ state_slots, const float* __restrict__ state,
+                     long long state_stride, long long conv_offset) {
+    pdl_wait();
+    const int first = (blockIdx.x * DP_WARPS + (threadIdx.x >> 5)) * per, lane = threadIdx.x & 31;
+    // the tokens of this warp that begin a four, looked up side by side
+    int b = 0, r = 1;
+    if (lane < per && first + lane < Tn) {
+        b = seq_ids[first + lane];
+        r = first + lane - q_start[b];
+    }
+    unsigned begins = __ballot_sync(0xffffffffu, r % DP_GROUP == 0);
+    while (begins) {
+        const int at = __ffs(begins) - 1;
+        begins &= begins - 1;
+        delta_prepare_four<T, VEC, NV, TAPS>(
+            first + at, __shfl_sync(0xffffffffu, b, at), __shfl_sync(0xffffffffu, r, at), x, x_stride, w, b_raw, a_raw,
+            gate_stride, dt_bias, A, qk, v_out, records, H, G, dk, dv, dkp, taps, q_scale, q_start, state_slots, state,
+            state_stride, conv_offset);
     }
 }
 
@@ -214,34 +305,38 @@ delta_prepare_kernel(const T* __restrict__ x, long long x_stride, const float* _
 // views with one stride; w float32 [taps][C], dt_bias and A = exp(A_log) float32 [H].
 TGO_API int tgo_delta_prepare(const void* x, long long x_stride, int dtype, const float* w, const void* b_raw,
                               const void* a_raw, long long gate_stride, const float* dt_bias, const float* A,
-                              float* qk, float* v_out, float* gates, float* pairs, int T, int B, int H, int G,
+                              float* qk, float* v_out, float* records, int T, int B, int H, int G,
                               int dk, int dv, int taps, const int* seq_ids, const int* q_start,
                               const int* state_slots, const float* state, long long state_stride,
                               long long conv_offset, cudaStream_t stream) {
     if (T <= 0 || B <= 0) return 0;
-    const int C = 2 * G * dk + H * dv, dkp = (dk + 31) / 32 * 32;
+    const int C = 2 * G * dk + H * dv, dkp = delta_row_width(dk);
     if (H <= 0 || G <= 0 || H % G || dk <= 0 || dk > 256 || dv <= 0 || taps <= 0 || taps > 64 ||
-        state_stride < conv_offset + (long long)(taps - 1) * C || (uintptr_t)qk % 16 || (uintptr_t)gates % 16 ||
-        (uintptr_t)pairs % 16 || (dtype != TGO_BF16 && dtype != TGO_F32))
+        state_stride < conv_offset + (long long)(taps - 1) * C || (uintptr_t)qk % 16 || (uintptr_t)records % 16 ||
+         (dtype != TGO_BF16 && dtype != TGO_F32))
         return TGO_E_BAD_ARG;
     const uintptr_t width = dtype == TGO_BF16 ? 8 : 16;  // bytes of four elements
     const bool quads = dk % 4 == 0 && dv % 4 == 0 && x_stride % 4 == 0 && (uintptr_t)x % width == 0 &&
                        (uintptr_t)w % 16 == 0 && (uintptr_t)v_out % 16 == 0 && (uintptr_t)state % 16 == 0 &&
                        state_stride % 4 == 0 && conv_offset % 4 == 0;
     const int per = quads ? 128 : 32, v_units = (H * dv + per - 1) / per;
-    const long long units = (long long)G + v_units + (H + 31) / 32;
+    const long long units = (long long)G + v_units;
     if (units > 65535) return TGO_E_BAD_ARG;
-    const dim3 grid((T + DP_WARPS - 1) / DP_WARPS, (unsigned)units);
+    const int each = T == B ? 1 : DP_GROUP;
+    const dim3 grid((T + DP_WARPS * each - 1) / (DP_WARPS * each), (unsigned)units);
     const float q_scale = 1.f / sqrtf((float)dk);
-#define DP_GO(TT, VEC, NV)                                                                                 \
-    tgo_launch_pdl(delta_prepare_kernel<TT, VEC, NV>, grid, dim3(32 * DP_WARPS), 0, stream, (const TT*)x, x_stride, \
-                   w, (const TT*)b_raw, (const TT*)a_raw, gate_stride, dt_bias, A, qk, v_out, (float4*)gates, \
-                   (float4*)pairs, T, H, G, dk, dv, dkp, taps, q_scale, v_units, seq_ids, q_start, state_slots, \
+#define DP_GO(TT, VEC, NV, TAPS)                                                                           \
+    tgo_launch_pdl(delta_prepare_kernel<TT, VEC, NV, TAPS>, grid, dim3(32 * DP_WARPS), 0, stream, (const TT*)x, x_stride, \
+                   w, (const TT*)b_raw, (const TT*)a_raw, gate_stride, dt_bias, A, qk, v_out, (float4*)records, T, \
+                   each, H, G, dk, dv, dkp, taps, q_scale, seq_ids, q_start, state_slots, \
                    state, state_stride, conv_offset)
-#define DP_SIZE(TT) (quads ? (dkp <= 128 ? DP_GO(TT, 4, 1) : DP_GO(TT, 4, 2))                              \
-                           : (dkp <= 64 ? DP_GO(TT, 1, 2) : dkp <= 128 ? DP_GO(TT, 1, 4) : DP_GO(TT, 1, 8)))
+#define DP_TAPS(TT, NV)                                                                                    \
+    (taps == 4 ? DP_GO(TT, 4, NV, 4) : taps == 3 ? DP_GO(TT, 4, NV, 3) : taps == 2 ? DP_GO(TT, 4, NV, 2)    \
+                                                                       : DP_GO(TT, 4, NV, 0))
+#define DP_SIZE(TT) (quads ? (dkp <= 128 ? DP_TAPS(TT, 1) : DP_TAPS(TT, 2)) : DP_GO(TT, 1, 8, 0))
     return dtype == TGO_BF16 ? DP_SIZE(bf16) : DP_SIZE(float);
 #undef DP_SIZE
+#undef DP_TAPS
 #undef DP_GO
 }
 
@@ -272,15 +367,14 @@ __device__ __forceinline__ void dl_keep_block(float* kept, const T* __restrict__
 }
 
 // ----------------------------------------------------------------------------------- scan
-// A block per (request, head, 16 columns of dv). A warp holds four columns, lane = 4 slice + column:
-// slice s keeps rows 32 i + 4 s + j (j = 0..3) of its column of S in registers for the whole walk
-// over the request's tokens. A pair costs four products with S, one exchange over the slices that
-// leaves a sum in each quarter of the warp, two broadcasts of the reads by k, and one update of S.
-// DS_TOK tokens at a time come through shared memory by asynchronous copies, two buffers. The order
-// of every sum depends on the sizes alone.
+// A block per (request, head, 16 or 32 columns of dv). L lanes of a warp share a column (the column in
+// the low bits of the lane): slice s keeps its rows 4 s + 4 L i + (0..3) in registers for the whole walk
+// over the request's tokens. Four tokens cost eight products of a vector with S, one transposing
+// exchange over the slices that leaves one of the eight sums in each, four broadcasts of the reads by
+// k, ten multiply-adds for the four u, and one update of S. DS_TOK tokens at a time come through shared
+// memory by asynchronous copies, two buffers. The order of every sum depends on the sizes alone.
 #define DS_TOK 16
-#define DS_COLS 16
-#define DS_THREADS (8 * DS_COLS)
+#define DS_THREADS 256
 
 __device__ __forceinline__ void ds_copy4(float* dst, const float* src, bool valid) {
     const int n = valid ? 4 : 0;
@@ -293,72 +387,69 @@ __device__ __forceinline__ void ds_copy16(float* dst, const void* src, bool vali
                      (uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(n));
 }
 
-// g x. A memory that decays slowly is multiplied by nearly 1 a thousand times, and a factor rounded
-// to the same side each time adds up: the float32 engine adds (g - 1) x while the decay is slow,
-// whose rounding is relative to the change.
-template <typename T> __device__ __forceinline__ float dl_decay(float x, float g, float gm1);
-template <> __device__ __forceinline__ float dl_decay<bf16>(float x, float g, float gm1) { return g * x; }
-template <> __device__ __forceinline__ float dl_decay<float>(float x, float g, float gm1) {
-    return gm1 > -0.3f ? fmaf(gm1, x, x) : g * x;
-}
+// A memory that decays slowly is multiplied by nearly 1 a thousand times, and a factor rounded to the
+// same side each time adds up: the float32 engine adds (P - 1) S while the decay is slow, whose rounding
+// is relative to the change.
+template <typename T> __device__ __forceinline__ bool dl_slow(float pm1) { return false; }
+template <> __device__ __forceinline__ bool dl_slow<float>(float pm1) { return pm1 > -0.3f; }
 
-template <typename T, int NI>
+template <typename T, int L, int NQ>
 __global__ void __launch_bounds__(DS_THREADS)
-delta_scan_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float4* __restrict__ gates,
-                  const float4* __restrict__ pairs, float* __restrict__ y, int H, int G, int dk, int dv,
+delta_scan_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float4* __restrict__ records,
+                  float* __restrict__ y, int H, int G, int dk, int dv,
                   const int* __restrict__ q_start, const int* __restrict__ state_slots, float* __restrict__ state,
                   long long state_stride, long long mem_offset, const T* __restrict__ conv_in,
                   long long conv_in_stride, int taps, long long conv_offset) {
-    constexpr int DKP = NI * 8;
-    constexpr int BUF = DS_TOK * (2 * DKP + DS_COLS + 8);
-    extern __shared__ __align__(16) float smem[];        // 2 x { qk [TOK][2 DKP], gates [TOK][4], pairs [TOK][4], v }
+    constexpr int NI = 4 * NQ, DKP = L * NI, CG = 32 / L, COLS = DS_THREADS / L;
+    constexpr int BUF = DS_TOK * (2 * DKP + COLS + 12);
+    extern __shared__ __align__(16) float smem[];        // 2 x { qk [TOK][2 DKP], records [TOK][12], v [TOK][COLS] }
     pdl_wait();
-    const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DS_COLS;
+    const int b = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
     const int t0 = q_start[b], n_tok = q_start[b + 1] - t0;
     if (n_tok <= 0) return;
     const int g = h / (H / G);
-    const int lane = threadIdx.x & 31, col = (threadIdx.x >> 5) * 4 + (lane & 3), s = lane >> 2;
-    const int c = c0 + col;
+    const int lane = threadIdx.x & 31, cg = lane % CG, s = lane / CG;
+    const int col = (threadIdx.x >> 5) * CG + cg, c = c0 + col;
     float* row = state + (size_t)state_slots[b] * state_stride;
     float* Sg = row + mem_offset + (size_t)h * dk * dv;
     // the memory comes and goes through shared memory ([dk][COLS + 1] floats fit in the buffers)
-    for (int i = threadIdx.x; i < dk * DS_COLS; i += DS_THREADS) {
-        const int n = i / DS_COLS, cc = i % DS_COLS;
-        smem[n * (DS_COLS + 1) + cc] = c0 + cc < dv ? Sg[(size_t)n * dv + c0 + cc] : 0.f;
+    for (int i = threadIdx.x; i < dk * COLS; i += DS_THREADS) {
+        const int n = i / COLS, cc = i % COLS;
+        smem[n * (COLS + 1) + cc] = c0 + cc < dv ? Sg[(size_t)n * dv + c0 + cc] : 0.f;
     }
     __syncthreads();
     float S[NI];
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-        const int n = 32 * (i >> 2) + 4 * s + (i & 3);
-        S[i] = n < dk ? smem[n * (DS_COLS + 1) + col] : 0.f;
+        const int n = 4 * s + 4 * L * (i >> 2) + (i & 3);
+        S[i] = n < dk ? smem[n * (COLS + 1) + col] : 0.f;
     }
     __syncthreads();
     auto stage = [&](int base, int buf) {
         float* qks = smem + buf * BUF;
-        float* gs = qks + DS_TOK * 2 * DKP;
-        float* ps = gs + DS_TOK * 4;
-        float* vs = ps + DS_TOK * 4;
-        const int nt = n_tok - base < DS_TOK ? n_tok - base : DS_TOK, ne = (nt + 1) & ~1;
+        float* rs = qks + DS_TOK * 2 * DKP;
+        float* vs = rs + DS_TOK * 12;
+        const int nt = n_tok - base < DS_TOK ? n_tok - base : DS_TOK, ne = (nt + 3) & ~3;
         for (int i = threadIdx.x; i < ne * (2 * DKP / 4); i += DS_THREADS) {
             const int r = i / (2 * DKP / 4), q = i % (2 * DKP / 4);
             const bool ok = r < nt;
             ds_copy16(qks + 4 * i, ok ? qk + ((size_t)(t0 + base + r) * G + g) * 2 * DKP + 4 * q : qk, ok);
         }
-        for (int i = threadIdx.x; i < ne * DS_COLS; i += DS_THREADS) {
-            const int r = i / DS_COLS, cc = i % DS_COLS;
+        for (int i = threadIdx.x; i < ne * COLS; i += DS_THREADS) {
+            const int r = i / COLS, cc = i % COLS;
             const bool ok = r < nt && c0 + cc < dv;
             ds_copy4(vs + i, ok ? v + ((size_t)(t0 + base + r) * H + h) * dv + c0 + cc : v, ok);
         }
-        if (threadIdx.x < ne) {
-            const bool ok = threadIdx.x < nt;
-            const size_t at = t0 + base + threadIdx.x;
-            ds_copy16(gs + 4 * threadIdx.x, ok ? (const void*)(gates + at * H + h) : (const void*)gates, ok);
-            ds_copy16(ps + 4 * threadIdx.x, ok ? (const void*)(pairs + at * G + g) : (const void*)pairs, ok);
+        if (threadIdx.x < 3 * ne) {
+            const int r = threadIdx.x / 3, part = threadIdx.x % 3;
+            const bool ok = r < nt;
+            ds_copy16(rs + 4 * threadIdx.x, ok ? records + ((size_t)(t0 + base + r) * H + h) * 3 + part : records, ok);
         }
         asm volatile("cp.async.commit_group;\n" ::);
     };
-    const bool upper = lane & 16, second = lane & 8;     // this lane's sum: by q (else k), of token 1 (else 0)
+    // the sum this slice ends with: the read by k of token `mine` of the four, or (by_q) by its q
+    const int vec = s / (L / 8), mine = vec & 3;
+    const bool stores = vec >= 4 && (s % (L / 8)) == 0 && c < dv;
     stage(0, 0);
     for (int base = 0, buf = 0; base < n_tok; base += DS_TOK, buf ^= 1) {
         const int nt = n_tok - base < DS_TOK ? n_tok - base : DS_TOK;
@@ -370,143 +461,175 @@ delta_scan_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
         }
         __syncthreads();
         const float* qks = smem + buf * BUF;
-        const float* gs = qks + DS_TOK * 2 * DKP;
-        const float* ps = gs + DS_TOK * 4;
-        const float* vs = ps + DS_TOK * 4;
-        for (int r = 0; r < nt; r += 2) {
+        const float* rs = qks + DS_TOK * 2 * DKP;
+        const float* vs = rs + DS_TOK * 12;
+        float* yt = y + ((size_t)(t0 + base + mine) * H + h) * dv + c;
+        auto four = [&](int r) {
             const float* q0 = qks + r * 2 * DKP + 4 * s;
-            const float* k0 = q0 + DKP;
-            const float* q1 = q0 + 2 * DKP;
-            const float* k1 = q1 + DKP;
-            const float4 ga = *(const float4*)(gs + 4 * r), pa = *(const float4*)(ps + 4 * r);
-            float4 gb = *(const float4*)(gs + 4 * r + 4), pb = *(const float4*)(ps + 4 * r + 4);
-            if (r + 1 >= nt) gb.x = 1.f;                 // no second token: it neither decays nor writes
-            const float va = vs[r * DS_COLS + col], vb = vs[(r + 1) * DS_COLS + col];
-            float4 ka[NI / 4], kb[NI / 4];
-            float sk0 = 0.f, sk1 = 0.f, sq0 = 0.f, sq1 = 0.f, tk0 = 0.f, tk1 = 0.f, tq0 = 0.f, tq1 = 0.f;
+            float4 ka[NQ][4];
+            float sum[8];                                // four reads by k, four by q
 #pragma unroll
-            for (int i = 0; i < NI / 4; ++i) {
-                ka[i] = *(const float4*)(k0 + 32 * i);
-                kb[i] = *(const float4*)(k1 + 32 * i);
-                const float4 qa = *(const float4*)(q0 + 32 * i), qb = *(const float4*)(q1 + 32 * i);
-                const float x = S[4 * i], yy = S[4 * i + 1], z = S[4 * i + 2], w = S[4 * i + 3];
-                sk0 = fmaf(ka[i].x, x, sk0); tk0 = fmaf(ka[i].y, yy, tk0);
-                sk1 = fmaf(kb[i].x, x, sk1); tk1 = fmaf(kb[i].y, yy, tk1);
-                sq0 = fmaf(qa.x, x, sq0);    tq0 = fmaf(qa.y, yy, tq0);
-                sq1 = fmaf(qb.x, x, sq1);    tq1 = fmaf(qb.y, yy, tq1);
-                sk0 = fmaf(ka[i].z, z, sk0); tk0 = fmaf(ka[i].w, w, tk0);
-                sk1 = fmaf(kb[i].z, z, sk1); tk1 = fmaf(kb[i].w, w, tk1);
-                sq0 = fmaf(qa.z, z, sq0);    tq0 = fmaf(qa.w, w, tq0);
-                sq1 = fmaf(qb.z, z, sq1);    tq1 = fmaf(qb.w, w, tq1);
-            }
-            sk0 += tk0; sk1 += tk1; sq0 += tq0; sq1 += tq1;
-            float a0 = upper ? sq0 : sk0, a1 = upper ? sq1 : sk1;
-            a0 += __shfl_xor_sync(0xffffffffu, upper ? sk0 : sq0, 16);
-            a1 += __shfl_xor_sync(0xffffffffu, upper ? sk1 : sq1, 16);
-            float m = second ? a1 : a0;
-            m += __shfl_xor_sync(0xffffffffu, second ? a0 : a1, 8);
-            m += __shfl_xor_sync(0xffffffffu, m, 4);
-            const float rk0 = __shfl_sync(0xffffffffu, m, lane & 3), rk1 = __shfl_sync(0xffffffffu, m, 8 + (lane & 3));
-            const float u0 = ga.z * (va - dl_decay<T>(rk0, ga.x, ga.y));
-            const float u1 = gb.z * (vb - dl_decay<T>(fmaf(pb.y, u0, dl_decay<T>(rk1, ga.x, ga.y)), gb.x, gb.y));
-            const float w0 = dl_decay<T>(u0, gb.x, gb.y);
-            const float gm = fmaf(ga.y, gb.y, ga.y + gb.y), gg = ga.x * gb.x;
-            if (sizeof(T) == 4 && gm > -0.3f) {
+            for (int j = 0; j < 8; ++j) sum[j] = 0.f;
 #pragma unroll
-                for (int i = 0; i < NI / 4; ++i) {
-                    S[4 * i] += fmaf(gm, S[4 * i], fmaf(kb[i].x, u1, ka[i].x * w0));
-                    S[4 * i + 1] += fmaf(gm, S[4 * i + 1], fmaf(kb[i].y, u1, ka[i].y * w0));
-                    S[4 * i + 2] += fmaf(gm, S[4 * i + 2], fmaf(kb[i].z, u1, ka[i].z * w0));
-                    S[4 * i + 3] += fmaf(gm, S[4 * i + 3], fmaf(kb[i].w, u1, ka[i].w * w0));
+            for (int i = 0; i < NQ; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float4 kk = *(const float4*)(q0 + j * 2 * DKP + DKP + 4 * L * i);
+                    const float4 qq = *(const float4*)(q0 + j * 2 * DKP + 4 * L * i);
+                    ka[i][j] = kk;
+                    sum[j] = fmaf(kk.x, S[4 * i], sum[j]);
+                    sum[4 + j] = fmaf(qq.x, S[4 * i], sum[4 + j]);
+                    sum[j] = fmaf(kk.y, S[4 * i + 1], sum[j]);
+                    sum[4 + j] = fmaf(qq.y, S[4 * i + 1], sum[4 + j]);
+                    sum[j] = fmaf(kk.z, S[4 * i + 2], sum[j]);
+                    sum[4 + j] = fmaf(qq.z, S[4 * i + 2], sum[4 + j]);
+                    sum[j] = fmaf(kk.w, S[4 * i + 3], sum[j]);
+                    sum[4 + j] = fmaf(qq.w, S[4 * i + 3], sum[4 + j]);
                 }
-            } else {
+            float4 ra[4];                                // (b P_j, the three k_m.k_j terms); zeros past the end
+            float2 rc[4];                                // P_j, E_j
+            float vj[4];
 #pragma unroll
-                for (int i = 0; i < NI / 4; ++i) {
-                    S[4 * i] = fmaf(kb[i].x, u1, fmaf(ka[i].x, w0, gg * S[4 * i]));
-                    S[4 * i + 1] = fmaf(kb[i].y, u1, fmaf(ka[i].y, w0, gg * S[4 * i + 1]));
-                    S[4 * i + 2] = fmaf(kb[i].z, u1, fmaf(ka[i].z, w0, gg * S[4 * i + 2]));
-                    S[4 * i + 3] = fmaf(kb[i].w, u1, fmaf(ka[i].w, w0, gg * S[4 * i + 3]));
+            for (int j = 0; j < 4; ++j) {
+                ra[j] = *(const float4*)(rs + 12 * (r + j));
+                rc[j] = *(const float2*)(rs + 12 * (r + j) + 8);
+                vj[j] = vs[(r + j) * COLS + col];
+            }
+            const float2 total = *(const float2*)(rs + 12 * r + 10);         // P_last, P_last - 1
+            const float4 rd = *(const float4*)(rs + 12 * (r + mine) + 4);
+            const float p_mine = rs[12 * (r + mine) + 8];
+#pragma unroll
+            for (int half = 4; half > 0; half >>= 1) {   // a slice keeps half of its sums
+                const int o = half * (L / 8);
+                const bool up = s & o;
+#pragma unroll
+                for (int i = 0; i < half; ++i) {
+                    const float give = up ? sum[i] : sum[i + half], have = up ? sum[i + half] : sum[i];
+                    sum[i] = have + __shfl_xor_sync(0xffffffffu, give, CG * o);
                 }
             }
-            if (upper && !(lane & 4) && c < dv && r + (second ? 1 : 0) < nt) {
-                const float first = dl_decay<T>(m, ga.x, ga.y);
-                const float o = second ? fmaf(pb.x, u1, dl_decay<T>(fmaf(pb.z, u0, first), gb.x, gb.y))
-                                       : fmaf(pa.x, u0, first);
-                y[((size_t)(t0 + base + r + (second ? 1 : 0)) * H + h) * dv + c] = o;
+#pragma unroll
+            for (int o = L / 16; o > 0; o >>= 1) sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], CG * o);
+            float u[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float x = __shfl_sync(0xffffffffu, sum[0], j * (L / 8) * CG + cg);
+                u[j] = fmaf(-ra[j].x, x, vj[j]);
             }
+            u[1] = fmaf(-ra[1].y, u[0], u[1]);
+            u[2] = fmaf(-ra[2].y, u[0], u[2]);
+            u[3] = fmaf(-ra[3].y, u[0], u[3]);
+            u[2] = fmaf(-ra[2].z, u[1], u[2]);
+            u[3] = fmaf(-ra[3].z, u[1], u[3]);
+            u[3] = fmaf(-ra[3].w, u[2], u[3]);
+            const float o0 = fmaf(rd.y, u[1], fmaf(rd.x, u[0], p_mine * sum[0]));
+            const float o1 = fmaf(rd.w, u[3], rd.z * u[2]);
+            if (stores && r + mine < nt) *yt = o0 + o1;
+            yt += (size_t)4 * H * dv;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) u[j] *= rc[j].y;                      // decayed by the later ones
+            const bool slow = dl_slow<T>(total.y);
+            const float f = slow ? total.y : total.x;
+#pragma unroll
+            for (int i = 0; i < NQ; ++i) {
+                float4 a = make_float4(f * S[4 * i], f * S[4 * i + 1], f * S[4 * i + 2], f * S[4 * i + 3]);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    a.x = fmaf(ka[i][j].x, u[j], a.x);
+                    a.y = fmaf(ka[i][j].y, u[j], a.y);
+                    a.z = fmaf(ka[i][j].z, u[j], a.z);
+                    a.w = fmaf(ka[i][j].w, u[j], a.w);
+                }
+                S[4 * i] = slow ? S[4 * i] + a.x : a.x;
+                S[4 * i + 1] = slow ? S[4 * i + 1] + a.y : a.y;
+                S[4 * i + 2] = slow ? S[4 * i + 2] + a.z : a.z;
+                S[4 * i + 3] = slow ? S[4 * i + 3] + a.w : a.w;
+            }
+        };
+        if (nt == DS_TOK) {                              // unrolled: the next four's rows load while these are joined
+#pragma unroll
+            for (int r = 0; r < DS_TOK; r += 4) four(r);
+        } else {
+            for (int r = 0; r < nt; r += 4) four(r);
         }
         __syncthreads();
     }
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-        const int n = 32 * (i >> 2) + 4 * s + (i & 3);
-        if (n < dk) smem[n * (DS_COLS + 1) + col] = S[i];
+        const int n = 4 * s + 4 * L * (i >> 2) + (i & 3);
+        if (n < dk) smem[n * (COLS + 1) + col] = S[i];
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < dk * DS_COLS; i += DS_THREADS) {
-        const int n = i / DS_COLS, cc = i % DS_COLS;
-        if (c0 + cc < dv) Sg[(size_t)n * dv + c0 + cc] = smem[n * (DS_COLS + 1) + cc];
+    for (int i = threadIdx.x; i < dk * COLS; i += DS_THREADS) {
+        const int n = i / COLS, cc = i % COLS;
+        if (c0 + cc < dv) Sg[(size_t)n * dv + c0 + cc] = smem[n * (COLS + 1) + cc];
     }
-    dl_keep_block(row + conv_offset, conv_in, conv_in_stride, H, G, dk, dv, h, c0, DS_COLS, taps, t0, n_tok);
+    dl_keep_block(row + conv_offset, conv_in, conv_in_stride, H, G, dk, dv, h, c0, COLS, taps, t0, n_tok);
 }
 
-template <typename T, int NI>
-static int launch_delta_scan(const float* qk, const float* v, const float* gates, const float* pairs, float* y,
+template <typename T, int L, int NQ>
+static int launch_delta_scan(const float* qk, const float* v, const float* records, float* y,
                              int B, int H, int G, int dk, int dv, const int* q_start, const int* state_slots,
                              float* state, long long state_stride, long long mem_offset, const T* conv_in,
                              long long conv_in_stride, int taps, long long conv_offset, cudaStream_t stream) {
-    const size_t smem = 2 * (size_t)DS_TOK * (2 * NI * 8 + DS_COLS + 8) * sizeof(float);
-    auto kernel = delta_scan_kernel<T, NI>;
+    constexpr int DKP = 4 * L * NQ, COLS = DS_THREADS / L;
+    const size_t smem = 2 * (size_t)DS_TOK * (2 * DKP + COLS + 12) * sizeof(float);
+    auto kernel = delta_scan_kernel<T, L, NQ>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return tgo_launch_pdl(kernel, dim3(B, H, (dv + DS_COLS - 1) / DS_COLS), dim3(DS_THREADS), smem, stream, qk, v,
-                          (const float4*)gates, (const float4*)pairs, y, H, G, dk, dv, q_start, state_slots, state,
+    return tgo_launch_pdl(kernel, dim3(B, H, (dv + COLS - 1) / COLS), dim3(DS_THREADS), smem, stream, qk, v,
+                          (const float4*)records, y, H, G, dk, dv, q_start, state_slots, state,
                           state_stride, mem_offset, conv_in, conv_in_stride, taps, conv_offset);
 }
 
 static bool delta_sizes_ok(int H, int G, int dk, int dv, int taps, long long state_stride, long long mem_offset,
                            long long conv_offset) {
-    return H > 0 && G > 0 && H % G == 0 && H <= 65535 && dk > 0 && dk <= 256 && dv > 0 && dv <= 65535 * DS_COLS &&
+    return H > 0 && G > 0 && H % G == 0 && H <= 65535 && dk > 0 && dk <= 256 && dv > 0 && dv <= 1 << 20 &&
            taps > 0 && taps <= 64 && state_stride >= mem_offset + (long long)H * dk * dv &&
            state_stride >= conv_offset + (long long)(taps - 1) * (2 * G * dk + H * dv);
 }
 
-TGO_API int tgo_delta_scan(const float* qk, const float* v, const float* gates, const float* pairs, float* y, int B,
+TGO_API int tgo_delta_scan(const float* qk, const float* v, const float* records, float* y, int B,
                            int H, int G, int dk, int dv, const int* q_start, const int* state_slots, float* state,
                            long long state_stride, long long mem_offset, const void* conv_in,
                            long long conv_in_stride, int dtype, int taps, long long conv_offset,
                            cudaStream_t stream) {
     if (B <= 0) return 0;
     if (!delta_sizes_ok(H, G, dk, dv, taps, state_stride, mem_offset, conv_offset) || (uintptr_t)qk % 16 ||
-        (uintptr_t)gates % 16 || (uintptr_t)pairs % 16 || (dtype != TGO_BF16 && dtype != TGO_F32))
+        (uintptr_t)records % 16 || (dtype != TGO_BF16 && dtype != TGO_F32))
         return TGO_E_BAD_ARG;
-#define DS_GO(TT, NI)                                                                                      \
-    launch_delta_scan<TT, NI>(qk, v, gates, pairs, y, B, H, G, dk, dv, q_start, state_slots, state, state_stride, \
-                              mem_offset, (const TT*)conv_in, conv_in_stride, taps, conv_offset, stream)
-#define DS_CASE(n) case n: return dtype == TGO_BF16 ? DS_GO(bf16, 4 * n) : DS_GO(float, 4 * n);
-    switch ((dk + 31) / 32) {                            // the rows are DKP = 32 n wide
-        DS_CASE(1) DS_CASE(2) DS_CASE(3) DS_CASE(4) DS_CASE(5) DS_CASE(6) DS_CASE(7) DS_CASE(8)
-    }
-#undef DS_CASE
+#define DS_GO(TT, L, NQ)                                                                                   \
+    launch_delta_scan<TT, L, NQ>(qk, v, records, y, B, H, G, dk, dv, q_start, state_slots, state, state_stride, \
+                                 mem_offset, (const TT*)conv_in, conv_in_stride, taps, conv_offset, stream)
+#define DS_SIZE(TT)                                                                                        \
+    (width == 32 ? DS_GO(TT, 8, 1) : width == 64 ? DS_GO(TT, 16, 1) : width == 128 ? DS_GO(TT, 16, 2) : DS_GO(TT, 16, 4))
+    const int width = delta_row_width(dk);
+    return dtype == TGO_BF16 ? DS_SIZE(bf16) : DS_SIZE(float);
+#undef DS_SIZE
 #undef DS_GO
-    return TGO_E_BAD_ARG;
 }
 
 // ----------------------------------------------------------------------------------- step
-// Requests of one token each. A block per (request, head): thread (row group q, column quad) holds
-// rows q, q + R, .. of four columns of S in registers between the reads and the update, so the memory
-// is read and written once, in whole rows. The reads by k and q are joined over the row groups
-// through shared memory, in order. Then, in the same block, the head's output is divided by its root
-// mean square over dv, multiplied by the gain [dv] and by SiLU of the gate.
-#define DT_THREADS 512
-template <typename T, int NR>
+// Requests of one token each. A block per (request, head): the head's memory comes into shared memory
+// whole by asynchronous copies, as many blocks to a multiprocessor as fit, and goes out once. Thread
+// (row group, column quad) takes rows q, q + R, .. of four columns; the reads by k and q are joined
+// over the row groups through shared memory, in order. Then, in the same block, the head's output is
+// divided by its root mean square over dv, multiplied by the gain [dv] and by SiLU of the gate.
+#define DT_THREADS 256
+#define DT_SMEM (200 * 1024)
+static size_t delta_step_smem(int dk, int dv) {
+    const int R = DT_THREADS / (dv / 4), dkp = delta_row_width(dk);
+    return ((size_t)dk * dv + 2 * dkp + 2 * dv + (size_t)2 * R * dv) * sizeof(float);
+}
+
+template <typename T>
 __global__ void __launch_bounds__(DT_THREADS)
-delta_step_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float4* __restrict__ gates,
-                  const float4* __restrict__ pairs, const T* __restrict__ z, long long z_stride,
+delta_step_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float4* __restrict__ records,
+                  const T* __restrict__ z, long long z_stride,
                   const float* __restrict__ gain, float eps, T* __restrict__ out, int H, int G, int dk, int dv,
                   int dkp, const int* __restrict__ q_start, const int* __restrict__ state_slots,
                   float* __restrict__ state, long long state_stride, long long mem_offset,
                   const T* __restrict__ conv_in, long long conv_in_stride, int taps, long long conv_offset) {
-    extern __shared__ __align__(16) float smem[];        // qk [2 dkp], u [dv], parts [2][R][dv]
+    extern __shared__ __align__(16) float smem[];        // S [dk][dv], qk [2 dkp], u [dv], o [dv], parts [2][R][dv]
     __shared__ float scratch[33];
     pdl_wait();
     const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
@@ -515,86 +638,80 @@ delta_step_kernel(const float* __restrict__ qk, const float* __restrict__ v, con
     const int QN = dv / 4, R = DT_THREADS / QN, g = h / (H / G);
     const int rg = tid / QN, quad = tid % QN;
     const bool works = rg < R;
-    float* qs = smem;
+    float* qs = smem + (size_t)dk * dv;
     float* us = qs + 2 * dkp;
-    float* part = us + dv;
+    float* os = us + dv;
+    float* part = os + dv;
     float* row = state + (size_t)state_slots[b] * state_stride;
-    float* Sg = row + mem_offset + (size_t)h * dk * dv + 4 * quad;
-    float4 S[NR];
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        const int n = rg + i * R;
-        S[i] = (works && n < dk) ? *(const float4*)(Sg + (size_t)n * dv) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    const float4 gt = gates[(size_t)t * H + h], pr = pairs[(size_t)t * G + g];
+    float* Sg = row + mem_offset + (size_t)h * dk * dv;
+    for (int i = tid; i < dk * QN; i += DT_THREADS) ds_copy16(smem + 4 * i, Sg + 4 * i, true);
+    asm volatile("cp.async.commit_group;\n" ::);
+    const float4* rec = records + ((size_t)t * H + h) * 3;
+    const float bp = rec[0].x, kq = rec[1].x, decay = rec[2].x, decay_m1 = rec[2].w;
     for (int i = tid; i < 2 * dkp; i += DT_THREADS) qs[i] = qk[((size_t)t * G + g) * 2 * dkp + i];
+    asm volatile("cp.async.wait_group 0;\n" ::);
     __syncthreads();
     if (works) {
         float4 sk = make_float4(0.f, 0.f, 0.f, 0.f), sq = sk;
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int n = rg + i * R;
-            if (n < dk) {
-                const float kn = qs[dkp + n], qn = qs[n];
-                sk.x = fmaf(kn, S[i].x, sk.x); sk.y = fmaf(kn, S[i].y, sk.y);
-                sk.z = fmaf(kn, S[i].z, sk.z); sk.w = fmaf(kn, S[i].w, sk.w);
-                sq.x = fmaf(qn, S[i].x, sq.x); sq.y = fmaf(qn, S[i].y, sq.y);
-                sq.z = fmaf(qn, S[i].z, sq.z); sq.w = fmaf(qn, S[i].w, sq.w);
-            }
+#pragma unroll 4
+        for (int n = rg; n < dk; n += R) {
+            const float kn = qs[dkp + n], qn = qs[n];
+            const float4 S = *(const float4*)(smem + (size_t)n * dv + 4 * quad);
+            sk.x = fmaf(kn, S.x, sk.x); sk.y = fmaf(kn, S.y, sk.y);
+            sk.z = fmaf(kn, S.z, sk.z); sk.w = fmaf(kn, S.w, sk.w);
+            sq.x = fmaf(qn, S.x, sq.x); sq.y = fmaf(qn, S.y, sq.y);
+            sq.z = fmaf(qn, S.z, sq.z); sq.w = fmaf(qn, S.w, sq.w);
         }
         *(float4*)(part + (size_t)rg * dv + 4 * quad) = sk;
         *(float4*)(part + (size_t)(R + rg) * dv + 4 * quad) = sq;
     }
     __syncthreads();
-    float o = 0.f;
-    if (tid < dv) {
+    float ss = 0.f;
+    for (int c = tid; c < dv; c += DT_THREADS) {
         float sk = 0.f, sq = 0.f;
         for (int i = 0; i < R; ++i) {
-            sk += part[(size_t)i * dv + tid];
-            sq += part[(size_t)(R + i) * dv + tid];
+            sk += part[(size_t)i * dv + c];
+            sq += part[(size_t)(R + i) * dv + c];
         }
-        const float u = gt.z * (v[((size_t)t * H + h) * dv + tid] - dl_decay<T>(sk, gt.x, gt.y));
-        us[tid] = u;
-        o = fmaf(pr.x, u, dl_decay<T>(sq, gt.x, gt.y));
+        const float u = fmaf(-bp, sk, v[((size_t)t * H + h) * dv + c]);
+        const float o = fmaf(kq, u, decay * sq);
+        us[c] = u;
+        os[c] = o;
+        ss += o * o;
     }
-    const float ss = block_sum(o * o, scratch);          // its barriers make `us` visible too
+    ss = block_sum(ss, scratch);                         // its barriers make `us` visible too
     if (works) {
         const float4 u = *(const float4*)(us + 4 * quad);
-        const bool slow = sizeof(T) == 4 && gt.y > -0.3f;
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int n = rg + i * R;
-            if (n < dk) {
-                const float kn = qs[dkp + n];
-                float4 r;
-                if (slow) {
-                    r.x = S[i].x + fmaf(gt.y, S[i].x, kn * u.x); r.y = S[i].y + fmaf(gt.y, S[i].y, kn * u.y);
-                    r.z = S[i].z + fmaf(gt.y, S[i].z, kn * u.z); r.w = S[i].w + fmaf(gt.y, S[i].w, kn * u.w);
-                } else {
-                    r.x = fmaf(kn, u.x, gt.x * S[i].x); r.y = fmaf(kn, u.y, gt.x * S[i].y);
-                    r.z = fmaf(kn, u.z, gt.x * S[i].z); r.w = fmaf(kn, u.w, gt.x * S[i].w);
-                }
-                *(float4*)(Sg + (size_t)n * dv) = r;
+        const bool slow = dl_slow<T>(decay_m1);
+#pragma unroll 4
+        for (int n = rg; n < dk; n += R) {
+            const float kn = qs[dkp + n];
+            const float4 S = *(const float4*)(smem + (size_t)n * dv + 4 * quad);
+            float4 r;
+            if (slow) {
+                r.x = S.x + fmaf(decay_m1, S.x, kn * u.x); r.y = S.y + fmaf(decay_m1, S.y, kn * u.y);
+                r.z = S.z + fmaf(decay_m1, S.z, kn * u.z); r.w = S.w + fmaf(decay_m1, S.w, kn * u.w);
+            } else {
+                r.x = fmaf(kn, u.x, decay * S.x); r.y = fmaf(kn, u.y, decay * S.y);
+                r.z = fmaf(kn, u.z, decay * S.z); r.w = fmaf(kn, u.w, decay * S.w);
             }
+            *(float4*)(Sg + (size_t)n * dv + 4 * quad) = r;
         }
     }
-    if (tid < dv) {
-        const float a = (o * rsqrtf(ss / (float)dv + eps)) * gain[tid];
-        out[((size_t)t * H + h) * dv + tid] =
-            from_f32<T>(a * dl_silu<T>(to_f32(z[(size_t)t * z_stride + (size_t)h * dv + tid])));
+    for (int c = tid; c < dv; c += DT_THREADS) {
+        const float a = (os[c] * rsqrtf(ss / (float)dv + eps)) * gain[c];
+        out[((size_t)t * H + h) * dv + c] =
+            from_f32<T>(a * dl_silu<T>(to_f32(z[(size_t)t * z_stride + (size_t)h * dv + c])));
     }
     dl_keep_block(row + conv_offset, conv_in, conv_in_stride, H, G, dk, dv, h, 0, dv, taps, t, 1);
 }
 
 TGO_API int tgo_delta_step_supports(int H, int G, int dk, int dv, long long state_stride, long long mem_offset) {
-    if (H <= 0 || G <= 0 || H % G || H > 65535 || dk <= 0 || dk > 256 || dv <= 0 || dv > DT_THREADS || dv % 4 ||
-        state_stride % 4 || mem_offset % 4)
-        return 0;
-    const int R = DT_THREADS / (dv / 4);
-    return (dk + R - 1) / R <= 16 ? 1 : 0;
+    return (H > 0 && G > 0 && H % G == 0 && H <= 65535 && dk > 0 && dk <= 256 && dv > 0 && dv <= 4 * DT_THREADS &&
+            dv % 4 == 0 && state_stride % 4 == 0 && mem_offset % 4 == 0 && delta_step_smem(dk, dv) <= DT_SMEM) ? 1 : 0;
 }
 
-TGO_API int tgo_delta_step(const float* qk, const float* v, const float* gates, const float* pairs, const void* z,
+TGO_API int tgo_delta_step(const float* qk, const float* v, const float* records, const void* z,
                            long long z_stride, const float* gain, float eps, void* out, int B, int H, int G, int dk,
                            int dv, const int* q_start, const int* state_slots, float* state, long long state_stride,
                            long long mem_offset, const void* conv_in, long long conv_in_stride, int dtype, int taps,
@@ -602,17 +719,20 @@ TGO_API int tgo_delta_step(const float* qk, const float* v, const float* gates, 
     if (B <= 0) return 0;
     if (!tgo_delta_step_supports(H, G, dk, dv, state_stride, mem_offset) ||
         !delta_sizes_ok(H, G, dk, dv, taps, state_stride, mem_offset, conv_offset) || (uintptr_t)state % 16 ||
-        (uintptr_t)gates % 16 || (uintptr_t)pairs % 16 || (dtype != TGO_BF16 && dtype != TGO_F32))
+        (uintptr_t)records % 16 || (dtype != TGO_BF16 && dtype != TGO_F32))
         return TGO_E_BAD_ARG;
-    const int R = DT_THREADS / (dv / 4), nr = (dk + R - 1) / R, dkp = (dk + 31) / 32 * 32;
-    const size_t smem = ((size_t)2 * dkp + dv + (size_t)2 * R * dv) * sizeof(float);    // at most 20 KB
-#define DT_GO(TT, NR)                                                                                      \
-    tgo_launch_pdl(delta_step_kernel<TT, NR>, dim3(B, H), dim3(DT_THREADS), smem, stream, qk, v, (const float4*)gates, \
-                   (const float4*)pairs, (const TT*)z, z_stride, gain, eps, (TT*)out, H, G, dk, dv, dkp, q_start, \
-                   state_slots, state, state_stride, mem_offset, (const TT*)conv_in, conv_in_stride, taps, conv_offset)
-#define DT_SIZE(TT) (nr <= 1 ? DT_GO(TT, 1) : nr <= 2 ? DT_GO(TT, 2) : nr <= 4 ? DT_GO(TT, 4) : nr <= 8 ? DT_GO(TT, 8) \
-                                                                                 : DT_GO(TT, 16))
-    return dtype == TGO_BF16 ? DT_SIZE(bf16) : DT_SIZE(float);
-#undef DT_SIZE
+    const int dkp = delta_row_width(dk);
+    const size_t smem = delta_step_smem(dk, dv);
+#define DT_GO(TT)                                                                                          \
+    do {                                                                                                   \
+        auto kernel = delta_step_kernel<TT>;                                                               \
+        if (smem > 48 * 1024)                                                                              \
+            cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);          \
+        return tgo_launch_pdl(kernel, dim3(B, H), dim3(DT_THREADS), smem, stream, qk, v, (const float4*)records, \
+                              (const TT*)z, z_stride, gain, eps, (TT*)out, H, G, dk, dv, dkp, q_start, state_slots, \
+                              state, state_stride, mem_offset, (const TT*)conv_in, conv_in_stride, taps, conv_offset); \
+    } while (0)
+    if (dtype == TGO_BF16) DT_GO(bf16);
+    DT_GO(float);
 #undef DT_GO
 }

@@ -537,8 +537,9 @@ gated_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate,
 
 // Groups of up to 512 channels: a warp a (token, group), the group's values in registers between
 // the sum of squares and the scaling, no block-wide sum. Four warps a block.
+// PER channels a lane.
 #define GGN_PER 16
-template <typename T>
+template <typename T, int PER>
 __global__ void __launch_bounds__(128)
 gated_group_norm_warp_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long gate_stride,
                              const float* __restrict__ gain, T* __restrict__ out, int width, int groups,
@@ -552,10 +553,10 @@ gated_group_norm_warp_kernel(const float* __restrict__ o, const T* __restrict__ 
     const int n = width / groups;
     const float* x = o + (size_t)t * width + (size_t)g * n;
     const T* gz = gate ? gate + (size_t)t * gate_stride + (size_t)g * n : nullptr;
-    float v[GGN_PER], z[GGN_PER];
+    float v[PER], z[PER];
     float ss = 0.f;
 #pragma unroll
-    for (int u = 0; u < GGN_PER; ++u) {
+    for (int u = 0; u < PER; ++u) {
         const int i = lane + 32 * u;
         v[u] = i < n ? x[i] : 0.f;
         z[u] = (gz && i < n) ? gate_value(to_f32(gz[i]), gate_act) : 1.f;
@@ -566,7 +567,7 @@ gated_group_norm_warp_kernel(const float* __restrict__ o, const T* __restrict__ 
     const float r = rsqrtf(ss / (float)n + eps);
     T* y = out + (size_t)t * width + (size_t)g * n;
 #pragma unroll
-    for (int u = 0; u < GGN_PER; ++u) {
+    for (int u = 0; u < PER; ++u) {
         const int i = lane + 32 * u;
         if (i < n) {
             float a = v[u] * r;
@@ -588,14 +589,12 @@ TGO_API int tgo_gated_group_norm(const float* o, const void* gate, long long gat
     const long long pairs = (long long)T * groups;
     if (n <= 32 * GGN_PER && (pairs + 3) / 4 <= 0x7fffffffLL) {
         const dim3 wgrid((unsigned)((pairs + 3) / 4)), wblock(128);
-        if (dtype == TGO_BF16)
-            return tgo_launch_pdl(gated_group_norm_warp_kernel<bf16>, wgrid, wblock, 0, stream, o,
-                                  (const bf16*)gate, gate_stride, gain, (bf16*)out, width, groups, eps, gate_act,
-                                  gate_first, pairs);
-        if (dtype == TGO_F32)
-            return tgo_launch_pdl(gated_group_norm_warp_kernel<float>, wgrid, wblock, 0, stream, o,
-                                  (const float*)gate, gate_stride, gain, (float*)out, width, groups, eps,
-                                  gate_act, gate_first, pairs);
+#define GGN_GO(TT, PER)                                                                                    \
+    tgo_launch_pdl(gated_group_norm_warp_kernel<TT, PER>, wgrid, wblock, 0, stream, o, (const TT*)gate, gate_stride, \
+                   gain, (TT*)out, width, groups, eps, gate_act, gate_first, pairs)
+        if (dtype == TGO_BF16) return n <= 32 * 4 ? GGN_GO(bf16, 4) : GGN_GO(bf16, GGN_PER);
+        if (dtype == TGO_F32) return n <= 32 * 4 ? GGN_GO(float, 4) : GGN_GO(float, GGN_PER);
+#undef GGN_GO
         return TGO_E_BAD_ARG;
     }
     const int threads = n >= 256 ? 256 : ((n + 31) / 32) * 32;

@@ -865,15 +865,159 @@ def measure_bekunex_kernels(width: int, heads: int, head_dim: int, latent_rank: 
     return out
 
 
+def measure_kesozen_kernels(width: int, heads: int, kv_heads: int, head_dim: int, delta_heads: int,
+                            delta_kv: int, delta_key: int, delta_value: int, taps: int, experts: int, top: int,
+                            groups: int, keep: int, expert_ff: int, prompt: int = 2048, batch: int = 64,
+                            context: int = 1024, page: int = 16, device="cuda:0") -> List[Dict[str, object]]:
+    """The kernels of the layers that norm each sublayer's input and output around an attention whose
+    values are its keys (one added to the denominator, a gate per head) or a gated delta rule, and
+    experts without a gate matrix chosen inside groups, each timed alone beside the like kernel of the
+    framework's closest layers at equal sizes (same timing and denominators as `measure_kernels`)."""
+    from types import SimpleNamespace
+
+    from ..parts.attention_sink import sink_attention
+    dev = torch.device(device)
+    peaks = load_peaks()
+    hbm, tc, fma = peaks["hbm_gbs"], peaks["bf16_tflops"], _fma_tflops(dev)
+    flush = L2Flusher(dev)
+    out: List[Dict[str, object]] = []
+    bf = torch.bfloat16
+
+    def row(name, ms, like, like_ms, bound, work, like_work=None):
+        peak = {"hbm": hbm * 1e9, "tensor": tc * 1e12, "fma": fma * 1e12}[bound]
+        rec = {"kernel": name, "us": round(ms * 1e3, 1), "bound": bound,
+               "frac": round(work / (ms * 1e-3) / peak, 4)}
+        if like:
+            rec.update(like=like, like_us=round(like_ms * 1e3, 1),
+                       like_frac=round((like_work or work) / (like_ms * 1e-3) / peak, 4))
+        out.append(rec)
+
+    def context_of(n_req, extent, first):
+        T = n_req * extent
+        pos = (torch.arange(extent, dtype=torch.int32, device=dev) + first).repeat(n_req)
+        seq = torch.arange(n_req, dtype=torch.int32, device=dev).repeat_interleave(extent)
+        qs = torch.arange(n_req + 1, dtype=torch.int32, device=dev) * extent
+        z = torch.zeros(n_req, dtype=torch.int32, device=dev)
+        return StepContext(T, n_req, pos, pos, seq, qs, z, torch.arange(n_req, dtype=torch.int32, device=dev),
+                           z, bf, extents=[extent] * n_req, first_positions=[first] * n_req,
+                           max_extent=extent, max_context=first + extent, decode_only=extent == 1)
+
+    H, G, dk = heads, kv_heads, head_dim
+    cases = ((1, prompt, 0, f"{prompt} tokens"), (batch, 1, context - 1, f"batch {batch} x {context} keys"))
+    # ---- attention: a constant sink and a gate per head, beside the learned sink without a gate; and
+    # the projection rows, whose keys are read twice, beside rows with values of their own
+    sinks, nought = torch.randn(H, device=dev), torch.zeros(H, device=dev)
+    for n_req, extent, first, what in cases:
+        T = n_req * extent
+        ctx = context_of(n_req, extent, first)
+        kc, table = _paged(n_req, first + extent, G, dk, page, dev)
+        vc, _ = _paged(n_req, first + extent, G, dk, page, dev)
+        rows = torch.randn((T, (H + 2 * G) * dk + H), device=dev).to(bf)
+        q, k, v = rows[:, :H * dk], rows[:, H * dk:(H + G) * dk], rows[:, (H + G) * dk:(H + 2 * G) * dk]
+        gate = rows[:, (H + 2 * G) * dk:]
+        o = torch.empty((T, H * dk), dtype=bf, device=dev)
+        cache = SimpleNamespace(k=kc, v=vc, page_size=page, block_tables=table)
+        ms = _timed(lambda: sink_attention(q, o, H, G, dk, dk, cache, ctx, 0.05, 0, nought, gate=gate), flush)
+        like_ms = _timed(lambda: sink_attention(q, o, H, G, dk, dk, cache, ctx, 0.05, 0, sinks), flush)
+        bound = ("tensor", 4.0 * H * dk * (prompt * (prompt + 1) / 2)) if extent > 1 else \
+            ("hbm", 4.0 * n_req * G * context * dk)
+        row(f"attention with one added and a gate per head, {what}", ms, "attention with a learned sink", like_ms, *bound)
+        slots = table.reshape(n_req, -1)[ctx.seq_ids.long(), (ctx.positions // page).long()] * page + ctx.positions % page
+        slots = slots.to(torch.int32).contiguous()
+        rot = ops.rope_table(ctx.positions, torch.rand(dk // 2, dtype=torch.float64, device=dev))
+        args = (H, G, dk, dk, None, None, None, rot, dk, False, slots, kc, vc, page)
+        ms = _timed(lambda: ops.qkv_bias_rope_cache(q, k, k, *args), flush)
+        like_ms = _timed(lambda: ops.qkv_bias_rope_cache(q, k, v, *args), flush)
+        row(f"projection rows, keys as values, {what}", ms, "projection rows with values", like_ms, "hbm",
+            2.0 * T * dk * (2 * H + 3 * G), 2.0 * T * dk * (2 * H + 4 * G))
+    # ---- the delta rule: its preparation beside the convolution of as many channels (with its kept
+    # inputs), the rule beside a selective scan with a state of equal size, single tokens with the norm
+    # and the gate beside scan and gated norm
+    Hd, Gd, dkd, dvd = delta_heads, delta_kv, delta_key, delta_value
+    C, vw, mem = 2 * Gd * dkd + Hd * dvd, Hd * dvd, Hd * dkd * dvd
+    floats = mem + (taps - 1) * C
+    w, wc = torch.randn((taps, C), device=dev) * 0.3, torch.randn((C, taps), device=dev) * 0.3
+    zero_h, one_h = torch.zeros(Hd, device=dev), torch.ones(Hd, device=dev)
+    gain, gain_row = torch.ones(dvd, device=dev), torch.ones(vw, device=dev)
+    C2 = vw + 2 * Gd * dkd
+    for n_req, extent, what in ((1, prompt, f"{prompt} tokens"), (batch, 1, f"batch {batch}"), (8, 1, "batch 8")):
+        T = n_req * extent
+        ctx = context_of(n_req, extent, 1)
+        rows = (torch.randn((T, C + vw + 2 * Hd), device=dev) * 0.5).to(bf)
+        raw, z, b, a = rows[:, :C], rows[:, C:C + vw], rows[:, C + vw:C + vw + Hd], rows[:, C + vw + Hd:]
+        st = torch.zeros((n_req + 1, floats), device=dev)
+        uf = torch.empty((T, C), device=dev)
+        sizes = (n_req, Hd, Gd, dkd, dvd)
+        prep = lambda: ops.delta_prepare(raw, w, b, a, zero_h, one_h, *sizes, ctx.seq_ids, ctx.q_start,   # noqa: E731
+                                         ctx.state_slots, st, mem)
+        ms = _timed(prep, flush)
+        like_ms = _timed(lambda: ops.causal_conv_act(raw, wc, None, uf, n_req, ctx.seq_ids, ctx.q_start,
+                                                     ctx.state_slots, st, mem), flush)
+        row(f"delta_prepare, {C} channels, {what}", ms, "causal_conv_act, float32 rows out + kept inputs", like_ms,
+            "hbm", 6.0 * T * C)
+        got = prep()
+        y = torch.empty((T, vw), device=dev)
+        n = torch.empty((T, vw), dtype=bf, device=dev)
+        xbc = torch.randn((T, C2), device=dev)
+        scan2 = lambda: ops.selective_scan(xbc, b, zero_h, zero_h, zero_h, y, n_req, Hd, Gd, dkd, dvd,     # noqa: E731
+                                           ctx.q_start, ctx.state_slots, st, 0)
+        norm = lambda: ops.gated_group_norm(y, z, gain_row, n, Hd, 1e-6, "silu", False)                    # noqa: E731
+        if extent > 1:
+            ms = _timed(lambda: ops.delta_scan(got, y, *sizes, ctx.q_start, ctx.state_slots, st, 0, raw, taps, mem), flush)
+            row(f"delta_scan, {Hd} heads of {dkd} x {dvd}, {what}", ms, "selective_scan, state of equal size",
+                _timed(scan2, flush), "fma", 6.0 * T * mem)
+            ms = _timed(norm, flush)
+            like_ms = _timed(lambda: ops.head_norm_gate(y, z, n, Hd, dvd, 1e-6), flush)
+            row(f"gated_group_norm, {what}", ms, "head_norm_gate", like_ms, "hbm", 8.0 * T * vw)
+        else:
+            ms = _timed(lambda: ops.delta_step(got, z, gain, 1e-6, n, *sizes, ctx.q_start, ctx.state_slots, st, 0, raw,
+                                               taps, mem), flush)
+            like_ms = _timed(lambda: (scan2(), norm()), flush)
+            row(f"delta_step with its norm and gate, {Hd} heads of {dkd} x {dvd}, {what}", ms,
+                "selective_scan, state of equal size, + gated_group_norm", like_ms, "hbm", 8.0 * n_req * mem)
+    # ---- the norms
+    for T, what in ((prompt, f"{prompt} rows"), (batch, f"{batch} rows")):
+        h, y = torch.randn((T, width), device=dev), torch.randn((T, width), device=dev)
+        n = torch.empty((T, width), dtype=bf, device=dev)
+        g = torch.ones(width, device=dev)
+        ms = _timed(lambda: ops.norm_add_norm(h, y, g, 1e-6, g, 1e-6, n), flush)
+        like_ms = _timed(lambda: (ops.group_norm_scale_add(h, y, g, None, 1e-6, 1),
+                                  ops.group_norm_rows(h, None, g, 1e-6, 1, n)), flush)
+        row(f"norm_add_norm, {what}", ms, "group_norm_scale_add + group_norm_rows", like_ms, "hbm", T * width * 14.0)
+        table = torch.randn((32768, width), device=dev).to(bf)
+        ids = torch.randint(0, 32768, (T,), dtype=torch.int32, device=dev)
+        ms = _timed(lambda: ops.embed_rmsnorm(table, ids, g, 1e-6, h, y), flush)
+        like_ms = _timed(lambda: ops.embed(table, ids, h), flush)
+        row(f"embed_rmsnorm with a copy, {what}", ms, "embed", like_ms, "hbm", T * width * 10.0, T * width * 6.0)
+    # ---- routed experts without a gate matrix: groups by their largest score, beside no groups
+    E, ff = experts, expert_ff
+    wr, corr = torch.randn((E, width), device=dev) * 0.05, torch.randn(E, device=dev) * 0.1
+    wu = (torch.randn((E, ff, width), device=dev) * 0.02).to(bf)
+    wd = (torch.randn((E, width, ff), device=dev) * 0.02).to(bf)
+    for T, what in ((prompt, f"{prompt} tokens"), (batch, f"batch {batch}"), (8, "batch 8")):
+        x = torch.randn((T, width), device=dev).to(bf)
+        ms = _timed(lambda: ops.moe_feed_forward(x, wr, None, None, wu, wd, top, "relu_squared", None, "all", corr, 0,
+                                                 False, groups, keep, False, 1.0, group_best=1), flush)
+        like_ms = _timed(lambda: ops.moe_feed_forward(x, wr, None, None, wu, wd, top, "relu_squared", None, "all", corr),
+                         flush)
+        bound = ("tensor", 4.0 * T * top * width * ff) if T >= 1024 else \
+            ("hbm", 4.0 * min(E, T * top) * width * ff)
+        row(f"routed experts without gates ({E}, top {top}, best {keep} of {groups} groups, ff {ff}), {what}", ms,
+            "routed experts without gates or groups", like_ms, *bound)
+    return out
+
+
 if __name__ == "__main__":
-    # python -m tgo_b200.engine.measure_kernels bekunex|vimelorn|derosun|totatar|gafonex [width]: the kernels of one design
+    # python -m tgo_b200.engine.measure_kernels kesozen|bekunex|vimelorn|derosun|totatar|gafonex [width]: the kernels of one design
     # at one size, a JSON line each (small enough to run under a profiler)
     import json
     import sys
     design = sys.argv[1] if len(sys.argv) > 1 else "totatar"
     w = int(sys.argv[2]) if len(sys.argv) > 2 else 2048
     ff = 3 * w
-    if design == "bekunex":
+    if design == "kesozen":
+        recs = measure_kesozen_kernels(w, 16, 4, 128, 16, 16, 128, 128, 4, 32, 4, 4, 2, ff // 8)
+    elif design == "bekunex":
         recs = measure_bekunex_kernels(w, 16, 128, 512, 64, 1024, 2 * w, 16, w // 16, 4, 32, 4, 4, 2, ff // 8)
     elif design == "vimelorn":
         recs = measure_vimelorn_kernels(w, 16, 4, 128, 128, 1024, 4, 4, 4, 32, 2, 4, ff // 8)

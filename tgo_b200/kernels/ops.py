@@ -1023,6 +1023,11 @@ def channel_scan(x: torch.Tensor, z: torch.Tensor, dt_raw: torch.Tensor, dt_bias
         "channel_scan", f"(channels={C}, state={N})")
 
 
+def delta_row_width(key_dim: int) -> int:
+    """How wide a prepared q or k row of the delta rule is: the next of 32, 64, 128 and 256."""
+    return next(w for w in (32, 64, 128, 256) if key_dim <= w)
+
+
 def delta_prepare(x: torch.Tensor, w: torch.Tensor, b_raw: torch.Tensor, a_raw: torch.Tensor,
                   dt_bias: torch.Tensor, decay: torch.Tensor, num_seqs: int, heads: int, groups: int,
                   key_dim: int, value_dim: int, seq_ids: torch.Tensor, q_start: torch.Tensor,
@@ -1032,9 +1037,9 @@ def delta_prepare(x: torch.Tensor, w: torch.Tensor, b_raw: torch.Tensor, a_raw: 
     the last row meets the current token; earlier inputs from the state row's [taps - 1, C] at
     `conv_offset`) and SiLU; q and k become unit vectors per head (q times key_dim^-1/2). b_raw and
     a_raw [T, heads]: the step size sigmoid(b) and the decay exp(-decay softplus(a + dt_bias)). All
-    float32: (qk [T, groups, 2, key_dim rounded up to 32], v [T, heads * value_dim], gates [T, heads,
-    4] = (g, g - 1, beta, 0), pairs [T, groups, 4] = k.q of a token and, for the second of a pair
-    counted from a request's first token of the step, k and q with the first one's k)."""
+    float32: (qk [T, groups, 2, `delta_row_width`], v times the step size [T, heads * value_dim],
+    records [T, heads, 12]: the factors of the rule that do not depend on the memory, for tokens
+    taken four at a time from a request's first token of the step)."""
     _need_cuda(x, w, b_raw, a_raw, dt_bias, decay, seq_ids, q_start, state_slots, state)
     T, C = x.shape
     taps = w.shape[0]
@@ -1048,32 +1053,30 @@ def delta_prepare(x: torch.Tensor, w: torch.Tensor, b_raw: torch.Tensor, a_raw: 
     assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
     assert seq_ids.dtype == q_start.dtype == state_slots.dtype == torch.int32
     assert q_start.numel() == num_seqs + 1 and state_slots.numel() == num_seqs and seq_ids.numel() == T
-    wide = (key_dim + 31) // 32 * 32
+    wide = delta_row_width(key_dim)
     n_qk, n_v = T * groups * 2 * wide, (T * heads * value_dim + 3) // 4 * 4
-    buf = torch.empty(n_qk + n_v + 4 * T * (heads + groups), dtype=torch.float32, device=x.device)
+    buf = torch.empty(n_qk + n_v + 12 * T * heads, dtype=torch.float32, device=x.device)
     qk = buf[:n_qk].view(T, groups, 2, wide)
     v = buf[n_qk:n_qk + T * heads * value_dim].view(T, heads * value_dim)
-    at = n_qk + n_v
-    gates = buf[at:at + 4 * T * heads].view(T, heads, 4)
-    pairs = buf[at + 4 * T * heads:].view(T, groups, 4)
+    records = buf[n_qk + n_v:].view(T, heads, 12)
     lib = load_library("delta")
     _check(lib.tgo_delta_prepare(
         _ptr(x), c_ll(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(w), _ptr(b_raw), _ptr(a_raw),
-        c_ll(a_raw.stride(0)), _ptr(dt_bias), _ptr(decay), _ptr(qk), _ptr(v), _ptr(gates), _ptr(pairs),
+        c_ll(a_raw.stride(0)), _ptr(dt_bias), _ptr(decay), _ptr(qk), _ptr(v), _ptr(records),
         c_int(T), c_int(num_seqs), c_int(heads), c_int(groups), c_int(key_dim), c_int(value_dim), c_int(taps),
         _ptr(seq_ids), _ptr(q_start), _ptr(state_slots), _ptr(state), c_ll(state.stride(0)),
         c_ll(conv_offset), _stream()), "delta_prepare",
         f"(heads={heads}/{groups}, dk={key_dim}, dv={value_dim}, taps={taps})")
-    return qk, v, gates, pairs
+    return qk, v, records
 
 
 def _delta_args(prepared, conv_in, heads, groups, key_dim, value_dim, num_seqs, q_start, state_slots, state):
-    qk, v, gates, pairs = prepared
+    qk, v, records = prepared
     T = qk.shape[0]
-    _need_cuda(qk, v, gates, pairs, conv_in, q_start, state_slots, state)
+    _need_cuda(qk, v, records, conv_in, q_start, state_slots, state)
     assert all(t.dtype == torch.float32 and t.is_contiguous() for t in prepared)
-    assert qk.shape == (T, groups, 2, (key_dim + 31) // 32 * 32) and v.shape == (T, heads * value_dim)
-    assert gates.shape == (T, heads, 4) and pairs.shape == (T, groups, 4)
+    assert qk.shape == (T, groups, 2, delta_row_width(key_dim)) and v.shape == (T, heads * value_dim)
+    assert records.shape == (T, heads, 12)
     assert conv_in.shape == (T, 2 * groups * key_dim + heads * value_dim) and conv_in.stride(1) == 1
     assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
     assert q_start.dtype == state_slots.dtype == torch.int32
@@ -1089,11 +1092,11 @@ def delta_scan(prepared: tuple, y: torch.Tensor, num_seqs: int, heads: int, grou
     value_dim]. The convolution's kept inputs [taps - 1, C] at `conv_offset` are moved on by the raw
     inputs `conv_in` [T, C]."""
     _delta_args(prepared, conv_in, heads, groups, key_dim, value_dim, num_seqs, q_start, state_slots, state)
-    qk, v, gates, pairs = prepared
+    qk, v, records = prepared
     assert y.dtype == torch.float32 and y.is_contiguous() and y.shape == v.shape and y.is_cuda
     lib = load_library("delta")
     _check(lib.tgo_delta_scan(
-        _ptr(qk), _ptr(v), _ptr(gates), _ptr(pairs), _ptr(y), c_int(num_seqs), c_int(heads), c_int(groups),
+        _ptr(qk), _ptr(v), _ptr(records), _ptr(y), c_int(num_seqs), c_int(heads), c_int(groups),
         c_int(key_dim), c_int(value_dim), _ptr(q_start), _ptr(state_slots), _ptr(state),
         c_ll(state.stride(0)), c_ll(mem_offset), _ptr(conv_in), c_ll(conv_in.stride(0)),
         c_int(dtype_code(conv_in.dtype)), c_int(taps), c_ll(conv_offset), _stream()), "delta_scan",
@@ -1115,14 +1118,14 @@ def delta_step(prepared: tuple, z: torch.Tensor, gain: torch.Tensor, eps: float,
     each head's row * silu(z), z [T, heads * value_dim] a 2-D view and out contiguous, both in the
     activation type, gain float32 [value_dim]."""
     _delta_args(prepared, conv_in, heads, groups, key_dim, value_dim, num_seqs, q_start, state_slots, state)
-    qk, v, gates, pairs = prepared
+    qk, v, records = prepared
     _need_cuda(z, gain, out)
     assert z.shape == out.shape == v.shape and z.stride(1) == 1 and out.is_contiguous()
     assert z.dtype == out.dtype == conv_in.dtype and num_seqs == v.shape[0]
     assert gain.dtype == torch.float32 and gain.numel() == value_dim and gain.is_contiguous()
     lib = load_library("delta")
     _check(lib.tgo_delta_step(
-        _ptr(qk), _ptr(v), _ptr(gates), _ptr(pairs), _ptr(z), c_ll(z.stride(0)), _ptr(gain), c_float(eps),
+        _ptr(qk), _ptr(v), _ptr(records), _ptr(z), c_ll(z.stride(0)), _ptr(gain), c_float(eps),
         _ptr(out), c_int(num_seqs), c_int(heads), c_int(groups), c_int(key_dim), c_int(value_dim),
         _ptr(q_start), _ptr(state_slots), _ptr(state), c_ll(state.stride(0)), c_ll(mem_offset),
         _ptr(conv_in), c_ll(conv_in.stride(0)), c_int(dtype_code(conv_in.dtype)), c_int(taps),
