@@ -419,11 +419,19 @@ FAMILIES = {"whole": tiny.trace_whole, "tail": lambda r: tiny.trace_tail(r, 12),
 @pytest.mark.parametrize("family", list(FAMILIES))
 @pytest.mark.parametrize("name", sorted(kt.CONFIGS))
 def test_replay_against_plain(models, tmp_path, name, family, dtype):
+    """K1 through the program that replays traces, the others through the engine it drives."""
+    import tgo_b200
     d, cfg, W, page = models[name]
     requests = tiny.random_requests(cfg["vocab"], [70, 9, 1, 45, 33, 21], seed=6)
     trace = FAMILIES[family](requests)
-    got = tiny.run_trace_program(d, dtype, trace, tmp_path / "out", cfg["vocab"],
-                                 extra=["--page-size", str(page), "--max-live", "4"])
+    if name == "K1":
+        got = tiny.run_trace_program(d, dtype, trace, tmp_path / "out", cfg["vocab"],
+                                     extra=["--page-size", str(page), "--max-live", "4"])
+    else:
+        eng = tgo_b200.open(d, dtype=dtype).new_engine(
+            page_size=page, max_tokens=tiny.max_tokens_of(trace, page), num_slots=4)
+        got = tiny.run_trace_engine(eng, trace)
+        eng.check_kernels()
     assert len(got) == sum(len(t) for t in requests.values())
     held = rows_close(got, cfg, W, requests, dtype)
     assert held >= len(got) // 2
